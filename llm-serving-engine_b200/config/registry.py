@@ -120,6 +120,18 @@ def _register_builtin() -> None:
             checkpoint_layout=lanilorn_checkpoint_layout,
         )
     )
+    from ..models.miberax import miberax_checkpoint_layout, miberax_plan
+    from .miberax import MiberaxConfig
+
+    register_architecture(
+        Architecture(
+            name="Miberax",
+            model_type="miberax",
+            config_cls=MiberaxConfig,
+            plan=miberax_plan,
+            checkpoint_layout=miberax_checkpoint_layout,
+        )
+    )
 
 
 _register_builtin()

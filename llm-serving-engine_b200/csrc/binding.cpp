@@ -88,13 +88,14 @@ void embedding(const Tensor& ids, const Tensor& table, Tensor& out) {
 }
 
 void add_rmsnorm(Tensor& x, const OptTensor& residual, const Tensor& weight, double eps,
-                 Tensor& out, const OptTensor& rows) {
+                 Tensor& out, const OptTensor& rows, int64_t groups) {
   check_f32(x, "x");
   check_f32(weight, "weight");
   check_cuda(out, "out");
   TORCH_CHECK(x.dim() == 2 && out.dim() == 2 && weight.dim() == 1, "add_rmsnorm: bad ranks");
   const int H = (int)x.size(1);
   TORCH_CHECK(weight.size(0) == H && out.size(1) == H, "add_rmsnorm: widths differ");
+  TORCH_CHECK(groups >= 1 && H % groups == 0, "add_rmsnorm: the groups must divide the width");
   int rcode = LSE_F32;
   const void* rptr = nullptr;
   if (residual) {
@@ -112,7 +113,7 @@ void add_rmsnorm(Tensor& x, const OptTensor& residual, const Tensor& weight, dou
   }
   TORCH_CHECK(out.size(0) == T, "add_rmsnorm: out has ", num(out.size(0)), " rows, expected ", num(T));
   done(lse_add_rmsnorm(x.data_ptr<float>(), rptr, rcode, weight.data_ptr<float>(), (float)eps,
-                       out.data_ptr(), dtype_code(out, "out"), rows_ptr, T, H, stream()),
+                       out.data_ptr(), dtype_code(out, "out"), rows_ptr, T, H, stream(), (int)groups),
        "add_rmsnorm");
 }
 
@@ -168,15 +169,26 @@ Tensor rope_kv_write(Tensor& qkv, int64_t nq, int64_t nk, int64_t D, const Tenso
   return q;
 }
 
-void silu_mul(const Tensor& gu, Tensor& out, int64_t act) {
+void silu_mul(const Tensor& gu, Tensor& out, int64_t act, double limit) {
   check_cuda(gu, "gu");
   check_cuda(out, "out");
   TORCH_CHECK(gu.dim() == 2 && out.dim() == 2 && gu.size(1) == 2 * out.size(1) &&
                   gu.size(0) == out.size(0),
               "silu_mul: gu must be [T, 2I] and out [T, I]");
   done(lse_silu_mul(gu.data_ptr(), dtype_code(gu, "gu"), out.data_ptr(), dtype_code(out, "out"),
-                    (int)gu.size(0), (int)out.size(1), (int)act, stream()),
+                    (int)gu.size(0), (int)out.size(1), (int)act, stream(), (float)limit),
        "silu_mul");
+}
+
+// z float32, bfloat16 or the fixed-point sums of a product (taken)
+void poly_norm(const Tensor& z, const Tensor& coef, double eps, Tensor& out) {
+  check_cuda(z, "z");
+  check_f32(coef, "coef");
+  check_cuda(out, "out");
+  TORCH_CHECK(z.dim() == 2 && out.sizes() == z.sizes() && coef.numel() == 4, "poly_norm: need z and out [T, N], coef [4]");
+  done(lse_poly_norm(z.data_ptr(), dtype_code(z, "z"), coef.data_ptr<float>(), (float)eps, out.data_ptr(),
+                     dtype_code(out, "out"), (int)z.size(0), (int)z.size(1), stream()),
+       "poly_norm");
 }
 
 void gemm_f32(const Tensor& a, const Tensor& w, const OptTensor& bias, Tensor& out) {
@@ -498,7 +510,8 @@ void head_linear(const Tensor& a, int64_t col0, const Tensor& w, Tensor& out, in
 }
 
 void moe_route(const Tensor& h, const Tensor& router, int64_t E, int64_t top, Tensor& idx, Tensor& wts,
-               const OptTensor& gate, const OptTensor& bias, int64_t mode) {
+               const OptTensor& gate, const OptTensor& bias, int64_t mode, int64_t groups, int64_t keep,
+               double scale) {
   check_cuda(h, "h");
   check_f32(router, "router");
   check_i32(idx, "idx");
@@ -516,7 +529,7 @@ void moe_route(const Tensor& h, const Tensor& router, int64_t E, int64_t top, Te
   }
   done(lse_moe_route(h.data_ptr(), out_code(h, "h"), router.data_ptr<float>(), (int)T, (int)W, (int)E,
                      has_gate, (int)top, idx.data_ptr<int>(), wts.data_ptr<float>(), g, stream(),
-                     opt_f32(bias, E, "router bias"), (int)mode),
+                     opt_f32(bias, E, "router bias"), (int)mode, (int)groups, (int)keep, (float)scale),
        "moe_route");
 }
 
@@ -589,7 +602,8 @@ void expert_linear(const Tensor& a, const Tensor& w, Tensor& out, const Tensor& 
 }
 
 void moe_combine(const Tensor& y, const Tensor& work, int64_t E, int64_t top, const OptTensor& shared_out,
-                 const OptTensor& gate, Tensor& out, bool accumulate, const OptTensor& wts) {
+                 const OptTensor& gate, Tensor& out, bool accumulate, const OptTensor& wts,
+                 const OptTensor& h) {
   check_f32(y, "y");
   check_i32(work, "work");
   check_f32(out, "out");
@@ -606,8 +620,17 @@ void moe_combine(const Tensor& y, const Tensor& work, int64_t E, int64_t top, co
       gp = gate->data_ptr<float>();
     }
   }
+  const void* hp = nullptr;  // what identity experts hand on
+  int hc = LSE_F32;
+  if (h) {
+    check_cuda(*h, "h");
+    TORCH_CHECK(h->sizes() == out.sizes(), "moe_combine: h needs out's shape");
+    hp = h->data_ptr();
+    hc = out_code(*h, "h");
+  }
   done(lse_moe_combine(y.data_ptr<float>(), work.data_ptr<int>() + E + 1 + n, (int)top, sp, gp,
-                       out.data_ptr<float>(), accumulate ? 1 : 0, (int)T, (int)W, stream(), opt_f32(wts, n, "experts' weights")),
+                       out.data_ptr<float>(), accumulate ? 1 : 0, (int)T, (int)W, stream(), opt_f32(wts, n, "experts' weights"),
+                       hp, hc),
        "moe_combine");
 }
 
@@ -649,12 +672,12 @@ const float* opt_f32(const OptTensor& t, int64_t n, const char* what) {
 }
 
 void rmsnorm_add(Tensor& x, const Tensor& a, const OptTensor& b, const OptTensor& wa, const OptTensor& wb,
-                 double ca, double cb, double eps_in, const Tensor& w, double eps, const OptTensor& out,
-                 const OptTensor& then_w, double then_eps) {
+                 double ca, double cb, double eps_in, const OptTensor& w, double eps, const OptTensor& out,
+                 const OptTensor& then_w, double then_eps, int64_t then_groups) {
   check_f32(x, "x");
   check_cuda(a, "a");
-  check_f32(w, "w");
-  TORCH_CHECK(x.dim() == 2 && a.sizes() == x.sizes() && w.numel() == x.size(1), "rmsnorm_add: bad shapes");
+  TORCH_CHECK(x.dim() == 2 && a.sizes() == x.sizes(), "rmsnorm_add: bad shapes");
+  TORCH_CHECK(then_groups >= 1 && x.size(1) % then_groups == 0, "rmsnorm_add: the groups must divide the width");
   const int branch_code = dtype_code(a, "a");  // float32, or the fixed-point sums of a few-rows product
   TORCH_CHECK(branch_code == LSE_F32 || branch_code == LSE_FIXED64, "rmsnorm_add: a must be float32 or sums");
   const int64_t H = x.size(1);
@@ -676,8 +699,8 @@ void rmsnorm_add(Tensor& x, const Tensor& a, const OptTensor& b, const OptTensor
   }
   TORCH_CHECK(!then_w || out, "rmsnorm_add: the norm that follows needs an output tensor");
   done(lse_rmsnorm_add(x.data_ptr<float>(), a.data_ptr(), bp, branch_code, opt_f32(wa, H, "wa"), opt_f32(wb, H, "wb"),
-                       (float)ca, (float)cb, (float)eps_in, w.data_ptr<float>(), (float)eps, op, oc,
-                       opt_f32(then_w, H, "then_w"), (float)then_eps, (int)x.size(0), (int)H, stream()),
+                       (float)ca, (float)cb, (float)eps_in, opt_f32(w, H, "w"), (float)eps, op, oc,
+                       opt_f32(then_w, H, "then_w"), (float)then_eps, (int)x.size(0), (int)H, stream(), (int)then_groups),
        "rmsnorm_add");
 }
 
@@ -759,6 +782,70 @@ void norm_rope_kv_write(const Tensor& qkv, Tensor& q_out, int64_t nq, int64_t nk
                               block_tables.data_ptr<int>(), (int)block_tables.size(1), (int)page_tokens,
                               (int)norm_dim, stream(), qkv.size(1)),
        "norm_rope_kv_write");
+}
+
+// proj: columns col0 .. of each row are q | k | v | gate | b | a (see lse_delta_inputs)
+void delta_inputs(const Tensor& proj, int64_t col0, const Tensor& conv, const OptTensor& conv_state, const Tensor& A_log,
+                  const Tensor& dt_bias, const Tensor& token_seq, const Tensor& cu_q, const Tensor& ctx_lens,
+                  const Tensor& slots, Tensor& qkv, Tensor& scal, int64_t H, int64_t G, int64_t dk, int64_t dv,
+                  double q_scale) {
+  check_f32(proj, "proj");
+  check_f32(conv, "conv");
+  check_f32(A_log, "A_log");
+  check_f32(dt_bias, "dt_bias");
+  check_i32(token_seq, "token_seq");
+  check_i32(cu_q, "cu_q");
+  check_i32(ctx_lens, "ctx_lens");
+  check_i32(slots, "slots");
+  check_f32(qkv, "qkv");
+  check_f32(scal, "scal");
+  TORCH_CHECK(H > 0 && G > 0 && H % G == 0 && dk > 0 && dk <= 256 && dv > 0, "delta_inputs: bad head counts or sizes");
+  const int64_t T = proj.size(0), C = 2 * G * dk + H * dv;
+  TORCH_CHECK(proj.dim() == 2 && col0 >= 0 && col0 + C + H * dv + 2 * H <= proj.size(1), "delta_inputs: columns outside proj");
+  TORCH_CHECK(conv.dim() == 2 && conv.size(0) >= 1 && conv.size(1) == C, "delta_inputs: conv must be [taps, channels]");
+  TORCH_CHECK(A_log.numel() == H && dt_bias.numel() == H, "delta_inputs: one A_log and dt_bias per head");
+  TORCH_CHECK(qkv.dim() == 2 && qkv.size(0) == T && qkv.size(1) == C && scal.numel() == T * H * 4,
+              "delta_inputs: qkv must be [T, channels], scal [T, heads, 4]");
+  TORCH_CHECK(token_seq.numel() >= T && cu_q.numel() == ctx_lens.numel() + 1 && slots.numel() >= ctx_lens.numel(),
+              "delta_inputs: the batch arrays disagree");
+  const int64_t taps = conv.size(0);
+  float* st = nullptr;
+  if (taps > 1) {
+    TORCH_CHECK(conv_state.has_value(), "delta_inputs: the convolution needs its state");
+    check_state(*conv_state, "conv_state", dk % 4 == 0 && dv % 4 == 0 ? 4 : 1);
+    TORCH_CHECK(conv_state->dim() == 3 && conv_state->size(1) == taps - 1 && conv_state->size(2) == C,
+                "delta_inputs: conv_state must be [slots, taps - 1, channels]");
+    st = conv_state->data_ptr<float>();
+  }
+  done(lse_delta_inputs(proj.data_ptr<float>() + col0, proj.size(1), conv.data_ptr<float>(), (int)taps, st,
+                        A_log.data_ptr<float>(), dt_bias.data_ptr<float>(), token_seq.data_ptr<int>(), cu_q.data_ptr<int>(),
+                        ctx_lens.data_ptr<int>(), slots.data_ptr<int>(), qkv.data_ptr<float>(), scal.data_ptr<float>(),
+                        (int)T, (int)H, (int)G, (int)dk, (int)dv, (float)q_scale, stream()),
+       "delta_inputs");
+}
+
+void delta_rule(const Tensor& qkv, const Tensor& scal, Tensor& state, Tensor& out, const Tensor& cu_q,
+                const Tensor& ctx_lens, const Tensor& slots, int64_t H, int64_t G, int64_t dk, int64_t dv) {
+  check_f32(qkv, "qkv");
+  check_f32(scal, "scal");
+  check_state(state, "state", dk);
+  check_f32(out, "out");
+  check_i32(cu_q, "cu_q");
+  check_i32(ctx_lens, "ctx_lens");
+  check_i32(slots, "slots");
+  TORCH_CHECK(H > 0 && G > 0 && H % G == 0 && dk > 0 && dk <= 256 && dv > 0, "delta_rule: bad head counts or sizes");
+  const int64_t T = qkv.size(0);
+  TORCH_CHECK(qkv.dim() == 2 && qkv.size(1) == 2 * G * dk + H * dv && scal.numel() == T * H * 4 && out.dim() == 2 &&
+                  out.size(0) == T && out.size(1) == H * dv,
+              "delta_rule: qkv must be [T, channels], scal [T, heads, 4], out [T, heads * value_dim]");
+  TORCH_CHECK(state.dim() == 4 && state.size(1) == H && state.size(2) == dv && state.size(3) == dk,
+              "delta_rule: state must be [slots, heads, value_dim, key_dim]");
+  TORCH_CHECK(cu_q.numel() == ctx_lens.numel() + 1 && slots.numel() >= ctx_lens.numel(),
+              "delta_rule: per-sequence arrays disagree");
+  done(lse_delta_rule(qkv.data_ptr<float>(), scal.data_ptr<float>(), state.data_ptr<float>(), out.data_ptr<float>(),
+                      cu_q.data_ptr<int>(), ctx_lens.data_ptr<int>(), slots.data_ptr<int>(), (int)ctx_lens.numel(),
+                      (int)H, (int)G, (int)dk, (int)dv, stream()),
+       "delta_rule");
 }
 
 void decay_linear_attention(const Tensor& proj, Tensor& out, Tensor& state, const OptTensor& decay, const Tensor& cu_q,
@@ -1175,7 +1262,7 @@ void qkv_norm_rope_write(const Tensor& proj, Tensor& q_out, int64_t nq, int64_t 
                          int64_t Dp, const OptTensor& qw, const OptTensor& kw, double eps, double temp_coef,
                          int64_t temp_every, const Tensor& positions, const Tensor& token_seq, const OptTensor& cos,
                          const OptTensor& sin, const OptTensor& k_pages, const OptTensor& v_pages,
-                         const Tensor& block_tables, int64_t page_tokens) {
+                         const Tensor& block_tables, int64_t page_tokens, int64_t col0) {
   check_f32(proj, "proj");
   check_cuda(q_out, "q_out");
   check_i32(positions, "positions");
@@ -1183,7 +1270,7 @@ void qkv_norm_rope_write(const Tensor& proj, Tensor& q_out, int64_t nq, int64_t 
   check_i32(block_tables, "block_tables");
   const int64_t T = proj.size(0);
   TORCH_CHECK(proj.dim() == 2 && nq > 0 && nk > 0 && nv >= 0 && D > 0 && Dp >= D && Dp <= 256 &&
-                  proj.size(1) >= (nq + nk) * D + nv * Dv,
+                  col0 >= 0 && col0 % 4 == 0 && proj.size(1) >= col0 + (nq + nk) * D + nv * Dv,
               "qkv_norm_rope_write: the projection is too narrow for these heads");
   TORCH_CHECK(q_out.dim() == 2 && q_out.size(0) == T && q_out.size(1) == nq * Dp, "qkv_norm_rope_write: q_out shape");
   TORCH_CHECK(positions.numel() >= T && token_seq.numel() >= T && block_tables.dim() == 2,
@@ -1210,7 +1297,7 @@ void qkv_norm_rope_write(const Tensor& proj, Tensor& q_out, int64_t nq, int64_t 
     kp = k_pages->data_ptr();
     vp = v_pages->data_ptr();
   }
-  done(lse_qkv_norm_rope_write(proj.data_ptr<float>(), proj.size(1), (int)T, (int)nq, (int)nk, (int)nv, (int)D, (int)Dv,
+  done(lse_qkv_norm_rope_write(proj.data_ptr<float>() + col0, proj.size(1), (int)T, (int)nq, (int)nk, (int)nv, (int)D, (int)Dv,
                                (int)Dp, opt_f32(qw, nq * D, "q weight"), opt_f32(kw, nk * D, "k weight"), (float)eps,
                                (float)temp_coef, (int)temp_every, positions.data_ptr<int>(), token_seq.data_ptr<int>(),
                                cos ? cos->data_ptr<float>() : nullptr, sin ? sin->data_ptr<float>() : nullptr, rot,
@@ -1237,9 +1324,12 @@ void differential_combine(const Tensor& a, const Tensor& gate, int64_t gate_col0
 
 PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("embedding", &embedding);
-  m.def("add_rmsnorm", &add_rmsnorm);
+  m.def("add_rmsnorm", &add_rmsnorm, py::arg("x"), py::arg("residual"), py::arg("weight"), py::arg("eps"),
+        py::arg("out"), py::arg("rows"), py::arg("groups") = 1);
   m.def("rope_kv_write", &rope_kv_write);
-  m.def("silu_mul", &silu_mul, py::arg("gu"), py::arg("out"), py::arg("act") = 0);
+  m.def("silu_mul", &silu_mul, py::arg("gu"), py::arg("out"), py::arg("act") = 0,
+        py::arg("limit") = 0.0);
+  m.def("poly_norm", &poly_norm);
   m.def("gemm_f32", &gemm_f32);
   m.def("gemm_bf16_skinny", &gemm_bf16_skinny);
   m.def("gemm_bf16_skinny_max_rows", &gemm_bf16_skinny_max_rows);
@@ -1262,20 +1352,26 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("head_linear", &head_linear, py::arg("a"), py::arg("col0"), py::arg("w"), py::arg("out"), py::arg("kind"),
         py::arg("a_head_cols") = 0, py::arg("out_head_cols") = 0);
   m.def("moe_route", &moe_route, py::arg("h"), py::arg("router"), py::arg("num_experts"), py::arg("top"),
-        py::arg("idx"), py::arg("wts"), py::arg("gate"), py::arg("bias") = py::none(), py::arg("mode") = 0);
+        py::arg("idx"), py::arg("wts"), py::arg("gate"), py::arg("bias") = py::none(), py::arg("mode") = 0,
+        py::arg("groups") = 1, py::arg("keep") = 1, py::arg("scale") = 1.0);
   m.def("moe_max_tiles", &moe_max_tiles);
   m.def("moe_tile_rows", &moe_tile_rows);
   m.def("moe_sort", &moe_sort);
   m.def("expert_linear", &expert_linear);
   m.def("moe_combine", &moe_combine, py::arg("y"), py::arg("work"), py::arg("num_experts"), py::arg("top"),
-        py::arg("shared_out"), py::arg("gate"), py::arg("out"), py::arg("accumulate"), py::arg("wts") = py::none());
+        py::arg("shared_out"), py::arg("gate"), py::arg("out"), py::arg("accumulate"), py::arg("wts") = py::none(),
+        py::arg("h") = py::none());
   m.def("latent_rope_write", &latent_rope_write);
   m.def("latent_query_rope", &latent_query_rope);
   m.def("sigmoid_gate_mul", &sigmoid_gate_mul);
   m.def("act_rows", &act_rows);
   m.def("cast_f32", &cast_f32);
   m.def("token_shift", &token_shift);
-  m.def("rmsnorm_add", &rmsnorm_add);
+  m.def("rmsnorm_add", &rmsnorm_add, py::arg("x"), py::arg("a"), py::arg("b"), py::arg("wa"), py::arg("wb"),
+        py::arg("ca"), py::arg("cb"), py::arg("eps_in"), py::arg("w"), py::arg("eps"), py::arg("out"),
+        py::arg("then_w"), py::arg("then_eps"), py::arg("then_groups") = 1);
+  m.def("delta_inputs", &delta_inputs);
+  m.def("delta_rule", &delta_rule);
   m.def("mix_normed", &mix_normed);
   m.def("gated_group_norm", &gated_group_norm);
   m.def("norm_rope_kv_write", &norm_rope_kv_write);
@@ -1286,7 +1382,11 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
   m.def("streams_spread", &streams_spread);
   m.def("streams_read_norm", &streams_read_norm);
   m.def("streams_write", &streams_write);
-  m.def("qkv_norm_rope_write", &qkv_norm_rope_write);
+  m.def("qkv_norm_rope_write", &qkv_norm_rope_write, py::arg("proj"), py::arg("q_out"), py::arg("nq"), py::arg("nk"),
+        py::arg("nv"), py::arg("D"), py::arg("Dv"), py::arg("Dp"), py::arg("qw"), py::arg("kw"), py::arg("eps"),
+        py::arg("temp_coef"), py::arg("temp_every"), py::arg("positions"), py::arg("token_seq"), py::arg("cos"),
+        py::arg("sin"), py::arg("k_pages"), py::arg("v_pages"), py::arg("block_tables"), py::arg("page_tokens"),
+        py::arg("col0") = 0);
   m.def("differential_combine", &differential_combine);
   m.def("linear_attention_chunk", []() { return (int64_t)lse_linear_attention_chunk(); });
   m.def("paged_attention_from_sums", &paged_attention_from_sums);

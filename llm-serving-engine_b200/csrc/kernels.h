@@ -30,7 +30,10 @@ int lse_embedding(const int* ids, const void* table, int table_dtype, float* out
 // cleared as they are read.
 int lse_add_rmsnorm(float* x, const void* residual, int residual_dtype, const float* weight,
                     float eps, void* out, int out_dtype, const int* rows, int T, int H,
-                    cudaStream_t stream);
+                    cudaStream_t stream,
+                    // groups > 1: every row is that many equal consecutive parts, normed one by one
+                    // (a fixed-point residual then needs parts of a multiple of 4)
+                    int groups = 1);
 
 // Rotate the q and k heads of the fused projection and write this step's k and v rows into their
 // pages. qkv [T, (nq + 2 nk) D] of in_dtype; the rotated queries go to q_out as `dtype`:
@@ -49,8 +52,16 @@ int lse_rope_kv_write(const void* qkv, int in_dtype, void* q_out, int dtype, int
 // as it is read). act: LSE_ACT_SILU (a / (1 + exp(-a))) or LSE_ACT_GELU_TANH (the tanh form of gelu).
 #define LSE_ACT_SILU 0
 #define LSE_ACT_GELU_TANH 1
+// or LSE_ACT_CLAMPED_GLU: g sigmoid(1.702 g) (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit)
+#define LSE_ACT_CLAMPED_GLU 2
 int lse_silu_mul(const void* gu, int in_dtype, void* out, int dtype, int T, int I, int act,
-                 cudaStream_t stream);
+                 cudaStream_t stream, float limit = 0.f);
+
+// out[t] = coef[0] N(z[t]) + coef[1] N(z[t]^2) + coef[2] N(z[t]^3) + coef[3], powers element by element,
+// N(y) = y / sqrt(mean(y^2) + eps) over the row's N values. z float32, bfloat16 or LSE_FIXED64 (taken;
+// bfloat16 out, N a multiple of 4 and at most 16384).
+int lse_poly_norm(const void* z, int in_dtype, const float* coef, float eps, void* out, int dtype, int T,
+                  int N, cudaStream_t stream);
 
 // True float32 matrix product: out[T, N] = a[T, K] . w[N, K]^T (+ bias[N]). Each output element is
 // accumulated over k in ascending order by one thread, so a row's result does not depend on T.
@@ -126,11 +137,13 @@ int lse_token_shift(const float* x, const float* mix, float* state, void* out, i
 // out (may be null) = the new x in out_dtype. rms(v) = sqrt(mean(v^2) + eps), eps_in for a and b.
 // branch_dtype: LSE_F32, or LSE_FIXED64 when a (and b) are the sums of few-rows products, which are
 // taken (left zero); then H * (b ? 2 : 1) floats must fit 48 KB of shared memory. With then_w,
-// out = then_w * x / rms(x) of the new x (eps then_eps) instead of the new x itself.
+// out = then_w * x / rms(x) of the new x (eps then_eps) instead of the new x itself. w null: x += y,
+// without the norm of y. then_groups > 1: the norm that follows takes every row as that many equal
+// parts (shared memory then also holds H / 4 floats, or H where a part is no multiple of 4).
 int lse_rmsnorm_add(float* x, const void* a, const void* b, int branch_dtype, const float* wa,
                     const float* wb, float ca, float cb, float eps_in, const float* w, float eps,
                     void* out, int out_dtype, const float* then_w, float then_eps, int T, int H,
-                    cudaStream_t stream);
+                    cudaStream_t stream, int then_groups = 1);
 // out = ca * wa * a / rms(a) (+ cb * wb * b / rms(b) if b)
 int lse_mix_normed(const float* a, const float* b, const float* wa, const float* wb, float ca,
                    float cb, float eps, float* out, int T, int H, cudaStream_t stream);
@@ -176,6 +189,26 @@ int lse_decay_linear_attention(const float* proj, long long stride, float* out, 
                                // gate_z is overwritten with the decays (it is the caller's temporary).
                                const float* gate_z = nullptr, long long gate_stride = 0, float decay_root = 1.f,
                                float query_scale = 1.f, float* chunk_decay = nullptr, int total_rows = 0);
+// ---- the gated delta rule (delta_rule.cu)
+
+// What enters the recurrence, from rows of proj (row length `stride`): q (G*dk) | k (G*dk) | v (H*dv) |
+// gate (H*dv) | b (H) | a (H); value head h belongs to key head h / (H / G).
+//   q, k, v: y[t] = sum_j conv[taps - 1 - j] * x[t - j] per channel (conv [taps, 2 G dk + H dv], zeros
+//   before the start; conv_state [slots, taps - 1, 2 G dk + H dv] keeps the last inputs, oldest
+//   first), then silu; q and k divided by sqrt(sum of squares + 1e-6) per head, q times q_scale.
+//   scal [T, H, 4] = (exp(-exp(A_log) softplus(a + dt_bias)), sigmoid(b), k . q, 0)
+// qkv [T, 2 G dk + H dv]. dk <= 256.
+int lse_delta_inputs(const float* proj, long long stride, const float* conv, int taps,
+                     float* conv_state, const float* A_log, const float* dt_bias, const int* token_seq,
+                     const int* cu_q, const int* ctx_lens, const int* slots, float* qkv, float* scal,
+                     int T, int H, int G, int dk, int dv, float q_scale, cudaStream_t stream);
+
+// S <- g S; u = beta (v - S^T k); S <- S + k u^T; out = S^T q per head and token, float32, with qkv and
+// scal as lse_delta_inputs leaves them; state [slots, H, dv, dk]; out [T, H*dv]. dk <= 256.
+int lse_delta_rule(const float* qkv, const float* scal, float* state, float* out, const int* cu_q,
+                   const int* ctx_lens, const int* slots, int num_seqs, int H, int G, int dk, int dv,
+                   cudaStream_t stream);
+
 // ---- several residual streams, rows of q/k/v prepared a token at a time, differential attention
 // (streams_mixers.cu). The residual state is float32 [T, S * W]: a token's S streams of W values.
 
@@ -255,21 +288,25 @@ int lse_head_linear(const void* a, int a_dtype, long long a_stride, long long a_
 // Routed experts. h [T, W]; router float32 [E (+1), W].
 //   lse_moe_route: z = router . h (+ bias); idx [T, top] the experts with the largest z (largest
 //     first, the lower index on a tie). mode 0: wts = sigmoid(z) of the chosen; mode 1: wts = the
-//     softmax over the chosen z alone. With has_gate, gate[t] = sigmoid(router[E] . h).
+//     softmax over the chosen z alone. mode 2: s = softmax(z) over all E; chosen by the largest
+//     s + bias among the `keep` best of `groups` equal groups of neighbours (a group's score is its
+//     largest s + bias; bias is no part of z); wts = s / (sum of the chosen s + 1e-20) * scale.
+//     With has_gate, gate[t] = sigmoid(router[E] . h).
 //   lse_moe_sort: the n = T * top choices sorted by expert: offsets [E + 1], perm [n] (sorted row ->
 //     choice), pos_of [n] (choice -> sorted row), and tiles of at most lse_moe_tile_rows() rows of one
 //     expert each (tile_batch, tile_row0: room for n / tile_rows + E entries; num_tiles [1]);
-//     tile_rows is lse_moe_tile_rows() for lse_expert_linear.
+//     tile_rows is lse_moe_tile_rows() for lse_expert_linear. Choices idx >= E (identity experts)
+//     get no row: pos_of = -1; perm beyond offsets[E] is zero.
 //   lse_expert_linear: out[r, :] = w[expert of r] . arow(r) for every sorted row r, float32 out
 //     [rows, N]; arow(r) = a[a_rows[r] / a_div] * a_scale[a_rows[r]] (a_rows null: a[r], unscaled);
 //     w [E, N, K]. Launched for max_tiles tiles; tiles beyond *num_tiles do nothing. kind as above
 //     (kinds 1 and 2 multiply the float32 sums by a_scale, which is the same product).
 //   lse_moe_combine: out[t] (+)= sum_k wts[t*top + k] * y[pos_of[t*top + k]] (+ gate[t] * shared_out[t]);
-//     wts null: 1; gate null: 1.
+//     wts null: 1; gate null: 1. A choice with pos_of < 0 adds wts * h[t] (h [T, W]; null: nothing).
 int lse_moe_tile_rows(void);
 int lse_moe_route(const void* h, int h_dtype, const float* router, int T, int W, int E, int has_gate,
                   int top, int* idx, float* wts, float* gate, cudaStream_t stream,
-                  const float* bias = nullptr, int mode = 0);
+                  const float* bias = nullptr, int mode = 0, int groups = 1, int keep = 1, float scale = 1.f);
 int lse_moe_sort(const int* idx, int n, int E, int tile_rows, int* offsets, int* perm, int* pos_of,
                  int* tile_batch, int* tile_row0, int* num_tiles, cudaStream_t stream);
 // out[r] = a[perm[r] / top] for the n sorted rows (bfloat16, K a multiple of 8)
@@ -289,7 +326,7 @@ int lse_expert_linear(const void* a, int a_dtype, long long a_stride, const int*
                       const int* num_tiles, int max_tiles, int kind, cudaStream_t stream);
 int lse_moe_combine(const float* y, const int* pos_of, int top, const float* shared_out,
                     const float* gate, float* out, int accumulate, int T, int W, cudaStream_t stream,
-                    const float* wts = nullptr);
+                    const float* wts = nullptr, const void* h = nullptr, int h_dtype = LSE_F32);
 
 // Latent attention with a rotated key part (rotary_latent.cu). cos/sin: float32 [positions, rot/2];
 // neighbouring dims (2i, 2i+1) are a pair; of a part's Dr dims the first rot are turned.

@@ -7,10 +7,12 @@
 //                     and scaled and whose weights are chosen per head (batched over heads) or per
 //                     tile (experts); each output element is one thread's in-order sum over k, so
 //                     a row's result does not depend on the batch it is in
-//   moe_route         a router's logits (+ bias), the top-k experts per token with sigmoid scores or
-//                     a softmax over the chosen logits, a shared gate
+//   moe_route         a router's logits (+ bias), the top-k experts per token with sigmoid scores,
+//                     a softmax over the chosen logits or a softmax over all of them (chosen by
+//                     the score plus a correction, from the best groups of experts), a shared gate
 //   moe_sort          tokens' expert choices sorted by expert, as tiles of rows for rows_gemm
-//   moe_combine       per token: the sum of its experts' rows (+ gate * shared expert), into x
+//   moe_combine       per token: the sum of its experts' rows (an identity expert's row is the
+//                     token's input itself) (+ gate * shared expert), into x
 #include "common.cuh"
 #include "kernels.h"
 
@@ -455,13 +457,17 @@ __global__ void __launch_bounds__(GV_WARPS * 32, 2) rows_gemv_kernel(const RowsG
 // first warp picks the `top` largest (the lower index on a tie). Their weights: sigmoid(z) (mode 0;
 // the sigmoid is monotone, so the order is that of z) or the softmax over the chosen z alone
 // (mode 1). Row E of the router, if there is one, is the shared expert's gate.
+// Mode 2: scores s = softmax(z) over all E; the choice goes by c = s + bias, which is then not part
+// of z; the experts form `groups` equal groups of neighbours, of which only the `keep` with the
+// largest c in them can be chosen from; a chosen expert's weight is s / (sum of the chosen s + 1e-20) * scale.
 constexpr int ROUTE_WARPS = 8;
 
 template <typename TH>
 __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 moe_route_kernel(const TH* __restrict__ h, const float* __restrict__ router, int W, int E,
                  int has_gate, int top, int* __restrict__ idx, float* __restrict__ wts,
-                 float* __restrict__ gate, const float* __restrict__ bias, int mode) {
+                 float* __restrict__ gate, const float* __restrict__ bias, int mode, int groups, int keep,
+                 float scale) {
   pdl_trigger();
   pdl_wait();  // everything below reads what kernels before this one wrote
   extern __shared__ float s[];  // [E + 1] scores, then [E + 1][ROUTE_WARPS] partial sums
@@ -482,11 +488,49 @@ moe_route_kernel(const TH* __restrict__ h, const float* __restrict__ router, int
     float d = 0.f;
 #pragma unroll
     for (int w = 0; w < ROUTE_WARPS; ++w) d += part[e * ROUTE_WARPS + w];
-    if (e < E) s[e] = d + (bias ? bias[e] : 0.f);
+    if (e < E) s[e] = d + (bias && mode != 2 ? bias[e] : 0.f);
     else gate[t] = 1.f / (1.f + expf(-d));
   }
   __syncthreads();
   if (warp != 0) return;
+  float* score = part;  // mode 2: the scores without the correction, [E] (the partial sums are used up)
+  if (mode == 2) {
+    float m = -INFINITY;
+    for (int e = lane; e < E; e += 32) m = fmaxf(m, s[e]);
+    m = warp_max(m);
+    float sum = 0.f;
+    for (int e = lane; e < E; e += 32) {
+      const float x = expf(s[e] - m);
+      score[e] = x;
+      sum += x;
+    }
+    sum = warp_sum(sum);
+    __syncwarp();
+    for (int e = lane; e < E; e += 32) {
+      const float x = score[e] / sum;
+      score[e] = x;
+      s[e] = x + (bias ? bias[e] : 0.f);
+    }
+    __syncwarp();
+    if (keep < groups) {
+      float* best_of = score + E;  // [groups]: the largest choice score of each group
+      const int size = E / groups;
+      for (int g = lane; g < groups; g += 32) {
+        float b = -INFINITY;
+        for (int e = g * size; e < (g + 1) * size; ++e) b = fmaxf(b, s[e]);
+        best_of[g] = b;
+      }
+      __syncwarp();
+      for (int g = lane; g < groups; g += 32) {  // a group is out if `keep` others come before it
+        int before = 0;
+        for (int o = 0; o < groups; ++o)
+          before += best_of[o] > best_of[g] || (best_of[o] == best_of[g] && o < g);
+        if (before >= keep)
+          for (int e = g * size; e < (g + 1) * size; ++e) s[e] = -INFINITY;
+      }
+      __syncwarp();
+    }
+  }
   float first = 0.f, total = 0.f;  // mode 1: the largest chosen logit, the sum of the exponentials
   for (int k = 0; k < top; ++k) {
     float best = -INFINITY;
@@ -507,7 +551,7 @@ moe_route_kernel(const TH* __restrict__ h, const float* __restrict__ router, int
     }
     if (bi == 0x7fffffff) bi = 0;  // only if every logit left is NaN
     if (k == 0) first = best;
-    const float wk = mode == 0 ? 1.f / (1.f + expf(-best)) : expf(best - first);
+    const float wk = mode == 0 ? 1.f / (1.f + expf(-best)) : mode == 1 ? expf(best - first) : score[bi];
     total += wk;
     if (lane == 0) {
       idx[t * top + k] = bi;
@@ -518,9 +562,12 @@ moe_route_kernel(const TH* __restrict__ h, const float* __restrict__ router, int
   }
   if (mode == 1)
     for (int k = lane; k < top; k += 32) wts[t * top + k] /= total;
+  if (mode == 2)
+    for (int k = lane; k < top; k += 32) wts[t * top + k] = wts[t * top + k] / (total + 1e-20f) * scale;
 }
 
-// One block. n choices idx[i] in [0, E): offsets[e] .. offsets[e+1] are expert e's rows in the
+// One block. A choice idx[i] >= E is an identity expert: it has no row in the sorted order
+// (pos_of[i] = -1), and perm beyond the last row is zero. The other choices in [0, E): offsets[e] .. offsets[e+1] are expert e's rows in the
 // sorted order, perm[r] the choice at sorted row r, pos_of[i] the sorted row of choice i, and the
 // rows as tiles of at most tile_rows rows of one expert (tile_batch, tile_row0, num_tiles).
 __global__ void __launch_bounds__(1024)
@@ -535,7 +582,8 @@ moe_sort_kernel(const int* __restrict__ idx, int n, int E, int tile_rows, int* _
   int* tstart = start + E + 1;
   for (int e = threadIdx.x; e < E; e += blockDim.x) counts[e] = 0;
   __syncthreads();
-  for (int i = threadIdx.x; i < n; i += blockDim.x) atomicAdd(&counts[idx[i]], 1);
+  for (int i = threadIdx.x; i < n; i += blockDim.x)
+    if (idx[i] < E) atomicAdd(&counts[idx[i]], 1);
   __syncthreads();
   if (threadIdx.x == 0) {
     int run = 0, tiles = 0;
@@ -563,10 +611,15 @@ moe_sort_kernel(const int* __restrict__ idx, int n, int E, int tile_rows, int* _
   // the order of an expert's rows among themselves is free: every row's result stands alone
   for (int i = threadIdx.x; i < n; i += blockDim.x) {
     const int e = idx[i];
+    if (e >= E) {
+      pos_of[i] = -1;
+      continue;
+    }
     const int r = start[e] + atomicAdd(&counts[e], 1);
     perm[r] = i;
     pos_of[i] = r;
   }
+  for (int r = start[E] + threadIdx.x; r < n; r += blockDim.x) perm[r] = 0;
 }
 
 // out[r] = a[perm[r] / top]: the tokens' rows in sorted order, in 16-byte pieces (K a multiple of 8)
@@ -583,14 +636,17 @@ moe_gather_rows_kernel(const bf16* __restrict__ a, const int* __restrict__ perm,
 }
 
 // x[t] (or out[t]) (+)= sum_k wts[t * top + k] * y[pos_of[t * top + k]] + gate[t] * shared[t] (a
-// null wts or gate counts as ones); a block per token and
+// null wts or gate counts as ones; a choice without a row, pos_of < 0, is an identity expert and adds
+// wts times the token's row of h); a block per token and
 // slice of 512 columns, four columns per thread (the experts' rows are added in the order k = 0, 1, ...)
 constexpr int COMBINE_SLICE = 512;
 
+template <typename TH>
 __global__ void __launch_bounds__(128)
 moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ pos_of, int top,
                    const float* __restrict__ shared_out, const float* __restrict__ gate,
-                   float* __restrict__ out, int accumulate, int W, const float* __restrict__ wts) {
+                   float* __restrict__ out, int accumulate, int W, const float* __restrict__ wts,
+                   const TH* __restrict__ h) {
   pdl_trigger();
   pdl_wait();  // everything below reads what kernels before this one wrote
   const int t = blockIdx.x;
@@ -600,8 +656,18 @@ moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ pos_of, 
 #pragma unroll
   for (int j = 0; j < COMBINE_SLICE / 128; ++j) v[j] = 0.f;
   for (int k = 0; k < top; ++k) {
-    const float* row = y + (size_t)pos_of[(size_t)t * top + k] * W;
+    const int pos = pos_of[(size_t)t * top + k];
     const float wk = wts ? wts[(size_t)t * top + k] : 1.f;
+    if (pos < 0) {
+      if (!h) continue;
+#pragma unroll
+      for (int j = 0; j < COMBINE_SLICE / 128; ++j) {
+        const int i = i0 + j * 128;
+        if (i < W) v[j] = fmaf(wk, Num<TH>::to_float(h[(size_t)t * W + i]), v[j]);
+      }
+      continue;
+    }
+    const float* row = y + (size_t)pos * W;
 #pragma unroll
     for (int j = 0; j < COMBINE_SLICE / 128; ++j) {
       const int i = i0 + j * 128;
@@ -739,16 +805,19 @@ extern "C" int lse_expert_linear(const void* a, int a_dtype, long long a_stride,
 
 extern "C" int lse_moe_route(const void* h, int h_dtype, const float* router, int T, int W, int E,
                              int has_gate, int top, int* idx, float* wts, float* gate,
-                             cudaStream_t stream, const float* bias, int mode) {
+                             cudaStream_t stream, const float* bias, int mode, int groups, int keep,
+                             float scale) {
   if (T <= 0) return LSE_OK;
-  if (E <= 0 || top <= 0 || top > E || E > 1024 || (has_gate && !gate) || mode < 0 || mode > 1) return LSE_BAD_ARGUMENT;
+  if (E <= 0 || top <= 0 || top > E || E > 1024 || (has_gate && !gate) || mode < 0 || mode > 2) return LSE_BAD_ARGUMENT;
+  if (mode == 2 && (groups < 1 || E % groups || keep < 1 || keep > groups || top > keep * (E / groups)))
+    return LSE_BAD_ARGUMENT;
   const size_t smem = (size_t)(E + 1) * (1 + ROUTE_WARPS) * sizeof(float);
   if (h_dtype == LSE_F32)
     launch(moe_route_kernel<float>, T, ROUTE_WARPS * 32, smem, stream, (const float*)h, router, W, E, has_gate, top,
-                                                                   idx, wts, gate, bias, mode);
+                                                                   idx, wts, gate, bias, mode, groups, keep, scale);
   else if (h_dtype == LSE_BF16)
     launch(moe_route_kernel<bf16>, T, ROUTE_WARPS * 32, smem, stream, (const bf16*)h, router, W, E, has_gate, top,
-                                                                  idx, wts, gate, bias, mode);
+                                                                  idx, wts, gate, bias, mode, groups, keep, scale);
   else
     return LSE_BAD_ARGUMENT;
   return LSE_CHECK_LAUNCH();
@@ -776,9 +845,16 @@ extern "C" int lse_moe_gather_rows(const void* a, const int* perm, int top, void
 
 extern "C" int lse_moe_combine(const float* y, const int* pos_of, int top, const float* shared_out,
                                const float* gate, float* out, int accumulate, int T, int W,
-                               cudaStream_t stream, const float* wts) {
+                               cudaStream_t stream, const float* wts, const void* h, int h_dtype) {
   if (T <= 0) return LSE_OK;
-  launch(moe_combine_kernel, dim3(T, (W + COMBINE_SLICE - 1) / COMBINE_SLICE), 128, 0, stream, y, pos_of, top,
-         shared_out, gate, out, accumulate, W, wts);
+  const dim3 grid(T, (W + COMBINE_SLICE - 1) / COMBINE_SLICE);
+  if (h && h_dtype == LSE_BF16)
+    launch(moe_combine_kernel<bf16>, grid, 128, 0, stream, y, pos_of, top, shared_out, gate, out, accumulate, W, wts,
+           (const bf16*)h);
+  else if (!h || h_dtype == LSE_F32)
+    launch(moe_combine_kernel<float>, grid, 128, 0, stream, y, pos_of, top, shared_out, gate, out, accumulate, W, wts,
+           (const float*)h);
+  else
+    return LSE_BAD_ARGUMENT;
   return LSE_CHECK_LAUNCH();
 }

@@ -38,6 +38,8 @@ __global__ void embedding_kernel(const int* __restrict__ ids, const T* __restric
 // ------------------------------------------------------------------------------------ rms norm
 // One block per output row. The row is visited twice by the same threads at the same indices, so
 // the second visit sees this thread's own writes of the first.
+// With groups > 1 a row is `groups` equal consecutive parts that are normed one by one: a block per
+// part, H being a part's size (weight and rows are indexed by the whole row).
 // V = 4 or 8 elements at a time (8: two groups of four for float, one 16-byte vector for bfloat16)
 template <typename T, int V>
 __device__ __forceinline__ void loadv(const T* p, float (&v)[V]) {
@@ -78,16 +80,17 @@ __device__ __forceinline__ void storev(T* p, const float (&v)[V]) {
 template <typename TR, typename TO, bool VEC4>
 __global__ void add_rmsnorm_kernel(float* __restrict__ x, const TR* __restrict__ residual,
                                    const float* __restrict__ weight, float eps,
-                                   TO* __restrict__ out, const int* __restrict__ rows, int H) {
+                                   TO* __restrict__ out, const int* __restrict__ rows, int H, int groups) {
   __shared__ float scratch[32];
   pdl_trigger();
   pdl_wait();
-  const int r = blockIdx.x;
-  const int src_row = rows ? rows[r] : r;
-  float* xr = x + (size_t)src_row * H;
-  const TR* rr = residual ? residual + (size_t)src_row * H : nullptr;
+  const int r = blockIdx.x / groups, g = blockIdx.x - r * groups;
+  const size_t src = ((size_t)(rows ? rows[r] : r) * groups + g) * H;
+  float* xr = x + src;
+  const TR* rr = residual ? residual + src : nullptr;
   const bool in_place = (rows == nullptr) && (rr != nullptr);
-  TO* o = out + (size_t)r * H;
+  TO* o = out + (size_t)blockIdx.x * H;
+  weight += (size_t)g * H;
   float ss = 0.f;
   if (VEC4) {
     for (int i = threadIdx.x * 4; i < H; i += blockDim.x * 4) {
@@ -143,9 +146,11 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ x, const TR* __restrict__
 template <typename TR, typename TO, int NV>
 __global__ void add_rmsnorm_regs_kernel(float* __restrict__ x, const TR* __restrict__ residual,
                                         const float* __restrict__ weight, float eps,
-                                        TO* __restrict__ out, const int* __restrict__ rows, int H) {
+                                        TO* __restrict__ out, const int* __restrict__ rows, int H, int groups) {
   __shared__ float scratch[32];
   pdl_trigger();
+  const int r = blockIdx.x / groups, g = blockIdx.x - r * groups;
+  weight += (size_t)g * H;
   float w[NV][4];
 #pragma unroll
   for (int k = 0; k < NV; ++k) {  // the weights are no result of the kernel before this one
@@ -153,12 +158,11 @@ __global__ void add_rmsnorm_regs_kernel(float* __restrict__ x, const TR* __restr
     if (i < H) load4<float>(weight + i, w[k]);
   }
   pdl_wait();
-  const int r = blockIdx.x;
-  const int src_row = rows ? rows[r] : r;
-  float* xr = x + (size_t)src_row * H;
-  const TR* rr = residual ? residual + (size_t)src_row * H : nullptr;
+  const size_t src = ((size_t)(rows ? rows[r] : r) * groups + g) * H;
+  float* xr = x + src;
+  const TR* rr = residual ? residual + src : nullptr;
   const bool in_place = (rows == nullptr) && (rr != nullptr);
-  TO* o = out + (size_t)r * H;
+  TO* o = out + (size_t)blockIdx.x * H;
   float v[NV][4];
 #pragma unroll
   for (int k = 0; k < NV; ++k) {
@@ -320,9 +324,16 @@ __global__ void rope_kv_write_vec_kernel(const TIn* qkv, T* q_out,
 // silu(a) * u. A bfloat16 result keeps 8 bits of mantissa, so the fast exponential and division
 // (relative error near 1e-6) give the same stored value as the exact ones; float32 results use
 // the exact ones.
-// act: LSE_ACT_SILU, or LSE_ACT_GELU_TANH = 0.5 a (1 + tanh(sqrt(2/pi) (a + 0.044715 a^3))).
+// act: LSE_ACT_SILU, or LSE_ACT_GELU_TANH = 0.5 a (1 + tanh(sqrt(2/pi) (a + 0.044715 a^3))), or
+// LSE_ACT_CLAMPED_GLU = g sigmoid(1.702 g) (u' + 1) with g = min(a, limit), u' = clamp(u, -limit, limit).
 template <typename T>
-__device__ __forceinline__ float silu_times(float a, float u, int act) {
+__device__ __forceinline__ float silu_times(float a, float u, int act, float limit) {
+  if (act == LSE_ACT_CLAMPED_GLU) {
+    a = fminf(a, limit);
+    u = fminf(fmaxf(u, -limit), limit) + 1.f;
+    if constexpr (std::is_same<T, bf16>::value) return __fdividef(a, 1.f + __expf(-1.702f * a)) * u;
+    else return a / (1.f + expf(-1.702f * a)) * u;
+  }
   if (act == LSE_ACT_GELU_TANH) {
     const float inner = 0.7978845608028654f * (a + 0.044715f * a * a * a);
     return 0.5f * a * (1.f + tanhf(inner)) * u;
@@ -331,7 +342,7 @@ __device__ __forceinline__ float silu_times(float a, float u, int act) {
   else return a / (1.f + expf(-a)) * u;
 }
 template <typename TIn, typename T>
-__global__ void silu_mul_kernel(const TIn* __restrict__ gu, T* __restrict__ out, int I, int act) {
+__global__ void silu_mul_kernel(const TIn* __restrict__ gu, T* __restrict__ out, int I, int act, float limit) {
   pdl_trigger();
   pdl_wait();
   const size_t t = blockIdx.x;
@@ -344,12 +355,12 @@ __global__ void silu_mul_kernel(const TIn* __restrict__ gu, T* __restrict__ out,
       load4<TIn>(g + i, gv);
       load4<TIn>(u + i, uv);
 #pragma unroll
-      for (int j = 0; j < 4; ++j) gv[j] = silu_times<T>(gv[j], uv[j], act);
+      for (int j = 0; j < 4; ++j) gv[j] = silu_times<T>(gv[j], uv[j], act, limit);
       store4<T>(o + i, gv);
     }
   } else {
     for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < I; i += gridDim.y * blockDim.x) {
-      o[i] = Num<T>::from_float(silu_times<T>(Num<TIn>::to_float(g[i]), Num<TIn>::to_float(u[i]), act));
+      o[i] = Num<T>::from_float(silu_times<T>(Num<TIn>::to_float(g[i]), Num<TIn>::to_float(u[i]), act, limit));
     }
   }
 }
@@ -359,7 +370,7 @@ __global__ void silu_mul_kernel(const TIn* __restrict__ gu, T* __restrict__ out,
 // vector per thread 15.6 us, two 19.0, four 28.8; the bytes alone take 15.1.)
 template <typename T>
 __global__ void silu_mul_wide_kernel(const T* __restrict__ gu, T* __restrict__ out, int I,
-                                     unsigned total, int act) {
+                                     unsigned total, int act, float limit) {
   constexpr int V = Num<T>::kVec;
   pdl_trigger();
   pdl_wait();
@@ -372,8 +383,80 @@ __global__ void silu_mul_wide_kernel(const T* __restrict__ gu, T* __restrict__ o
   Vec16<T> o;
 #pragma unroll
   for (int j = 0; j < V; ++j)
-    o.v[j] = Num<T>::from_float(silu_times<T>(Num<T>::to_float(g.v[j]), Num<T>::to_float(u.v[j]), act));
+    o.v[j] = Num<T>::from_float(silu_times<T>(Num<T>::to_float(g.v[j]), Num<T>::to_float(u.v[j]), act, limit));
   store16(out + (size_t)t * I + (size_t)c * V, o);
+}
+
+// ------------------------------------------------------------------------------------ polynomial of norms
+// out = a N(z) + b N(z^2) + c N(z^3) + e for each row z: powers element by element, N(y) = y / rms(y) of
+// the row; coef = {a, b, c, e}. One block per row. K > 0: a thread keeps its K groups of V elements
+// between the two visits (the only form for sums, which are cleared as they are read); K = 0: any
+// row length, z read twice.
+template <typename TIn, typename T, int V, int K>
+__global__ void poly_norm_kernel(const TIn* __restrict__ z, const float* __restrict__ coef, float eps,
+                                 T* __restrict__ out, int N) {
+  __shared__ float scratch[32];
+  pdl_trigger();
+  const float ca = coef[0], cb = coef[1], cc = coef[2], ce = coef[3];  // no result of a kernel before this one
+  pdl_wait();
+  const TIn* row = z + (size_t)blockIdx.x * N;
+  T* o = out + (size_t)blockIdx.x * N;
+  const int first = threadIdx.x * V, step = blockDim.x * V;
+  float s2 = 0.f, s4 = 0.f, s6 = 0.f;
+  auto ld = [&](int i, float (&v)[V]) {
+    if constexpr (V == 4) load4<TIn>(row + i, v);
+    else v[0] = Num<TIn>::to_float(row[i]);
+  };
+  auto sums = [&](const float (&v)[V]) {
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      const float q = v[j] * v[j];
+      s2 += q;
+      s4 = fmaf(q, q, s4);
+      s6 = fmaf(q * q, q, s6);
+    }
+  };
+  float keep[K > 0 ? K : 1][V];
+  if constexpr (K > 0) {
+#pragma unroll
+    for (int k = 0; k < K; ++k) {
+      const int i = first + k * step;
+      if (i < N) {
+        ld(i, keep[k]);
+        sums(keep[k]);
+      }
+    }
+  } else {
+    for (int i = first; i < N; i += step) {
+      float v[V];
+      ld(i, v);
+      sums(v);
+    }
+  }
+  s2 = block_sum(s2, scratch);
+  s4 = block_sum(s4, scratch);
+  s6 = block_sum(s6, scratch);
+  const float fa = ca * rsqrtf(s2 / (float)N + eps), fb = cb * rsqrtf(s4 / (float)N + eps),
+              fc = cc * rsqrtf(s6 / (float)N + eps);
+  auto put = [&](int i, float (&v)[V]) {
+#pragma unroll
+    for (int j = 0; j < V; ++j) v[j] = fmaf(v[j], fmaf(v[j], fmaf(v[j], fc, fb), fa), ce);
+    if constexpr (V == 4) store4<T>(o + i, v);
+    else o[i] = Num<T>::from_float(v[0]);
+  };
+  if constexpr (K > 0) {
+#pragma unroll
+    for (int k = 0; k < K; ++k) {
+      const int i = first + k * step;
+      if (i < N) put(i, keep[k]);
+    }
+  } else {
+    for (int i = first; i < N; i += step) {
+      float v[V];
+      ld(i, v);
+      put(i, v);
+    }
+  }
 }
 
 // ------------------------------------------------------------------------------------ fixed-point sums
@@ -430,8 +513,11 @@ extern "C" int lse_embedding(const int* ids, const void* table, int table_dtype,
 
 extern "C" int lse_add_rmsnorm(float* x, const void* residual, int residual_dtype,
                                const float* weight, float eps, void* out, int out_dtype,
-                               const int* rows, int T, int H, cudaStream_t stream) {
+                               const int* rows, int T, int H, cudaStream_t stream, int groups) {
   if (T <= 0) return LSE_OK;
+  if (groups < 1 || H % groups || (long long)T * groups > 0x7fffffffLL) return LSE_BAD_ARGUMENT;
+  H /= groups;  // from here on a part of a row, and a block per part
+  T *= groups;
   // Rows of up to 16384 elements: 16 elements per thread, held in registers, so that many rows
   // are resident on an SM together (2048 rows of 2048: 4.3 us; with 8 elements per thread 4.7, with
   // 4 elements 5.8). Longer rows: the kernel that visits the row twice.
@@ -441,13 +527,13 @@ extern "C" int lse_add_rmsnorm(float* x, const void* residual, int residual_dtyp
   do {                                                                        \
     if (regs)                                                                 \
       launch(add_rmsnorm_regs_kernel<TR, TO, 4>, T, threads, 0, stream,       \
-             x, (const TR*)residual, weight, eps, (TO*)out, rows, H);         \
+             x, (const TR*)residual, weight, eps, (TO*)out, rows, H, groups);         \
     else if (H % 4 == 0)                                                      \
       launch(add_rmsnorm_kernel<TR, TO, true>, T, threads, 0, stream,         \
-             x, (const TR*)residual, weight, eps, (TO*)out, rows, H);         \
+             x, (const TR*)residual, weight, eps, (TO*)out, rows, H, groups);         \
     else                                                                      \
       launch(add_rmsnorm_kernel<TR, TO, false>, T, threads, 0, stream,        \
-             x, (const TR*)residual, weight, eps, (TO*)out, rows, H);         \
+             x, (const TR*)residual, weight, eps, (TO*)out, rows, H, groups);         \
   } while (0)
   if (residual_dtype == LSE_F32 && out_dtype == LSE_F32) LSE_NORM(float, float);
   else if (residual_dtype == LSE_F32 && out_dtype == LSE_BF16) LSE_NORM(float, bf16);
@@ -458,10 +544,10 @@ extern "C" int lse_add_rmsnorm(float* x, const void* residual, int residual_dtyp
     if (!residual || rows || H % 4) return LSE_BAD_ARGUMENT;
     if (regs)
       launch(add_rmsnorm_regs_kernel<fixed64, bf16, 4>, T, threads, 0, stream, x,
-             (const fixed64*)residual, weight, eps, (bf16*)out, rows, H);
+             (const fixed64*)residual, weight, eps, (bf16*)out, rows, H, groups);
     else
       launch(add_rmsnorm_kernel<fixed64, bf16, true>, T, threads, 0, stream, x,
-             (const fixed64*)residual, weight, eps, (bf16*)out, rows, H);
+             (const fixed64*)residual, weight, eps, (bf16*)out, rows, H, groups);
   }
   else return LSE_BAD_ARGUMENT;
 #undef LSE_NORM
@@ -510,9 +596,9 @@ extern "C" int lse_rope_kv_write(const void* qkv, int in_dtype, void* q_out, int
 }
 
 extern "C" int lse_silu_mul(const void* gu, int in_dtype, void* out, int dtype, int T, int I,
-                            int act, cudaStream_t stream) {
+                            int act, cudaStream_t stream, float limit) {
   if (T <= 0 || I <= 0) return LSE_OK;
-  if (act != LSE_ACT_SILU && act != LSE_ACT_GELU_TANH) return LSE_BAD_ARGUMENT;
+  if (act != LSE_ACT_SILU && act != LSE_ACT_GELU_TANH && act != LSE_ACT_CLAMPED_GLU) return LSE_BAD_ARGUMENT;
   const int threads = 256;
   const int vec = in_dtype == LSE_BF16 ? 8 : 4;
   if (in_dtype == dtype && I % vec == 0 && (size_t)T * (I / vec) < (1ull << 31) &&
@@ -520,23 +606,53 @@ extern "C" int lse_silu_mul(const void* gu, int in_dtype, void* out, int dtype, 
     const unsigned total = (unsigned)((size_t)T * (I / vec));
     const unsigned blocks = (total + threads - 1) / threads;
     if (dtype == LSE_F32)
-      launch(silu_mul_wide_kernel<float>, blocks, threads, 0, stream, (const float*)gu, (float*)out, I, total, act);
+      launch(silu_mul_wide_kernel<float>, blocks, threads, 0, stream, (const float*)gu, (float*)out, I, total, act, limit);
     else
-      launch(silu_mul_wide_kernel<bf16>, blocks, threads, 0, stream, (const bf16*)gu, (bf16*)out, I, total, act);
+      launch(silu_mul_wide_kernel<bf16>, blocks, threads, 0, stream, (const bf16*)gu, (bf16*)out, I, total, act, limit);
     return LSE_CHECK_LAUNCH();
   }
   const int per_block = threads * 4;
   dim3 grid(T, min((I + per_block - 1) / per_block, 65535));
   if (in_dtype == LSE_F32 && dtype == LSE_F32)
-    launch(silu_mul_kernel<float, float>, grid, threads, 0, stream, (const float*)gu, (float*)out, I, act);
+    launch(silu_mul_kernel<float, float>, grid, threads, 0, stream, (const float*)gu, (float*)out, I, act, limit);
   else if (in_dtype == LSE_BF16 && dtype == LSE_BF16)
-    launch(silu_mul_kernel<bf16, bf16>, grid, threads, 0, stream, (const bf16*)gu, (bf16*)out, I, act);
+    launch(silu_mul_kernel<bf16, bf16>, grid, threads, 0, stream, (const bf16*)gu, (bf16*)out, I, act, limit);
   else if (in_dtype == LSE_F32 && dtype == LSE_BF16)
-    launch(silu_mul_kernel<float, bf16>, grid, threads, 0, stream, (const float*)gu, (bf16*)out, I, act);
+    launch(silu_mul_kernel<float, bf16>, grid, threads, 0, stream, (const float*)gu, (bf16*)out, I, act, limit);
   else if (in_dtype == LSE_FIXED64 && dtype == LSE_BF16 && I % 4 == 0)
-    launch(silu_mul_kernel<fixed64, bf16>, grid, threads, 0, stream, (const fixed64*)gu, (bf16*)out, I, act);
+    launch(silu_mul_kernel<fixed64, bf16>, grid, threads, 0, stream, (const fixed64*)gu, (bf16*)out, I, act, limit);
   else
     return LSE_BAD_ARGUMENT;
+  return LSE_CHECK_LAUNCH();
+}
+
+extern "C" int lse_poly_norm(const void* z, int in_dtype, const float* coef, float eps, void* out, int dtype, int T,
+                             int N, cudaStream_t stream) {
+  if (T <= 0) return LSE_OK;
+  if (N <= 0 || !coef) return LSE_BAD_ARGUMENT;
+  const bool vec = N % 4 == 0 && reinterpret_cast<uintptr_t>(z) % 16 == 0 && reinterpret_cast<uintptr_t>(out) % 16 == 0;
+  const int units = vec ? N / 4 : N;
+  // two groups of four per thread while that keeps a block at 1024 threads or fewer, then four
+  const int per = units <= 2048 ? 2 : 4;
+  const int threads = min(1024, ((units + per - 1) / per + 31) / 32 * 32);
+  const int visits = (units + threads - 1) / threads;
+#define LSE_PN(TIn, TO, V, K) \
+  launch(poly_norm_kernel<TIn, TO, V, K>, T, threads, 0, stream, (const TIn*)z, coef, eps, (TO*)out, N)
+#define LSE_PN_ANY(TIn, TO)                      \
+  do {                                           \
+    if (vec && visits <= 2) LSE_PN(TIn, TO, 4, 2); \
+    else if (vec && visits <= 4) LSE_PN(TIn, TO, 4, 4); \
+    else if (vec) LSE_PN(TIn, TO, 4, 0);         \
+    else LSE_PN(TIn, TO, 1, 0);                  \
+  } while (0)
+  if (in_dtype == LSE_F32 && dtype == LSE_F32) LSE_PN_ANY(float, float);
+  else if (in_dtype == LSE_F32 && dtype == LSE_BF16) LSE_PN_ANY(float, bf16);
+  else if (in_dtype == LSE_BF16 && dtype == LSE_BF16) LSE_PN_ANY(bf16, bf16);
+  else if (in_dtype == LSE_FIXED64 && dtype == LSE_BF16 && vec && visits <= 2) LSE_PN(fixed64, bf16, 4, 2);
+  else if (in_dtype == LSE_FIXED64 && dtype == LSE_BF16 && vec && visits <= 4) LSE_PN(fixed64, bf16, 4, 4);
+  else return LSE_BAD_ARGUMENT;
+#undef LSE_PN
+#undef LSE_PN_ANY
   return LSE_CHECK_LAUNCH();
 }
 

@@ -65,14 +65,31 @@ __global__ void token_shift_kernel(const float* __restrict__ x, const float* __r
 // K > 0: a thread visits at most K places of the row and keeps y and the new x of each in
 // registers, so that a and x are read once and x's old values are already on their way while the
 // block sums the squares; K = 0: any row length, y recomputed and x read back.
+// Without w the sum is x += y as it is. then_groups > 1: the next norm's rows are that many equal
+// parts normed one by one; the parts' sums are formed in shared memory behind what SUMS keeps there
+// (a part is a whole number of visits of V elements).
 template <typename TO, bool SUMS, int V, int K>
 __global__ void rmsnorm_add_kernel(float* __restrict__ x, const void* a, const void* b,
                                    const float* __restrict__ wa,
                                    const float* __restrict__ wb, float ca, float cb, float eps_in,
                                    const float* __restrict__ w, float eps, TO* __restrict__ out,
-                                   const float* __restrict__ then_w, float then_eps, int H) {
+                                   const float* __restrict__ then_w, float then_eps, int H, int then_groups) {
   __shared__ float scratch[32];
   extern __shared__ __align__(16) float taken[];  // SUMS: [H] for a, then [H] for b
+  float* part = taken + (SUMS ? (b ? 2 : 1) * H : 0);  // then_groups > 1: [H / V] sums of squares, then [groups]
+  const int part_size = H / then_groups;
+  float* part_inv = part + H / V;
+  auto norm_parts = [&]() {  // the parts' sums of squares (in `part`, a visit each) to 1 / rms
+    __syncthreads();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5, per = part_size / V;
+    for (int g = warp; g < then_groups; g += nw) {
+      float s = 0.f;
+      for (int i = lane; i < per; i += 32) s += part[g * per + i];
+      s = warp_sum(s);
+      if (lane == 0) part_inv[g] = rsqrtf(s / (float)part_size + then_eps);
+    }
+    __syncthreads();
+  };
   pdl_trigger();
   pdl_wait();
   const size_t row = (size_t)blockIdx.x * H;
@@ -156,34 +173,45 @@ __global__ void rmsnorm_add_kernel(float* __restrict__ x, const void* a, const v
         for (int j = 0; j < V; ++j) ss += yk[k][j] * yk[k][j];
       }
     }
-    ss = block_sum(ss, scratch);
-    const float inv = rsqrtf(ss / (float)H + eps);
+    float inv = 1.f;
+    if (w) {
+      ss = block_sum(ss, scratch);
+      inv = rsqrtf(ss / (float)H + eps);
+    }
     float s2 = 0.f;
 #pragma unroll
     for (int k = 0; k < K; ++k) {
       const int i = first + k * step;
       if (i < H) {
-        float wv[V];
-        ld(w + i, wv);
+        float wv[V], sq = 0.f;
+        if (w) ld(w + i, wv);
 #pragma unroll
         for (int j = 0; j < V; ++j) {
-          xk[k][j] += yk[k][j] * inv * wv[j];
-          s2 += xk[k][j] * xk[k][j];
+          xk[k][j] += w ? yk[k][j] * inv * wv[j] : yk[k][j];
+          sq += xk[k][j] * xk[k][j];
         }
+        s2 += sq;
+        if (then_w && then_groups > 1) part[i / V] = sq;
         if constexpr (V == 4) store4<float>(xr + i, xk[k]);
         else xr[i] = xk[k][0];
         if (out && !then_w) put(i, xk[k]);
       }
     }
     if (!out || !then_w) return;
-    s2 = block_sum(s2, scratch);
-    const float inv2 = rsqrtf(s2 / (float)H + then_eps);
+    float inv2 = 0.f;
+    if (then_groups > 1) {
+      norm_parts();
+    } else {
+      s2 = block_sum(s2, scratch);
+      inv2 = rsqrtf(s2 / (float)H + then_eps);
+    }
 #pragma unroll
     for (int k = 0; k < K; ++k) {
       const int i = first + k * step;
       if (i < H) {
         float wv[V];
         ld(then_w + i, wv);
+        if (then_groups > 1) inv2 = part_inv[i / part_size];
 #pragma unroll
         for (int j = 0; j < V; ++j) xk[k][j] *= inv2 * wv[j];
         put(i, xk[k]);
@@ -202,26 +230,34 @@ __global__ void rmsnorm_add_kernel(float* __restrict__ x, const void* a, const v
   const float inv = rsqrtf(ss / (float)H + eps);
   float s2 = 0.f;
   for (int i = first; i < H; i += step) {
-    float y[V], xv[V], wv[V];
+    float y[V], xv[V], wv[V], sq = 0.f;
     y_at(i, y);
     ld(xr + i, xv);
-    ld(w + i, wv);
+    if (w) ld(w + i, wv);
 #pragma unroll
     for (int j = 0; j < V; ++j) {
-      xv[j] += y[j] * inv * wv[j];
-      s2 += xv[j] * xv[j];
+      xv[j] += w ? y[j] * inv * wv[j] : y[j];
+      sq += xv[j] * xv[j];
     }
+    s2 += sq;
+    if (then_w && then_groups > 1) part[i / V] = sq;
     if constexpr (V == 4) store4<float>(xr + i, xv);
     else xr[i] = xv[0];
     if (out && !then_w) put(i, xv);
   }
   if (!out || !then_w) return;
-  s2 = block_sum(s2, scratch);
-  const float inv2 = rsqrtf(s2 / (float)H + then_eps);
+  float inv2 = 0.f;
+  if (then_groups > 1) {
+    norm_parts();
+  } else {
+    s2 = block_sum(s2, scratch);
+    inv2 = rsqrtf(s2 / (float)H + then_eps);
+  }
   for (int i = first; i < H; i += step) {
     float xv[V], wv[V];
     ld(xr + i, xv);  // this thread's own writes
     ld(then_w + i, wv);
+    if (then_groups > 1) inv2 = part_inv[i / part_size];
 #pragma unroll
     for (int j = 0; j < V; ++j) xv[j] *= inv2 * wv[j];
     put(i, xv);
@@ -815,25 +851,27 @@ extern "C" int lse_token_shift(const float* x, const float* mix, float* state, v
 extern "C" int lse_rmsnorm_add(float* x, const void* a, const void* b, int branch_dtype, const float* wa,
                                const float* wb, float ca, float cb, float eps_in, const float* w, float eps,
                                void* out, int out_dtype, const float* then_w, float then_eps, int T, int H,
-                               cudaStream_t stream) {
+                               cudaStream_t stream, int then_groups) {
   if (T <= 0) return LSE_OK;
-  if (!x || !a || !w || (b && !wa) || (wa && b && !wb)) return LSE_BAD_ARGUMENT;
+  if (!x || !a || (b && !wa) || (wa && b && !wb)) return LSE_BAD_ARGUMENT;
+  if (then_groups < 1 || H % then_groups) return LSE_BAD_ARGUMENT;
   if (branch_dtype != LSE_F32 && branch_dtype != LSE_FIXED64) return LSE_BAD_ARGUMENT;
   const bool sums = branch_dtype == LSE_FIXED64;
-  const size_t smem = sums ? (size_t)H * (b ? 2 : 1) * sizeof(float) : 0;
-  if (smem > 48 * 1024) return LSE_BAD_ARGUMENT;
   if (then_w && !out) return LSE_BAD_ARGUMENT;
   const int threads = H >= 2048 ? 512 : (H >= 512 ? 256 : 128);
   const bool to_bf16 = out && out_dtype == LSE_BF16;
   if (!to_bf16 && out && out_dtype != LSE_F32) return LSE_BAD_ARGUMENT;
   auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
   const bool vec = H % 4 == 0 && aligned(x) && aligned(w) && aligned(out) && aligned(wa) && aligned(wb) &&
-                   aligned(then_w) && (sums || (aligned(a) && aligned(b)));
+                   aligned(then_w) && (sums || (aligned(a) && aligned(b))) && (H / then_groups) % 4 == 0;
+  size_t smem = sums ? (size_t)H * (b ? 2 : 1) * sizeof(float) : 0;
+  if (then_w && then_groups > 1) smem += ((size_t)H / (vec ? 4 : 1) + then_groups) * sizeof(float);
+  if (smem > 48 * 1024) return LSE_BAD_ARGUMENT;
   const int per_visit = threads * (vec ? 4 : 1);
   const int visits = (H + per_visit - 1) / per_visit;  // places of the row per thread
 #define LSE_RNA_V(TO, S, V, K) \
   launch(rmsnorm_add_kernel<TO, S, V, K>, T, threads, smem, stream, x, a, b, wa, wb, ca, cb, eps_in, w, eps, \
-         (TO*)out, then_w, then_eps, H)
+         (TO*)out, then_w, then_eps, H, then_groups)
 #define LSE_RNA(TO, S) \
   do { \
     if (vec && visits == 1) LSE_RNA_V(TO, S, 4, 1); \

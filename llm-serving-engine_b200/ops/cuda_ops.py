@@ -197,20 +197,25 @@ class CudaOps:
         self.launches += 1
         return out
 
-    def add_rmsnorm(self, x, residual, weight, eps, out_dtype, rows=None):
-        """``residual`` may be a :class:`PendingSums` for ``x``: its sums are added as they are read."""
+    def add_rmsnorm(self, x, residual, weight, eps, out_dtype, rows=None, groups=1):
+        """``residual`` may be a :class:`PendingSums` for ``x`` or a :class:`DeferredProduct`: its sums
+        are added as they are read. ``groups``: a row is that many equal consecutive parts, each
+        divided by its own root mean square."""
         sums = None
+        if isinstance(residual, DeferredProduct):
+            residual = PendingSums(self, residual.sums, x)
         if isinstance(residual, PendingSums):
             if residual.into is not x:
                 raise ValueError("these pending sums belong to another tensor")
-            if rows is None and out_dtype == torch.bfloat16 and x.shape[1] % 4 == 0 and residual.sums is not None:
+            if (rows is None and out_dtype == torch.bfloat16 and (x.shape[1] // groups) % 4 == 0
+                    and residual.sums is not None):
                 sums, residual.sums = residual.sums, None
                 residual = sums
             else:  # only some rows are read here, so the whole product is added first
                 residual = residual.resolve()
         n = x.shape[0] if rows is None else rows.shape[0]
         out = torch.empty(n, x.shape[1], dtype=out_dtype, device=x.device)
-        self.ext.add_rmsnorm(x, residual, weight, float(eps), out, rows)
+        self.ext.add_rmsnorm(x, residual, weight, float(eps), out, rows, int(groups))
         self.launches += 1
         if sums is not None:
             self._sums_taken(sums)
@@ -235,13 +240,15 @@ class CudaOps:
     def _sums_taken(self, buf: torch.Tensor) -> None:
         self._sums_live.discard(buf.data_ptr())
 
-    _ACTIVATIONS = {"silu": 0, "gelu_tanh": 1}
+    _ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "clamped_glu": 2}
 
-    def silu_mul(self, gu, out_dtype=None, activation="silu"):
-        """``act(gate) * up`` of ``gu = [gate | up]``; ``activation``: silu or gelu_tanh."""
+    def silu_mul(self, gu, out_dtype=None, activation="silu", limit=0.0):
+        """``act(gate) * up`` of ``gu = [gate | up]``; ``activation``: silu or gelu_tanh, or
+        ``clamped_glu``: ``g sigmoid(1.702 g) (u + 1)`` with the gate cut at ``limit`` from above
+        and ``u`` between ``-limit`` and ``limit``."""
         out_dtype = out_dtype or gu.dtype
         out = torch.empty(gu.shape[0], gu.shape[1] // 2, dtype=out_dtype, device=gu.device)
-        self.ext.silu_mul(gu, out, self._ACTIVATIONS[activation])
+        self.ext.silu_mul(gu, out, self._ACTIVATIONS[activation], float(limit))
         self.launches += 1
         return out
 
@@ -303,17 +310,17 @@ class CudaOps:
             return torch.addmm(bias, a, w.t())  # bias added before the one rounding to bfloat16
         return torch.mm(a, w.t())
 
-    def gated_silu(self, h, w, bias=None, out_dtype=None, activation="silu"):
+    def gated_silu(self, h, w, bias=None, out_dtype=None, activation="silu", limit=0.0):
         """``act(h @ gate.T) * (h @ up.T)`` for ``w = [gate rows; up rows]``. With few bfloat16
         rows the gate meets its activation as a float32 value (the activation kernel takes the
         product's fixed-point sums); otherwise as the product's rounded output."""
         out_dtype = out_dtype or h.dtype
         if self._few_rows(h, w) and out_dtype == torch.bfloat16 and w.shape[0] % 8 == 0:
             sums = self._product_sums(h, w, bias)
-            out = self.silu_mul(sums, out_dtype=out_dtype, activation=activation)
+            out = self.silu_mul(sums, out_dtype=out_dtype, activation=activation, limit=limit)
             self._sums_taken(sums)
             return out
-        return self.silu_mul(self.linear(h, w, bias), out_dtype=out_dtype, activation=activation)
+        return self.silu_mul(self.linear(h, w, bias), out_dtype=out_dtype, activation=activation, limit=limit)
 
     def project_rope_kv_write(self, h, w, bias, *, num_heads, num_kv_heads, head_dim, positions,
                               token_seq, cos, sin, k_pages, v_pages, block_tables, page_tokens,
@@ -548,25 +555,46 @@ class CudaOps:
             return out
         return self.activation(self.linear(h, w, None, out_dtype=torch.float32), activation, out_dtype)
 
-    # ------------------------------------------------------------------ routed experts
-    _ROUTER_WEIGHTS = {"sigmoid": 0, "softmax_of_chosen": 1}
+    def poly_norm_linear(self, h, w, coef, eps, out_dtype):
+        """``a N(z) + b N(z^2) + c N(z^3) + e`` of ``z = h @ w.T`` (``coef``: float32 ``[4]``), ``N`` a
+        row divided by its root mean square. With few bfloat16 rows the product's sums are taken."""
+        out = torch.empty(h.shape[0], w.shape[0], dtype=out_dtype, device=h.device)
+        sums = None
+        if self._few_rows(h, w) and out_dtype == torch.bfloat16 and w.shape[0] % 4 == 0 and w.shape[0] <= 16384:
+            z = sums = self._product_sums(h, w, None)
+        else:
+            z = self.linear(h, w, None, out_dtype=torch.float32)
+        self.ext.poly_norm(z, coef, float(eps), out)
+        self.launches += 1
+        if sums is not None:
+            self._sums_taken(sums)
+        return out
 
-    def moe_route(self, h, router, num_experts, top, has_gate, bias=None, weights="sigmoid"):
+    # ------------------------------------------------------------------ routed experts
+    _ROUTER_WEIGHTS = {"sigmoid": 0, "softmax_of_chosen": 1, "softmax_of_all": 2}
+
+    def moe_route(self, h, router, num_experts, top, has_gate, bias=None, weights="sigmoid", groups=1, keep=1,
+                  scale=1.0):
         """Router logits (+ ``bias``) in float32; returns (the ``top`` experts with the largest
         logits ``[T, top]`` int32, their weights ``[T, top]``, the shared expert's gate ``[T]`` or
         None). ``weights``: ``sigmoid`` of each chosen logit, or ``softmax_of_chosen``: the softmax
-        over the chosen logits alone."""
+        over the chosen logits alone, or ``softmax_of_all``: scores ``s`` are the softmax over all
+        logits, ``bias`` is added to the scores for the choice only, which is limited to the
+        ``keep`` best of ``groups`` equal groups of neighbours, and a chosen expert's weight is
+        ``s / (sum of the chosen s + 1e-20) * scale``."""
         T = h.shape[0]
         idx = torch.empty(T, top, dtype=torch.int32, device=h.device)
         wts = torch.empty(T, top, dtype=torch.float32, device=h.device)
         gate = torch.empty(T, dtype=torch.float32, device=h.device) if has_gate else None
-        self.ext.moe_route(h, router, int(num_experts), int(top), idx, wts, gate, bias, self._ROUTER_WEIGHTS[weights])
+        self.ext.moe_route(h, router, int(num_experts), int(top), idx, wts, gate, bias, self._ROUTER_WEIGHTS[weights],
+                           int(groups), int(keep), float(scale))
         self.launches += 1
         return idx, wts, gate
 
     def moe_sort(self, idx, num_experts, dtype, width=0, kind=None):
         """The choices sorted by expert, as row ranges and tiles for :meth:`expert_linear`: a plan
-        that :meth:`moe_combine` reads too. ``dtype`` and ``width`` (of the experts' input) choose
+        that :meth:`moe_combine` reads too. A choice of ``num_experts`` or more is an identity
+        expert: it gets no row. ``dtype`` and ``width`` (of the experts' input) choose
         the kernel of the products: 0 the CUDA cores (float32), 2 the weight-streaming kernel (up
         to 48 choices: a few rows per expert; measured at 8 experts of 4096 x 2048, 2 per token:
         16 tokens 45 us against 55 us for the tiles, 32 tokens 72 against 58), 1 mma.sync tiles,
@@ -600,15 +628,15 @@ class CudaOps:
         self.launches += 1
         return out
 
-    def moe_combine(self, y, plan, top, shared, gate, residual, wts=None):
+    def moe_combine(self, y, plan, top, shared, gate, residual, wts=None, identity=None):
         """Per token the sum of its experts' rows of ``y``, each times its weight if ``wts``
         ``[T, top]`` is given, (+ gate * shared; no gate: + shared): added into ``residual``
-        (returns None) or returned."""
+        (returns None) or returned. ``identity`` ``[T, W]``: what an identity expert hands on."""
         work, num_experts = plan.work, plan.num_experts
         T = y.shape[0] // top
         out = residual if residual is not None else torch.empty(T, y.shape[1], dtype=torch.float32, device=y.device)
         self.ext.moe_combine(y, work, int(num_experts), int(top), shared, gate if shared is not None else None,
-                             out, residual is not None, wts)
+                             out, residual is not None, wts, identity)
         self.launches += 1
         return None if residual is not None else out
 
@@ -637,6 +665,20 @@ class CudaOps:
         cb = coefficients[1] if len(branches) == 2 else 0.0
         return branches[0], b, weights[0], wb, float(coefficients[0]), float(cb)
 
+    @staticmethod
+    def _parts_bytes(width, groups) -> int:
+        """Shared memory in which a norm of several parts per row forms their sums."""
+        if groups == 1:
+            return 0
+        return (width // (4 if (width // groups) % 4 == 0 else 1) + groups) * 4
+
+    def mix_add_rmsnorm(self, x, mix, weight, eps, out_dtype, groups=1):
+        """``x += mix`` (a ``BranchMix``: branches normed one by one and summed) and the norm of the
+        new ``x``, in one launch where the row's working space fits the kernel."""
+        if self._parts_bytes(x.shape[1], groups) > 48 * 1024:
+            return self.add_rmsnorm(x, mix.resolve(), weight, eps, out_dtype, groups=groups)
+        return self.rmsnorm_add(x, mix, None, 0.0, out_dtype, then_weight=weight, then_eps=eps, then_groups=groups)
+
     def mix_normed(self, branches, weights, coefficients, eps):
         branches = [m.resolve() if isinstance(m, DeferredProduct) else m for m in branches]
         a, b, wa, wb, ca, cb = self._two_branches(branches, weights, coefficients)
@@ -645,12 +687,12 @@ class CudaOps:
         self.launches += 1
         return out
 
-    def rmsnorm_add(self, x, branch, weight, eps, out_dtype=None, then_weight=None, then_eps=0.0):
+    def rmsnorm_add(self, x, branch, weight, eps, out_dtype=None, then_weight=None, then_eps=0.0, then_groups=1):
         """``x += weight * y / rms(y)`` with ``y`` the branch (a float32 tensor, or a
         ``BranchMix`` whose members are normed and summed in the same launch); returns the new
         ``x`` in ``out_dtype`` unless that is None. With ``then_weight`` what is returned is the
-        next norm of the new ``x``, ``then_weight * x / rms(x)`` (eps ``then_eps``), from the same
-        launch."""
+        next norm of the new ``x``, ``then_weight * x / rms(x)`` (eps ``then_eps``; of ``then_groups``
+        equal parts, each by itself), from the same launch. ``weight`` None: ``x += y``."""
         if then_weight is not None and out_dtype is None:
             raise ValueError("the norm that follows needs an output dtype")
         out = None if out_dtype is None else torch.empty(x.shape, dtype=out_dtype, device=x.device)
@@ -659,15 +701,15 @@ class CudaOps:
         # and their rows fit its shared memory; otherwise they are converted first
         deferred = [m for m in members if isinstance(m, DeferredProduct)]
         take = (len(deferred) == len(members) and all(m.sums is not None for m in deferred)
-                and x.shape[1] * len(members) * 4 <= 48 * 1024)
+                and x.shape[1] * len(members) * 4 + self._parts_bytes(x.shape[1], then_groups) <= 48 * 1024)
         tensors = [(m.sums if take else m.resolve()) if isinstance(m, DeferredProduct) else m for m in members]
         if hasattr(branch, "branches"):
             a, b, wa, wb, ca, cb = self._two_branches(tensors, branch.weights, branch.coefficients)
             self.ext.rmsnorm_add(x, a, b, wa, wb, ca, cb, float(branch.eps), weight, float(eps), out,
-                                 then_weight, float(then_eps))
+                                 then_weight, float(then_eps), int(then_groups))
         else:
             self.ext.rmsnorm_add(x, tensors[0], None, None, None, 1.0, 0.0, 0.0, weight, float(eps), out,
-                                 then_weight, float(then_eps))
+                                 then_weight, float(then_eps), int(then_groups))
         self.launches += 1
         if take:
             for m in deferred:
@@ -706,6 +748,31 @@ class CudaOps:
                                         float(key_scale), max_chunks, scratch, decay_logits, float(decay_root),
                                         float(query_scale))
         self.launches += 3 if max_chunks > 1 else 1
+        return out
+
+    # ------------------------------------------------------------------ gated delta rule
+    def delta_inputs(self, proj, col0, *, num_heads, num_kv_heads, key_dim, value_dim, conv, conv_state, A_log,
+                     dt_bias, query_scale, step):
+        """From the columns ``q | k | v | gate | b | a`` of the float32 ``proj`` (from ``col0`` on): short
+        convolution over time (``conv [taps, channels]``; ``conv_state`` keeps each request's last
+        inputs) and silu of q, k and v, unit norms of q (times ``query_scale``) and k, the decay and
+        step size. Returns ``(qkv [T, channels], scal [T, heads, 4])`` for :meth:`delta_rule`."""
+        T, C = proj.shape[0], conv.shape[1]
+        qkv = torch.empty(T, C, dtype=torch.float32, device=proj.device)
+        scal = torch.empty(T, num_heads, 4, dtype=torch.float32, device=proj.device)
+        self.ext.delta_inputs(proj, int(col0), conv, conv_state, A_log, dt_bias, step.token_seq, step.cu_q, step.ctx_lens,
+                              step.state_slots, qkv, scal, int(num_heads), int(num_kv_heads), int(key_dim),
+                              int(value_dim), float(query_scale))
+        self.launches += 1
+        return qkv, scal
+
+    def delta_rule(self, qkv, scal, *, num_heads, num_kv_heads, key_dim, value_dim, state, step):
+        """``S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q`` per head and token, from each
+        request's ``state [slots, heads, value_dim, key_dim]``; returns ``o [T, heads * value_dim]``."""
+        out = torch.empty(qkv.shape[0], num_heads * value_dim, dtype=torch.float32, device=qkv.device)
+        self.ext.delta_rule(qkv, scal, state, out, step.cu_q, step.ctx_lens, step.state_slots, int(num_heads),
+                            int(num_kv_heads), int(key_dim), int(value_dim))
+        self.launches += 1
         return out
 
     def gated_group_norm(self, o, proj, *, gate_offset, group, weight, eps, gate_activation, out_dtype):
@@ -757,8 +824,8 @@ class CudaOps:
     # ------------------------------------------------------------------ rows of q, k, v prepared a token at a time
     def qkv_norm_rope_write(self, qkv, *, num_heads, num_kv_heads, num_value_heads, head_dim, value_dim, out_dim,
                             q_weight, k_weight, eps, positions, token_seq, cos, sin, k_pages, v_pages,
-                            block_tables, page_tokens, out_dtype, temp_coef=0.0, temp_every=0):
-        """Of the float32 projection ``qkv`` (query heads, key heads, then ``num_value_heads`` value
+                            block_tables, page_tokens, out_dtype, temp_coef=0.0, temp_every=0, col0=0):
+        """Of the float32 projection ``qkv`` (from column ``col0``: query heads, key heads, then ``num_value_heads`` value
         heads; 0: a key head's value is its key as projected): RMS norm over all of a token's
         query values and over all of its key values (if weights of those sizes are given), a query
         factor ``1 + temp_coef * ln((pos + 1) // temp_every + 1)``, rotation of the first dims of
@@ -769,7 +836,7 @@ class CudaOps:
         self.ext.qkv_norm_rope_write(qkv, q, int(num_heads), int(num_kv_heads), int(num_value_heads), int(head_dim),
                                      int(value_dim), int(out_dim), q_weight, k_weight, float(eps), float(temp_coef),
                                      int(temp_every), positions, token_seq, cos, sin, k_pages, v_pages,
-                                     block_tables, int(page_tokens))
+                                     block_tables, int(page_tokens), int(col0))
         self.launches += 1
         return q
 

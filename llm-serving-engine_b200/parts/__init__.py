@@ -1,6 +1,6 @@
 """Parts a model is assembled from. Importing this package registers the built-in kinds."""
 
-from . import (attention, blocks, embed_terms, feed_forward, latent_attention, linear_attention, moe, norms,  # noqa: F401
+from . import (attention, blocks, delta_rule, embed_terms, feed_forward, latent_attention, linear_attention, moe, norms,  # noqa: F401
                parallel, positions, token_shift)
 from .attention import AttentionSpec, PagedAttention
 from .base import (
@@ -25,6 +25,7 @@ from .base import (
 from .blocks import BranchNormBlock, BranchNormBlockSpec, PreNormBlock, PreNormBlockSpec, SandwichBlock, SandwichBlockSpec
 from .linear_attention import (DecayLinearAttention, DecayLinearAttentionSpec, GatedLinearAttention,
                                GatedLinearAttentionSpec)
+from .delta_rule import GatedDeltaRule, GatedDeltaRuleSpec
 from .differential_attention import DifferentialAttention, DifferentialAttentionSpec
 from .streams import StreamsBlock, StreamsBlockSpec, StreamsRMSNorm, StreamsRMSNormSpec, StreamsWrite, StreamsWriteSpec
 from .parallel import ParallelMixer, ParallelMixerSpec
@@ -47,4 +48,5 @@ __all__ = [
     "RoutedExperts", "RoutedExpertsSpec", "SinusoidSpec", "SandwichBlock", "SandwichBlockSpec", "MLP", "MLPSpec",
     "GatedLinearAttention", "GatedLinearAttentionSpec", "DifferentialAttention", "DifferentialAttentionSpec",
     "StreamsBlock", "StreamsBlockSpec", "StreamsRMSNorm", "StreamsRMSNormSpec", "StreamsWrite", "StreamsWriteSpec",
+    "GatedDeltaRule", "GatedDeltaRuleSpec",
 ]

@@ -37,6 +37,9 @@ Further options of the spec, all off by default:
 * ``sinks``: a learned number per query head whose exponential joins the softmax's denominator
   without a key or a value.
 
+A rotation that pairs neighbouring dims (``RotarySpec.pairing``) becomes one of halves by an order of
+each query and key head's rows that is applied when the weights are bound.
+
 A position encoding whose tables cover fewer dims than the head size rotates the first of each
 head's dims (pairs ``(i, i + rotated/2)``) and passes the rest. That, and the norm over whole rows,
 are served by the kernel set's ``qkv_norm_rope_write``, which also fills a head up to the kernels'
@@ -51,6 +54,7 @@ from typing import Any
 import torch
 
 from .base import MIXERS, POSITION_ENCODINGS, Mixer, PagedKVNeed, ParamDecl, project_into
+from .positions import neighbours_to_halves
 
 
 def rows_to_whole_vectors(w, multiple: int = 8):
@@ -113,16 +117,21 @@ class PagedAttention(Mixer):
         self.rot_dims = 2 * self.rotary[0].shape[1] if self.rotary is not None else 0
         if self.rot_dims > spec.head_dim:
             raise ValueError("attention: more rotated dims than the head size")
-        # whole-row norms and partly rotated heads go through the kernel that prepares a token's rows at once
+        # whole-row norms, partly rotated heads, and any heads without a norm per head that the plain path does not
+        # serve, go through the kernel that prepares a token's rows at once
+        options = (spec.values_are_keys or spec.head_temperature or spec.distance_slopes is not None or spec.chunk > 0
+                   or self.value_dim != spec.head_dim or spec.gate == "head" or spec.sinks or spec.head_dim % 16 != 0)
         self.by_rows = ((spec.qk_norm_scope == "row" and spec.qk_norm_eps is not None)
-                        or (self.rotary is not None and self.rot_dims != spec.head_dim))
+                        or (self.rotary is not None and self.rot_dims != spec.head_dim)
+                        or (spec.qk_norm_eps is None and options and not spec.bias and not spec.keep_first
+                            and spec.gate != "element"))
         if self.by_rows and (spec.bias or spec.gate == "element" or spec.keep_first):
             raise NotImplementedError("attention: whole-row norm or a partly rotated head with bias, element gate or kept keys")
         # the plain path (fused projection, rotation, cache write and attention) serves none of these
         self.extended = (spec.qk_norm_eps is not None or spec.values_are_keys or spec.head_temperature
                          or spec.distance_slopes is not None or spec.chunk > 0
                          or self.value_dim != spec.head_dim or spec.keep_first > 0 or spec.gate != "none"
-                         or spec.sinks or self.by_rows)
+                         or spec.sinks or spec.head_dim % 16 != 0 or self.by_rows)
         # The attention kernels take head sizes that are multiples of 16. With the score options on,
         # any other head size is padded with zeros up to the next one when the weights are bound:
         # zero dims change no dot product, the norm divides by the true size, and the padded dims
@@ -170,6 +179,8 @@ class PagedAttention(Mixer):
         self.temperature = params.get("temperature")
         self.sinks = params.get("sinks")
         s = self.spec
+        if self.rotary is not None and getattr(s.position, "pairing", "halves") == "neighbours":
+            self._pair_halves()
         if s.qk_norm_eps is not None and not s.qk_norm_weight:  # the kernel's norm multiplies by a weight: ones
             row = s.qk_norm_scope == "row"
             self.q_norm_weight = torch.ones(self.q_size if row else s.head_dim, dtype=torch.float32, device=self.env.device)
@@ -185,6 +196,23 @@ class PagedAttention(Mixer):
             self.qkv_bias = torch.cat([self.qkv_bias, self.qkv_bias.new_zeros(self.gate_size)])
         if self.kernel_dim != s.head_dim or self.kernel_dim != self.value_dim:
             self._pad_heads()
+
+    def _pair_halves(self):
+        """Reorder every query and key head's rows so that rotated neighbours lie half a rotation apart."""
+        s, D = self.spec, self.spec.head_dim
+        if s.values_are_keys:
+            raise NotImplementedError("attention: neighbouring dims rotated in keys that are also the values")
+        order = torch.tensor(neighbours_to_halves(D, self.rot_dims), device=self.qkv_weight.device)
+        heads = torch.arange(s.num_heads + s.num_kv_heads, device=order.device)[:, None] * D + order[None, :]
+        rows = torch.cat([heads.reshape(-1), torch.arange(heads.numel(), self.qkv_weight.shape[0], device=order.device)])
+        self.qkv_weight = self.qkv_weight[rows].contiguous()
+        if self.qkv_bias is not None:
+            self.qkv_bias = self.qkv_bias[rows[: self.qkv_bias.shape[0]]].contiguous()
+        if self.q_norm_weight is not None:
+            n = heads.reshape(-1)
+            per_row = s.qk_norm_scope == "row"
+            self.q_norm_weight = self.q_norm_weight[n[: self.q_size] if per_row else order].contiguous()
+            self.k_norm_weight = self.k_norm_weight[n[: self.kv_size] if per_row else order].contiguous()
 
     def _pad_heads(self):
         """Every head's rows of q, k and v (and of a gate per element) filled up with zero rows to
@@ -219,7 +247,9 @@ class PagedAttention(Mixer):
     # what the cache manager has to keep for a layer of this kind
     def cache_need(self):
         s = self.spec
-        return PagedKVNeed(s.num_kv_heads, self.kernel_dim, s.window, keep_first=s.keep_first)
+        # no key before the query's chunk is read again: a chunk bounds what is kept as a window does
+        window = min(w for w in (s.window, s.chunk) if w > 0) if s.window or s.chunk else 0
+        return PagedKVNeed(s.num_kv_heads, self.kernel_dim, window, keep_first=s.keep_first)
 
     def reserve(self, max_seqs: int) -> None:
         """Allocate kernel scratch for up to ``max_seqs`` single-token sequences in a step."""
@@ -243,6 +273,22 @@ class PagedAttention(Mixer):
 
     accepts_residual = True
     accepts_deferral = True
+
+    @property
+    def input_weight(self):
+        """The matrix of this mixer's product with its input, where a mixer of several branches may
+        make it part of a larger one (``forward_projected``)."""
+        return self.qkv_weight if self.by_rows else None
+
+    @input_weight.setter
+    def input_weight(self, w):
+        self.qkv_weight = w
+
+    def forward_projected(self, proj, col0, step, cache, may_defer=False):
+        """As ``forward`` from the float32 product with the input, whose columns for this mixer start at ``col0``."""
+        cos, sin = self.rotary if self.rotary is not None else (None, None)
+        o = self._by_rows(proj, step, cache, step.block_tables[cache.group], cos, sin, col0)
+        return project_into(self.ops, o, self.o_weight, self.o_bias, self.env.residual_dtype, None, may_defer)
 
     def forward(self, h, step, cache, residual=None, may_defer=False):
         s = self.spec
@@ -300,12 +346,12 @@ class PagedAttention(Mixer):
             ops.sigmoid_gate_mul(o, qkv, col0, 1 if s.gate == "element" else self.kernel_dim)
         return o
 
-    def _by_rows(self, qkv, step, cache, tables, cos, sin):
+    def _by_rows(self, qkv, step, cache, tables, cos, sin, col0=0):
         """The same three or four launches with the kernel that prepares all rows of a token."""
         s, ops = self.spec, self.ops
         normed = s.qk_norm_eps is not None
         q = ops.qkv_norm_rope_write(
-            qkv, num_heads=s.num_heads, num_kv_heads=s.num_kv_heads,
+            qkv, col0=col0, num_heads=s.num_heads, num_kv_heads=s.num_kv_heads,
             num_value_heads=0 if s.values_are_keys else s.num_kv_heads, head_dim=s.head_dim,
             value_dim=self.value_dim, out_dim=self.kernel_dim,
             q_weight=self.q_norm_weight if normed else None, k_weight=self.k_norm_weight if normed else None,
@@ -319,6 +365,6 @@ class PagedAttention(Mixer):
             page_tokens=cache.page_tokens, step=step, plan=step.plans[self.plan_key()],
             head_scale=self.temperature, slopes=self.slopes, chunk=s.chunk, sinks=self.sinks)
         if s.gate == "head":  # one gate column per head, behind q, k (and v)
-            col0 = self.q_size + self.kv_size + self.v_size
-            ops.sigmoid_gate_mul(o, qkv, col0, self.kernel_dim)
+            gate0 = col0 + self.q_size + self.kv_size + self.v_size
+            ops.sigmoid_gate_mul(o, qkv, gate0, self.kernel_dim)
         return o

@@ -61,6 +61,8 @@ class PreNormBlock(Block):
         h = self.norm_in.forward(x, settle(pending, self.norm_in))
         if getattr(self.mixer, "accepts_residual", False):
             a = self.mixer.forward(h, step, cache, residual=x, may_defer=True)  # None: already added into x
+        elif getattr(self.mixer, "accepts_deferral", False) and getattr(self.ops, "defers_adds", False):
+            a = self.mixer.forward(h, step, cache, may_defer=True)  # may be a product or a sum not formed yet
         else:
             a = self.mixer.forward(h, step, cache)
         if self.feed_forward is None:

@@ -6,8 +6,13 @@
 
 No biases. The activation is computed in float32 (src/llmserve/kernels/csrc/fused_ops.cpp:75-91).
 
+``activation="clamped_glu"`` combines the two halves otherwise: ``g sigmoid(1.702 g) (u + 1)`` with ``g =
+min(gate, limit)`` and ``u = clamp(up, -limit, limit)``.
+
 ``mlp`` is the ungated form, ``y = Wdown act(Wup h)``, with ``act`` one of ``relu2`` (the square of
-relu), ``relu``, ``gelu_tanh``, ``silu``.
+relu), ``relu``, ``gelu_tanh``, ``silu``, or ``poly_norm``: with four learned numbers a, b, c, e,
+``a N(z) + b N(z^2) + c N(z^3) + e``, powers taken element by element and ``N`` a token's whole vector
+divided by its root mean square (``eps`` of the spec), in float32.
 """
 
 from __future__ import annotations
@@ -17,12 +22,16 @@ from dataclasses import dataclass
 from .base import FEED_FORWARDS, FeedForward, ParamDecl, project_into
 
 
+GATED_ACTIVATIONS = ("silu", "gelu_tanh", "clamped_glu")
+
+
 @dataclass(frozen=True)
 class SwiGLUSpec:
     hidden_size: int
     intermediate_size: int
     kind: str = "swiglu"
-    activation: str = "silu"  # or "gelu_tanh"
+    activation: str = "silu"  # or "gelu_tanh", "clamped_glu"
+    limit: float = 0.0  # of clamped_glu
 
 
 @FEED_FORWARDS.register("swiglu")
@@ -36,8 +45,9 @@ class SwiGLU(FeedForward):
 
     def __init__(self, spec: SwiGLUSpec, env) -> None:
         super().__init__(spec, env)
-        if spec.activation not in ("silu", "gelu_tanh"):
+        if spec.activation not in GATED_ACTIVATIONS:
             raise ValueError(f"gated feed-forward: activation {spec.activation!r} is not known")
+        self._options = {} if spec.activation != "clamped_glu" else {"limit": spec.limit}
 
     def bind(self, params):
         self.gate_up_weight = params["gate_up.weight"]
@@ -51,7 +61,7 @@ class SwiGLU(FeedForward):
             a = ops.gated_silu(h, self.gate_up_weight, None, out_dtype=self.env.dtype)
         else:
             a = ops.gated_silu(h, self.gate_up_weight, None, out_dtype=self.env.dtype,
-                               activation=self.spec.activation)
+                               activation=self.spec.activation, **self._options)
         return project_into(ops, a, self.down_weight, None, self.env.residual_dtype, residual, may_defer)
 
 
@@ -62,7 +72,8 @@ PLAIN_ACTIVATIONS = ("relu2", "relu", "gelu_tanh", "silu")
 class MLPSpec:
     hidden_size: int
     intermediate_size: int
-    activation: str = "relu2"
+    activation: str = "relu2"  # or another of PLAIN_ACTIVATIONS, or "poly_norm"
+    eps: float = 0.0  # of poly_norm
     kind: str = "mlp"
 
 
@@ -72,20 +83,27 @@ class MLP(FeedForward):
 
     def __init__(self, spec: MLPSpec, env) -> None:
         super().__init__(spec, env)
-        if spec.activation not in PLAIN_ACTIVATIONS:
+        if spec.activation not in PLAIN_ACTIVATIONS + ("poly_norm",):
             raise ValueError(f"feed-forward: activation {spec.activation!r} is not known")
 
     def param_decls(self):
         s = self.spec
-        return {
+        decls = {
             "up.weight": ParamDecl((s.intermediate_size, s.hidden_size), "matrix"),
             "down.weight": ParamDecl((s.hidden_size, s.intermediate_size), "matrix"),
         }
+        if s.activation == "poly_norm":
+            decls["coefficients"] = ParamDecl((4,), "scale")
+        return decls
 
     def bind(self, params):
         self.up_weight = params["up.weight"]
         self.down_weight = params["down.weight"]
+        self.coefficients = params.get("coefficients")
 
     def forward(self, h, step, residual=None, may_defer=False):
-        a = self.ops.activated_linear(h, self.up_weight, self.spec.activation, self.env.dtype)
+        if self.spec.activation == "poly_norm":
+            a = self.ops.poly_norm_linear(h, self.up_weight, self.coefficients, self.spec.eps, self.env.dtype)
+        else:
+            a = self.ops.activated_linear(h, self.up_weight, self.spec.activation, self.env.dtype)
         return project_into(self.ops, a, self.down_weight, None, self.env.residual_dtype, residual, may_defer)

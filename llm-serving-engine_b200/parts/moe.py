@@ -16,7 +16,15 @@ Options of the spec:
   differ whenever the expert is not linear in its input);
 * ``gated=False``: an expert is ``Wdown act(Wup z)`` with ``act`` a plain activation (``relu2``:
   the square of relu), and so is the shared expert;
-* ``shared_gate=False``: the shared expert is added as it is, without a sigmoid gate.
+* ``shared_gate=False``: the shared expert is added as it is, without a sigmoid gate;
+* ``router_weights="softmax_of_all"``: scores are the softmax over all of the router's logits; with
+  ``correction`` a learned number per expert is added to the scores for the choice alone; the
+  experts form ``groups`` equal groups of neighbours, of which only the ``keep_groups`` with the
+  largest choice scores in them can be chosen from; the weights are the chosen experts' scores
+  divided by their sum (+ 1e-20) and multiplied by ``router_scale``;
+* ``identity_experts``: the last rows of the router stand for experts whose output is their input;
+  they have no matrices and take part in the softmax, the groups and the choice like the others;
+* ``activation="clamped_glu"`` with ``limit`` (``shared_limit``: the shared expert's).
 
 The tokens' choices are sorted by expert on the device and the experts' products run as one
 launch over tiles of rows that belong to one expert each, so nothing comes back to the host
@@ -28,7 +36,7 @@ from __future__ import annotations
 from dataclasses import dataclass
 
 from .base import FEED_FORWARDS, FeedForward, ParamDecl
-from .feed_forward import PLAIN_ACTIVATIONS, MLPSpec, SwiGLUSpec
+from .feed_forward import GATED_ACTIVATIONS, PLAIN_ACTIVATIONS, MLPSpec, SwiGLUSpec
 
 
 @dataclass(frozen=True)
@@ -44,6 +52,13 @@ class RoutedExpertsSpec:
     weight_on: str = "input"  # or "output"
     gated: bool = True
     shared_gate: bool = True
+    correction: bool = False  # softmax_of_all: a learned number per expert, part of the choice only
+    groups: int = 1
+    keep_groups: int = 1
+    router_scale: float = 1.0
+    identity_experts: int = 0
+    limit: float = 0.0
+    shared_limit: float = 0.0
     kind: str = "routed_experts"
 
 
@@ -53,15 +68,27 @@ class RoutedExperts(FeedForward):
 
     def __init__(self, spec: RoutedExpertsSpec, env) -> None:
         super().__init__(spec, env)
-        if not 1 <= spec.top <= spec.num_experts:
+        self.choices = spec.num_experts + spec.identity_experts  # what the router chooses from
+        if not 1 <= spec.top <= self.choices:
             raise ValueError("routed_experts: top must lie between 1 and the number of experts")
-        if spec.router_weights not in ("sigmoid", "softmax_of_chosen") or spec.weight_on not in ("input", "output"):
+        self.of_all = spec.router_weights == "softmax_of_all"
+        if (spec.correction or spec.groups != 1 or spec.router_scale != 1.0 or spec.identity_experts) and not self.of_all:
+            raise ValueError("routed_experts: correction, groups, scale and identity experts go with softmax_of_all")
+        if self.of_all and (spec.router_bias or spec.weight_on != "output" or self.choices % spec.groups
+                            or not 1 <= spec.keep_groups <= spec.groups
+                            or spec.top > spec.keep_groups * (self.choices // spec.groups)):
+            raise ValueError("routed_experts: groups must be equal, and those kept hold at least top experts")
+        if spec.router_weights not in ("sigmoid", "softmax_of_chosen", "softmax_of_all") or spec.weight_on not in ("input", "output"):
             raise ValueError("routed_experts: unknown kind of router weights or of their place")
         if not spec.gated and spec.activation not in PLAIN_ACTIVATIONS:
             raise ValueError(f"routed_experts: activation {spec.activation!r} is not known for ungated experts")
+        if spec.gated and spec.activation not in GATED_ACTIVATIONS:
+            raise ValueError(f"routed_experts: activation {spec.activation!r} is not known for gated experts")
+        self._options = {} if spec.activation != "clamped_glu" else {"limit": spec.limit}
         self.children = {}
         if spec.shared_size:
-            shared = (SwiGLUSpec(spec.hidden_size, spec.shared_size, activation=spec.activation) if spec.gated
+            shared = (SwiGLUSpec(spec.hidden_size, spec.shared_size, activation=spec.activation, limit=spec.shared_limit)
+                      if spec.gated
                       else MLPSpec(spec.hidden_size, spec.shared_size, activation=spec.activation))
             self.children["shared"] = FEED_FORWARDS.build(shared, env)
         self.shared = self.children.get("shared")
@@ -71,7 +98,7 @@ class RoutedExperts(FeedForward):
         s = self.spec
         decls = {
             # one more row with a shared expert: its gate
-            "router.weight": ParamDecl((s.num_experts + (1 if self.has_gate else 0), s.hidden_size), "matrix32"),
+            "router.weight": ParamDecl((self.choices + (1 if self.has_gate else 0), s.hidden_size), "matrix32"),
             "experts.down.weight": ParamDecl((s.num_experts * s.hidden_size, s.expert_size), "matrix"),
         }
         if s.gated:
@@ -80,6 +107,8 @@ class RoutedExperts(FeedForward):
             decls["experts.up.weight"] = ParamDecl((s.num_experts * s.expert_size, s.hidden_size), "matrix")
         if s.router_bias:
             decls["router.bias"] = ParamDecl((s.num_experts,), "offset")
+        if s.correction:
+            decls["router.correction"] = ParamDecl((self.choices,), "offset")
         if self.shared is not None:
             for name, decl in self.shared.param_decls().items():
                 decls["shared." + name] = decl
@@ -89,6 +118,7 @@ class RoutedExperts(FeedForward):
         s = self.spec
         self.router_weight = params["router.weight"]
         self.router_bias = params.get("router.bias")
+        self.correction = params.get("router.correction")
         rows = 2 * s.expert_size if s.gated else s.expert_size
         self.gate_up_weight = params["experts.gate_up.weight" if s.gated else "experts.up.weight"].view(
             s.num_experts, rows, s.hidden_size)
@@ -98,7 +128,11 @@ class RoutedExperts(FeedForward):
 
     def forward(self, h, step, residual=None, may_defer=False):
         s, ops = self.spec, self.ops
-        if s.router_bias or s.router_weights != "sigmoid":
+        if self.of_all:
+            idx, wts, gate = ops.moe_route(h, self.router_weight, self.choices, s.top, self.has_gate,
+                                           bias=self.correction, weights=s.router_weights, groups=s.groups,
+                                           keep=s.keep_groups, scale=s.router_scale)
+        elif s.router_bias or s.router_weights != "sigmoid":
             idx, wts, gate = ops.moe_route(h, self.router_weight, s.num_experts, s.top, self.has_gate,
                                            bias=self.router_bias, weights=s.router_weights)
         else:
@@ -107,7 +141,7 @@ class RoutedExperts(FeedForward):
         on_input = s.weight_on == "input"
         gu = ops.expert_linear(h, self.gate_up_weight, plan, top=s.top, wts=wts if on_input else None)
         if s.gated:
-            a = ops.silu_mul(gu, out_dtype=self.env.dtype, activation=s.activation)
+            a = ops.silu_mul(gu, out_dtype=self.env.dtype, activation=s.activation, **self._options)
         else:
             a = ops.activation(gu, s.activation, self.env.dtype)
         y = ops.expert_linear(a, self.down_weight, plan)
@@ -116,6 +150,8 @@ class RoutedExperts(FeedForward):
             shared = shared.resolve()
         if on_input and self.has_gate == (shared is not None):
             return ops.moe_combine(y, plan, s.top, shared, gate, residual)
+        if s.identity_experts:
+            return ops.moe_combine(y, plan, s.top, shared, gate, residual, wts=wts, identity=h)
         return ops.moe_combine(y, plan, s.top, shared, gate, residual, wts=None if on_input else wts)
 
 

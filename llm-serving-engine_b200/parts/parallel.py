@@ -3,6 +3,9 @@ and summed with fixed coefficients.
 
     out = sum_b coefficient_b * w_b * a_b / sqrt(mean(a_b^2) + eps),      a_b = branch_b(h)
 
+Branches that can start from a product made for them (``input_weight``, ``forward_projected``) share
+one: their matrices are laid one below the other when the weights are bound.
+
 Each branch is a mixer of its own kind with its own cache need; the cache layer of the block holds
 all of them (pages for one, states for others), and each branch sees its own part of it.
 """
@@ -11,6 +14,8 @@ from __future__ import annotations
 
 from dataclasses import dataclass
 from typing import Any
+
+import torch
 
 from .base import MIXERS, BranchMix, Mixer, ParamDecl, count_states, flatten_needs, has_pages
 
@@ -55,6 +60,25 @@ class ParallelMixer(Mixer):
             prefix = name + "."
             child.bind({k[len(prefix):]: v for k, v in params.items() if k.startswith(prefix)})
             self.out_weights.append(params[f"out.{name}.weight"])
+        self._share_product()
+
+    def _share_product(self):
+        """One product with the input for all branches, if every branch can take its columns of it.
+        Every branch starts on a column that is a multiple of 8; what the branches hold of their
+        own becomes a view of the shared matrix."""
+        self.shared_weight = None
+        weights = [getattr(b, "input_weight", None) for b in self.branches]
+        if len(weights) < 2 or any(w is None for w in weights):
+            return
+        padded, self.columns, at = [], [], 0
+        for w in weights:
+            self.columns.append(at)
+            extra = (-w.shape[0]) % 8
+            padded += [w] + ([w.new_zeros(extra, w.shape[1])] if extra else [])
+            at += w.shape[0] + extra
+        self.shared_weight = torch.cat(padded, 0).contiguous()
+        for b, w, c in zip(self.branches, weights, self.columns):
+            b.input_weight = self.shared_weight[c : c + w.shape[0]]
 
     def cache_need(self):
         return tuple(n for b in self.branches for n in flatten_needs(b.cache_need()))
@@ -63,6 +87,11 @@ class ParallelMixer(Mixer):
 
     def forward(self, h, step, cache, may_defer=False):
         outs = []
+        if self.shared_weight is not None:
+            proj = self.ops.linear(h, self.shared_weight, None, out_dtype=torch.float32)
+            for b, c, (pages, first, n) in zip(self.branches, self.columns, self._parts):
+                outs.append(b.forward_projected(proj, c, step, cache.part(pages, first, n), may_defer=may_defer))
+            return BranchMix(self.ops, outs, self.out_weights, tuple(self.spec.coefficients), self.spec.eps)
         for b, (pages, first, n) in zip(self.branches, self._parts):
             defer = may_defer and getattr(b, "accepts_deferral", False)
             a = (b.forward(h, step, cache.part(pages, first, n), may_defer=True) if defer

@@ -15,6 +15,10 @@ both tables are multiplied by ``0.1 ln(factor) + 1``.
 ``head_dim`` is the number of rotated dims: a mixer whose heads are larger rotates the first
 ``head_dim`` dims of each head (pairs ``(i, i + head_dim/2)``) and passes the rest.
 
+``pairing="neighbours"``: the pairs are ``(2i, 2i + 1)`` instead. The tables are the same; the mixer
+reorders the rows of its query and key projections once (evens, then odds, then the rest), which
+leaves every product of a query and a key as it is.
+
 ``none``: no position information (for mixers that carry order in their own state).
 
 ``sinusoid``: an absolute encoding added to the embedded tokens: entry 2i of the vector of
@@ -44,6 +48,7 @@ class RotarySpec:
     original_max_positions: int = 0
     yarn_fast: float = 32.0  # turns over the original length above which a pair keeps its frequency
     yarn_slow: float = 1.0  # turns below which a pair is stretched by the whole factor
+    pairing: str = "halves"  # "neighbours": dim 2i is paired with dim 2i + 1
     kind: str = "rope"
 
 
@@ -88,12 +93,20 @@ def rotary_inverse_frequencies(spec: RotarySpec) -> torch.Tensor:
     return inv
 
 
+def neighbours_to_halves(head_dim: int, rotated: int) -> list[int]:
+    """Order of a head's dims in which the pairs (2i, 2i + 1) of its first ``rotated`` dims lie as
+    (i, i + rotated / 2)."""
+    return [*range(0, rotated, 2), *range(1, rotated, 2), *range(rotated, head_dim)]
+
+
 @POSITION_ENCODINGS.register("rope")
 class RotaryPositionEncoding(PositionEncoding):
     def __init__(self, spec: RotarySpec, env) -> None:
         super().__init__(spec, env)
         if spec.head_dim % 2:
             raise ValueError(f"rotary positions need an even head size, got {spec.head_dim}")
+        if spec.pairing not in ("halves", "neighbours"):
+            raise ValueError(f"rotary positions: pairing {spec.pairing!r} is not known")
         inv = rotary_inverse_frequencies(spec)
         ang = torch.outer(torch.arange(env.max_positions, dtype=torch.float64), inv)
         mag = rotary_table_factor(spec)

@@ -49,7 +49,7 @@ class PlainOps:
     def embedding(self, token_ids, table):
         return table[token_ids.long()].float()
 
-    def add_rmsnorm(self, x, residual, weight, eps, out_dtype, rows=None):
+    def add_rmsnorm(self, x, residual, weight, eps, out_dtype, rows=None, groups=1):
         if rows is not None:
             v = x[rows.long()]
             if residual is not None:
@@ -58,11 +58,23 @@ class PlainOps:
             if residual is not None:
                 x += residual.float()
             v = x
-        y = v * torch.rsqrt(v.pow(2).mean(-1, keepdim=True) + eps) * weight
+        p = v.reshape(v.shape[0], groups, -1)
+        y = (p * torch.rsqrt(p.pow(2).mean(-1, keepdim=True) + eps)).reshape(v.shape) * weight
         return y.to(out_dtype)
 
-    def silu_mul(self, gu, out_dtype=None, activation="silu"):
+    def mix_add_rmsnorm(self, x, mix, weight, eps, out_dtype, groups=1):
+        return self.add_rmsnorm(x, mix.resolve(), weight, eps, out_dtype, groups=groups)
+
+    def poly_norm_linear(self, h, w, coef, eps, out_dtype):
+        z = self.linear(h, w, None, out_dtype=torch.float32)
+        n = lambda y: y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps)
+        return (coef[0] * n(z) + coef[1] * n(z ** 2) + coef[2] * n(z ** 3) + coef[3]).to(out_dtype)
+
+    def silu_mul(self, gu, out_dtype=None, activation="silu", limit=0.0):
         g, u = gu.float().chunk(2, dim=-1)
+        if activation == "clamped_glu":
+            g, u = g.clamp(max=limit), u.clamp(-limit, limit)
+            return (g * torch.sigmoid(1.702 * g) * (u + 1)).to(out_dtype or gu.dtype)
         if activation == "gelu_tanh":
             act = 0.5 * g * (1 + torch.tanh(0.7978845608028654 * (g + 0.044715 * g ** 3)))
         else:
@@ -78,9 +90,9 @@ class PlainOps:
             return None
         return y.to(out_dtype or a.dtype)
 
-    def gated_silu(self, h, w, bias=None, out_dtype=None, activation="silu"):
+    def gated_silu(self, h, w, bias=None, out_dtype=None, activation="silu", limit=0.0):
         return self.silu_mul(self.linear(h, w, bias, out_dtype=torch.float32), out_dtype=out_dtype or h.dtype,
-                             activation=activation)
+                             activation=activation, limit=limit)
 
     # ------------------------------------------------------------------ attention
     def project_rope_kv_write(self, h, w, bias, *, out_dtype=None, **kw):
@@ -292,26 +304,40 @@ class PlainOps:
         return self.activation(self.linear(h, w, None, out_dtype=torch.float32), activation, out_dtype)
 
     # ------------------------------------------------------------------ routed experts
-    def moe_route(self, h, router, num_experts, top, has_gate, bias=None, weights="sigmoid"):
+    def moe_route(self, h, router, num_experts, top, has_gate, bias=None, weights="sigmoid", groups=1, keep=1,
+                  scale=1.0):
         z = h.float() @ router.float().T
         gate = torch.sigmoid(z[:, num_experts]) if has_gate else None
+        if weights == "softmax_of_all":
+            s = torch.softmax(z[:, :num_experts], -1)
+            c = s + (bias.float() if bias is not None else 0.0)
+            per = c.view(-1, groups, num_experts // groups)
+            best = torch.topk(per.max(-1).values, keep, dim=-1).indices
+            kept = torch.zeros(per.shape[:2], dtype=torch.bool).scatter_(1, best, True)
+            c = per.masked_fill(~kept[:, :, None], float("-inf")).view(-1, num_experts)
+            idx = torch.topk(c, top, dim=-1).indices
+            val = s.gather(1, idx)
+            return idx.to(torch.int32), val / (val.sum(-1, keepdim=True) + 1e-20) * scale, gate
         z = z[:, :num_experts] + (bias.float() if bias is not None else 0.0)
         val, idx = torch.topk(z, top, dim=-1)
         val = torch.sigmoid(val) if weights == "sigmoid" else torch.softmax(val, dim=-1)
         return idx.to(torch.int32), val, gate
 
     def moe_sort(self, idx, num_experts, dtype, width=0, kind=None):
+        self.num_real_experts = num_experts
         return idx  # the plain products below walk the choices as they are
 
     def expert_linear(self, a, w, plan, top=0, wts=None):
-        idx = plan.reshape(-1).long()
+        idx = plan.reshape(-1).long().clamp(max=w.shape[0] - 1)  # (an identity expert's row is not used)
         rows = a.float() if top == 0 else a.float().repeat_interleave(top, 0)
         if wts is not None:
             rows = rows * wts.reshape(-1, 1)
         return torch.einsum("rk,rnk->rn", rows, w.float()[idx])
 
-    def moe_combine(self, y, plan, top, shared, gate, residual, wts=None):
+    def moe_combine(self, y, plan, top, shared, gate, residual, wts=None, identity=None):
         rows = y.view(-1, top, y.shape[1])
+        if identity is not None:
+            rows = torch.where((plan >= self.num_real_experts)[:, :, None], identity.float()[:, None, :], rows)
         out = (rows * wts[:, :, None]).sum(1) if wts is not None else rows.sum(1)
         if shared is not None:
             out = out + (gate[:, None] * shared.float() if gate is not None else shared.float())
@@ -385,6 +411,54 @@ class PlainOps:
             state[slots[s_]] = S
         return out.reshape(T, H * dv)
 
+    def delta_inputs(self, proj, col0, *, num_heads, num_kv_heads, key_dim, value_dim, conv, conv_state, A_log,
+                     dt_bias, query_scale, step):
+        H, G, dk, dv, C = num_heads, num_kv_heads, key_dim, value_dim, conv.shape[1]
+        past = conv.shape[0] - 1
+        cu, ctx, slots = step.cu_q.tolist(), step.ctx_lens.tolist(), step.state_slots.tolist()
+        x = proj[:, col0 : col0 + C].float()
+        y = torch.zeros_like(x)
+        for s_ in range(len(ctx)):
+            a, b = cu[s_], cu[s_ + 1]
+            if past and ctx[s_] - (b - a) > 0:
+                before = conv_state[slots[s_]].clone()
+            else:
+                before = torch.zeros(past, C)
+            seen = torch.cat([before, x[a:b]], 0)
+            for j in range(past + 1):
+                y[a:b] += conv[j] * seen[j : j + b - a]
+            if past:
+                conv_state[slots[s_]] = seen[seen.shape[0] - past :]
+        y = y / (1 + torch.exp(-y))
+        T = proj.shape[0]
+        unit = lambda t: t / torch.sqrt(t.pow(2).sum(-1, keepdim=True) + 1e-6)
+        q = unit(y[:, : G * dk].view(T, G, dk)) * query_scale
+        k = unit(y[:, G * dk : 2 * G * dk].view(T, G, dk))
+        b0 = col0 + C + H * dv
+        g = torch.exp(-torch.exp(A_log) * torch.nn.functional.softplus(proj[:, b0 + H : b0 + 2 * H].float() + dt_bias))
+        beta = torch.sigmoid(proj[:, b0 : b0 + H].float())
+        qk = (q * k).sum(-1).repeat_interleave(H // G, 1)
+        return (torch.cat([q.reshape(T, -1), k.reshape(T, -1), y[:, 2 * G * dk :]], 1),
+                torch.stack([g, beta, qk, torch.zeros_like(g)], -1))
+
+    def delta_rule(self, qkv, scal, *, num_heads, num_kv_heads, key_dim, value_dim, state, step):
+        T, H, G, dk, dv = qkv.shape[0], num_heads, num_kv_heads, key_dim, value_dim
+        q = qkv[:, : G * dk].view(T, G, dk).repeat_interleave(H // G, 1)
+        k = qkv[:, G * dk : 2 * G * dk].view(T, G, dk).repeat_interleave(H // G, 1)
+        v = qkv[:, 2 * G * dk :].view(T, H, dv)
+        out = torch.empty(T, H, dv)
+        cu, ctx, slots = step.cu_q.tolist(), step.ctx_lens.tolist(), step.state_slots.tolist()
+        for s_ in range(len(ctx)):
+            a, b = cu[s_], cu[s_ + 1]
+            S = state[slots[s_]].clone() if ctx[s_] - (b - a) > 0 else torch.zeros_like(state[0])  # [H, dv, dk]
+            for t in range(a, b):
+                S = scal[t, :, 0, None, None] * S
+                u = scal[t, :, 1, None] * (v[t] - torch.einsum("hvk,hk->hv", S, k[t]))
+                S = S + u[:, :, None] * k[t][:, None, :]
+                out[t] = torch.einsum("hvk,hk->hv", S, q[t])
+            state[slots[s_]] = S
+        return out.reshape(T, H * dv)
+
     def gated_group_norm(self, o, proj, *, gate_offset, group, weight, eps, gate_activation, out_dtype):
         T, N = o.shape
         g = proj[:, gate_offset : gate_offset + N].float()
@@ -421,7 +495,8 @@ class PlainOps:
     # ------------------------------------------------------------------ rows of q, k, v prepared a token at a time
     def qkv_norm_rope_write(self, qkv, *, num_heads, num_kv_heads, num_value_heads, head_dim, value_dim, out_dim,
                             q_weight, k_weight, eps, positions, token_seq, cos, sin, k_pages,
-                            v_pages, block_tables, page_tokens, out_dtype, temp_coef=0.0, temp_every=0):
+                            v_pages, block_tables, page_tokens, out_dtype, temp_coef=0.0, temp_every=0, col0=0):
+        qkv = qkv[:, col0:]
         T, D, Dv, Dp = qkv.shape[0], head_dim, value_dim, out_dim
         nq, nk, nv = num_heads, num_kv_heads, num_value_heads
         p = qkv.float()
