@@ -19,7 +19,8 @@ and a float32 replay of one 8192-token sequence against the plain implementation
 reference's own harness (src/llmserve/bench/run.py:96,124-176): fixed output lengths, greedy, a
 warm-up run that is thrown away, one JSON line with the environment.
 
-``--workload designs`` (``--arms llama,gubotar,pazivik,rirovik,lanilorn``) puts four Lanilorn layers (four
+``--workload designs`` (``--arms llama,gubotar,pazivik,rirovik,lanilorn,miberax``) puts four Miberax layers (chunked
+attention beside the gated delta rule in every layer; dense and grouped routed feed-forwards), four Lanilorn layers (four
 residual streams; linear attention with a decay per channel and token, windowed attention with sinks and
 a norm over whole rows, differential attention; ungated dense feed-forwards), four Pazivik layers (latent attention
 with a window; dense and routed feed-forwards), four Gubotar layers (parallel, retention, retention, parallel) and
@@ -661,6 +662,27 @@ def lanilorn_layers(width, heads, kv_heads, head_dim, ff, window=1024, state_dim
     return [gla, att, diff, att]
 
 
+def miberax_layers(width, heads, kv_heads, head_dim, ff, chunk=512, state_dim=128, experts=8, identity=2, top=2):
+    """Four Miberax layers at a Llama layer's sizes: the Llama layer's heads on chunks of ``chunk``
+    positions beside the gated delta rule on heads of ``state_dim`` x ``state_dim`` (as the Gubotar arm's
+    linear attention); a dense feed-forward of the Llama layer's size in layers 0 and 2; in layers 1
+    and 3 ``experts`` gated experts of a quarter of that size and ``identity`` identity experts in two
+    groups of which one is kept, ``top`` per token, beside a shared one (as the Pazivik arm's)."""
+    lin = max(1, width // state_dim)
+
+    def layer(mlp):
+        return {"type": "parallel", "mlp": mlp, "mixer": {
+            "left": {"heads": heads, "kv_heads": kv_heads, "dim": head_dim, "vdim": head_dim, "scale": head_dim ** -0.5,
+                     "mask": {"size": chunk}, "rot": {"base": 500000.0, "dims": head_dim, "scaling": {"factor": 4.0}}},
+            "right": {"heads": lin, "kv_heads": lin, "dim": state_dim, "vdim": state_dim, "conv": 4}}}
+
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "router": {"experts": experts, "top": top, "groups": {"count": 2, "keep": 1},
+                                     "identity": identity, "scale": 2.5},
+           "expert": {"ff": ff // 4, "limit": 7.0}, "shared": {"ff": ff // 4, "limit": 7.0}}
+    return [layer(dense), layer(moe), layer(dense), layer(moe)]
+
+
 def kernel_profile(fn, reps=3) -> dict:
     """Device time of ``fn()`` by kernel, from the framework's profiler: microseconds per call."""
     import collections
@@ -706,6 +728,8 @@ def designs_main(args) -> int:
                                                  "layers": rirovik_layers(w, heads, kv, hd, ff)}),
             "lanilorn": ("random:lanilorn-2048", {"width": w, "vocab": ll["vocab_size"],
                                                    "layers": lanilorn_layers(w, heads, kv, hd, ff, state_dim=hd if w < 2048 else 128)}),
+            "miberax": ("random:miberax-2048", {"width": w, "vocab": ll["vocab_size"],
+                                                 "layers": miberax_layers(w, heads, kv, hd, ff, state_dim=hd if w < 2048 else 128)}),
         }
         arms = {k: v for k, v in arms.items() if k in args.arms.split(",")}
         row = {"sizes": f"{alias}: width {w}, ff {ff}, {heads} heads of {hd}, 4 layers"}
@@ -857,7 +881,7 @@ def main() -> int:
     ap.add_argument("--warmup", type=int, default=8)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--workload", default="decode", choices=["decode", "continuous", "long", "designs"])
-    ap.add_argument("--arms", default="llama,gubotar,pazivik,rirovik,lanilorn",
+    ap.add_argument("--arms", default="llama,gubotar,pazivik,rirovik,lanilorn,miberax",
                     help="--workload designs: which architectures run side by side")
     ap.add_argument("--model", default="smollm2-1.7b")
     ap.add_argument("--batch", type=int, default=8)

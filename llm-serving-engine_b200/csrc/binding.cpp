@@ -825,7 +825,8 @@ void delta_inputs(const Tensor& proj, int64_t col0, const Tensor& conv, const Op
 }
 
 void delta_rule(const Tensor& qkv, const Tensor& scal, Tensor& state, Tensor& out, const Tensor& cu_q,
-                const Tensor& ctx_lens, const Tensor& slots, int64_t H, int64_t G, int64_t dk, int64_t dv) {
+                const Tensor& ctx_lens, const Tensor& slots, int64_t H, int64_t G, int64_t dk, int64_t dv,
+                int64_t max_chunks, const OptTensor& scratch, bool short_too) {
   check_f32(qkv, "qkv");
   check_f32(scal, "scal");
   check_state(state, "state", dk);
@@ -842,9 +843,20 @@ void delta_rule(const Tensor& qkv, const Tensor& scal, Tensor& state, Tensor& ou
               "delta_rule: state must be [slots, heads, value_dim, key_dim]");
   TORCH_CHECK(cu_q.numel() == ctx_lens.numel() + 1 && slots.numel() >= ctx_lens.numel(),
               "delta_rule: per-sequence arrays disagree");
+  float* sp = nullptr;
+  int64_t total = 0;
+  if (max_chunks > 1) {
+    // every sequence of more than one chunk holds at most tokens / chunk + 1 of them
+    total = T / lse_delta_rule_chunk() + ctx_lens.numel();
+    TORCH_CHECK(scratch.has_value(), "delta_rule: long portions need the scratch");
+    check_f32(*scratch, "scratch");
+    TORCH_CHECK(scratch->numel() >= total * (int64_t)lse_delta_rule_chunk_floats((int)H, (int)dk, (int)dv),
+                "delta_rule: the scratch is too small");
+    sp = scratch->data_ptr<float>();
+  }
   done(lse_delta_rule(qkv.data_ptr<float>(), scal.data_ptr<float>(), state.data_ptr<float>(), out.data_ptr<float>(),
                       cu_q.data_ptr<int>(), ctx_lens.data_ptr<int>(), slots.data_ptr<int>(), (int)ctx_lens.numel(),
-                      (int)H, (int)G, (int)dk, (int)dv, stream()),
+                      (int)H, (int)G, (int)dk, (int)dv, stream(), (int)max_chunks, sp, (int)total, short_too ? 1 : 0),
        "delta_rule");
 }
 
@@ -1371,7 +1383,13 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
         py::arg("ca"), py::arg("cb"), py::arg("eps_in"), py::arg("w"), py::arg("eps"), py::arg("out"),
         py::arg("then_w"), py::arg("then_eps"), py::arg("then_groups") = 1);
   m.def("delta_inputs", &delta_inputs);
-  m.def("delta_rule", &delta_rule);
+  m.def("delta_rule", &delta_rule, py::arg("qkv"), py::arg("scal"), py::arg("state"), py::arg("out"), py::arg("cu_q"),
+        py::arg("ctx_lens"), py::arg("slots"), py::arg("H"), py::arg("G"), py::arg("dk"), py::arg("dv"),
+        py::arg("max_chunks") = 1, py::arg("scratch") = py::none(), py::arg("short_too") = true);
+  m.def("delta_rule_chunk", []() { return (int64_t)lse_delta_rule_chunk(); });
+  m.def("delta_rule_chunk_floats", [](int64_t H, int64_t dk, int64_t dv) {
+    return (int64_t)lse_delta_rule_chunk_floats((int)H, (int)dk, (int)dv);
+  });
   m.def("mix_normed", &mix_normed);
   m.def("gated_group_norm", &gated_group_norm);
   m.def("norm_rope_kv_write", &norm_rope_kv_write);

@@ -205,9 +205,16 @@ int lse_delta_inputs(const float* proj, long long stride, const float* conv, int
 
 // S <- g S; u = beta (v - S^T k); S <- S + k u^T; out = S^T q per head and token, float32, with qkv and
 // scal as lse_delta_inputs leaves them; state [slots, H, dv, dk]; out [T, H*dv]. dk <= 256.
+// A portion of more than lse_delta_rule_chunk() tokens runs as chunks (three launches) if max_chunks,
+// a bound on any sequence's chunks, is above one: scratch then holds total_chunks times
+// lse_delta_rule_chunk_floats() floats, total_chunks at least the chunks of all such sequences
+// together; short_too: the step may also hold shorter portions (one more launch).
+int lse_delta_rule_chunk(void);
+size_t lse_delta_rule_chunk_floats(int H, int dk, int dv);
 int lse_delta_rule(const float* qkv, const float* scal, float* state, float* out, const int* cu_q,
                    const int* ctx_lens, const int* slots, int num_seqs, int H, int G, int dk, int dv,
-                   cudaStream_t stream);
+                   cudaStream_t stream, int max_chunks = 1, float* scratch = nullptr, int total_chunks = 0,
+                   int short_too = 1);
 
 // ---- several residual streams, rows of q/k/v prepared a token at a time, differential attention
 // (streams_mixers.cu). The residual state is float32 [T, S * W]: a token's S streams of W values.

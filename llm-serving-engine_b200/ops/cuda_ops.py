@@ -150,6 +150,7 @@ class CudaOps:
         self._sums: dict[tuple[int, int], list[torch.Tensor]] = {}
         self._sums_live: set[int] = set()  # data_ptr of buffers whose sums have not been taken yet
         self._addmm_in_place: bool | None = None  # whether torch.addmm can add into a float32 tensor
+        self._chunk_scratch: dict[str, list[torch.Tensor]] = {}
         self.launches = 0  # kernels of this package enqueued (library matrix products not counted)
 
     # ------------------------------------------------------------------ capabilities
@@ -717,6 +718,17 @@ class CudaOps:
                 m.sums = None
         return out
 
+    def _kept_scratch(self, name: str, need: int) -> torch.Tensor:
+        """A float32 buffer of at least ``need`` values for the states of a portion's chunks."""
+        kept = self._chunk_scratch.setdefault(name, [])
+        if not kept or kept[-1].numel() < need:
+            if torch.cuda.is_current_stream_capturing():
+                raise RuntimeError(f"the {name} scratch must exist before graph capture")
+            # a captured step keeps the address of the scratch it was recorded with: an outgrown
+            # scratch is kept alive beside its successor
+            kept.append(torch.empty(need, dtype=torch.float32, device=self.device))
+        return kept[-1]
+
     def decay_linear_attention(self, proj, *, num_heads, key_dim, value_dim, decay, state, step,
                                activation, key_scale, cos, sin, decay_logits=None, decay_root=1.0,
                                query_scale=1.0):
@@ -735,14 +747,7 @@ class CudaOps:
             # a chunk's state, and with decays per channel the product of its decays behind them
             per_chunk = num_heads * (value_dim * key_dim + (key_dim if decay_logits is not None else 0))
             need = (T // L + int(step.cu_q.shape[0]) - 1) * per_chunk
-            scratch = getattr(self, "_la_scratch", None)
-            if scratch is None or scratch.numel() < need:
-                if torch.cuda.is_current_stream_capturing():
-                    raise RuntimeError("the linear-attention scratch must exist before graph capture")
-                # a captured step keeps the address of the scratch it was recorded with: an
-                # outgrown scratch is kept alive beside its successor
-                self._la_outgrown = getattr(self, "_la_outgrown", []) + ([scratch] if scratch is not None else [])
-                scratch = self._la_scratch = torch.empty(need, dtype=torch.float32, device=proj.device)
+            scratch = self._kept_scratch("linear attention", need)
         self.ext.decay_linear_attention(proj, out, state, decay, step.cu_q, step.ctx_lens, step.state_slots,
                                         num_heads, key_dim, value_dim, cos, sin, activation == "silu",
                                         float(key_scale), max_chunks, scratch, decay_logits, float(decay_root),
@@ -768,11 +773,22 @@ class CudaOps:
 
     def delta_rule(self, qkv, scal, *, num_heads, num_kv_heads, key_dim, value_dim, state, step):
         """``S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q`` per head and token, from each
-        request's ``state [slots, heads, value_dim, key_dim]``; returns ``o [T, heads * value_dim]``."""
-        out = torch.empty(qkv.shape[0], num_heads * value_dim, dtype=torch.float32, device=qkv.device)
+        request's ``state [slots, heads, value_dim, key_dim]``; returns ``o [T, heads * value_dim]``.
+        Portions longer than the kernel's chunk run as chunks (three launches and a scratch)."""
+        T = qkv.shape[0]
+        out = torch.empty(T, num_heads * value_dim, dtype=torch.float32, device=qkv.device)
+        L = self._delta_chunk = getattr(self, "_delta_chunk", None) or int(self.ext.delta_rule_chunk())
+        host = getattr(step, "host", None)
+        seqs = int(step.cu_q.shape[0]) - 1
+        longest = int(host.q_lens.max()) if host is not None else T - (seqs - 1)
+        max_chunks, scratch = max(1, -(-longest // L)), None
+        short_too = host is None or int(host.q_lens.min()) <= L
+        if max_chunks > 1:
+            need = (T // L + seqs) * int(self.ext.delta_rule_chunk_floats(int(num_heads), int(key_dim), int(value_dim)))
+            scratch = self._kept_scratch("delta_rule", need)
         self.ext.delta_rule(qkv, scal, state, out, step.cu_q, step.ctx_lens, step.state_slots, int(num_heads),
-                            int(num_kv_heads), int(key_dim), int(value_dim))
-        self.launches += 1
+                            int(num_kv_heads), int(key_dim), int(value_dim), max_chunks, scratch, short_too)
+        self.launches += (3 if max_chunks > 1 else 0) + (1 if short_too else 0)
         return out
 
     def gated_group_norm(self, o, proj, *, gate_offset, group, weight, eps, gate_activation, out_dtype):
