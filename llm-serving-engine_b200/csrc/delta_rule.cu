@@ -27,7 +27,10 @@ namespace lse {
 // The convolution of row i of a portion reads rows i - taps + 1 .. i, the first taps - 1 rows also
 // the inputs kept from the step before (state [slots, taps - 1, channels], oldest first). The warp
 // of a portion's row 0 makes all of these first rows and then writes the new state of its
-// channels, so nobody else touches them. V channels per lane and visit.
+// channels, so nobody else touches them. V channels per lane and visit, at most NK visits for a
+// key head. TAPS:
+// the number of taps (0: any; their inputs are then fetched one after another). STAGED: the inputs of
+// all rows of the warp are fetched together into shared memory.
 constexpr int DI_WARPS = 4, DI_MAX = 256;  // DI_MAX: largest key size
 
 struct DeltaInputs {
@@ -48,6 +51,12 @@ struct DeltaInputs {
   float q_scale;
 };
 
+__device__ __forceinline__ void dr_copy(float* smem, const float* gmem, bool wide) {
+  const uint32_t addr = (uint32_t)__cvta_generic_to_shared(smem);
+  if (wide) asm volatile("cp.async.ca.shared.global [%0], [%1], 16;\n" ::"r"(addr), "l"(gmem));
+  else asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"(addr), "l"(gmem));
+}
+
 template <int V>
 __device__ __forceinline__ void di_load(const float* p, float (&v)[V]) {
   if constexpr (V == 4) load4<float>(p, v);
@@ -59,137 +68,189 @@ __device__ __forceinline__ void di_store(float* p, const float (&v)[V]) {
   else p[0] = v[0];
 }
 
-template <int V>
+template <int V, int TAPS, int NK, bool STAGED>
 __global__ void __launch_bounds__(DI_WARPS * 32) delta_inputs_kernel(const DeltaInputs a) {
+  extern __shared__ __align__(16) float di_smem[];
   pdl_trigger();
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int job = blockIdx.y * DI_WARPS + warp;
-  const int past = a.taps - 1;
+  const bool is_qk = job < a.G;
+  const int past = (TAPS > 0 ? TAPS : a.taps) - 1;
+  const int C = 2 * a.G * a.dk + a.H * a.dv;
+  const int t_begin = blockIdx.x * a.rows, t_end = min(a.T, t_begin + a.rows);
+  const int d_lane = lane * V;
+  // this warp's channels: one run of q and one of k, or one run of v
+  const int len = is_qk ? a.dk : a.dv;
+  const int ch0 = is_qk ? job * a.dk : 2 * a.G * a.dk + (job - a.G) * a.dv;
+  const int ch1 = is_qk ? (a.G + job) * a.dk : 0;
+  // the sequence of the row at hand: looked up again only where the next one starts
+  int seq = a.token_seq[t_begin];
+  int r0 = a.cu_q[seq], r1 = a.cu_q[seq + 1];
+  bool from_zero = a.ctx_lens[seq] - (r1 - r0) == 0;
+  float* st = a.conv_state ? a.conv_state + (size_t)a.slots[seq] * past * C : nullptr;
   pdl_wait();
   if (job >= a.G + a.H) return;
-  const int t_end = min(a.T, (int)(blockIdx.x + 1) * a.rows);
-  for (int t = blockIdx.x * a.rows; t < t_end; ++t) {
-    const int seq = a.token_seq[t];
-    const int r0 = a.cu_q[seq], n = a.cu_q[seq + 1] - r0;
-    const int i0 = t - r0;  // this row's place in its portion
-    if (i0 > 0 && i0 < past) continue;  // made by the warp of row 0
-    const bool first = i0 == 0;
-    const bool from_zero = a.ctx_lens[seq] - n == 0;
-    const int C = 2 * a.G * a.dk + a.H * a.dv;
-    float* st = a.conv_state ? a.conv_state + (size_t)a.slots[seq] * past * C : nullptr;
-    const float* base = a.proj + (size_t)r0 * a.stride;
+  // STAGED: all inputs of the warp's rows (and of the rows just before them) are on their way together; a lane reads
+  // back only what it copied itself
+  const int s_begin = max(0, t_begin - past), width = max(2 * a.dk, a.dv);
+  float* staged = STAGED ? di_smem + (size_t)warp * (a.rows + past) * width : nullptr;
+  if constexpr (STAGED) {
+    for (int t = s_begin; t < t_end; ++t) {
+      const float* src = a.proj + (size_t)t * a.stride;
+      float* dst = staged + (t - s_begin) * width;
+      for (int d = d_lane; d < len; d += 32 * V) {
+        dr_copy(dst + d, src + ch0 + d, V == 4);
+        if (is_qk) dr_copy(dst + a.dk + d, src + ch1 + d, V == 4);
+      }
+    }
+    asm volatile("cp.async.commit_group;\n" ::);
+    asm volatile("cp.async.wait_group 0;\n" ::);
+  }
 
-    // the convolution of row i, channels ch .. ch + V - 1, then silu
-    auto conv = [&](int i, int ch, float (&y)[V]) {
-      float x[V], w[V];
-      di_load<V>(base + (size_t)i * a.stride + ch, x);
-      di_load<V>(a.conv + (size_t)past * C + ch, w);
+  // x_j of row i: the input j rows back, of dims d .. d + V - 1 of run `second` (0: q or v, 1: k)
+  auto input = [&](int i, int j, int second, int d, float (&x)[V]) {
+    const int ch = (second ? ch1 : ch0) + d;
+    const int t = r0 + i - j;
+    if (i - j >= 0) {
+      if (STAGED && t >= s_begin && t < t_end) di_load<V>(staged + (t - s_begin) * width + second * a.dk + d, x);
+      else di_load<V>(a.proj + (size_t)t * a.stride + ch, x);
+    } else if (!from_zero) {
+      di_load<V>(st + (size_t)(past + i - j) * C + ch, x);
+    } else {
 #pragma unroll
-      for (int e = 0; e < V; ++e) y[e] = w[e] * x[e];
-      for (int j = 1; j <= past; ++j) {
-        float xp[V];
-        if (i - j >= 0) {
-          di_load<V>(base + (size_t)(i - j) * a.stride + ch, xp);
-        } else if (from_zero) {
-          break;
-        } else {
-          di_load<V>(st + (size_t)(past + i - j) * C + ch, xp);
-        }
+      for (int e = 0; e < V; ++e) x[e] = 0.f;
+    }
+  };
+  // the convolution of row i, then silu
+  auto conv = [&](int i, int second, int d, float (&y)[V]) {
+    const int ch = (second ? ch1 : ch0) + d;
+    const bool alone = r1 - r0 == 1;  // a single row: the state moves on by one, while the inputs are at hand
+    if constexpr (TAPS > 0) {
+      float x[TAPS][V], w[TAPS][V];
+      const bool direct = STAGED && i >= TAPS - 1 && r0 + i < t_end;  // all of it lies in shared memory
+      const float* xp = staged + (direct ? (r0 + i - s_begin) * width + second * a.dk + d : 0);
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) {
+        if (direct) di_load<V>(xp - j * width, x[j]);
+        else input(i, j, second, d, x[j]);
+        di_load<V>(a.conv + (size_t)(TAPS - 1 - j) * C + ch, w[j]);
+      }
+#pragma unroll
+      for (int e = 0; e < V; ++e) y[e] = w[0][e] * x[0][e];
+#pragma unroll
+      for (int j = 1; j < TAPS; ++j)
+#pragma unroll
+        for (int e = 0; e < V; ++e) y[e] = fmaf(w[j][e], x[j][e], y[e]);
+      if (alone)
+#pragma unroll
+        for (int j = 0; j + 1 < TAPS; ++j) di_store<V>(st + (size_t)(TAPS - 2 - j) * C + ch, x[j]);
+    } else {
+#pragma unroll
+      for (int e = 0; e < V; ++e) y[e] = 0.f;
+      for (int j = past; j >= 0; --j) {  // oldest first: a place of the state is read before it is written
+        float x[V], w[V];
+        input(i, j, second, d, x);
         di_load<V>(a.conv + (size_t)(past - j) * C + ch, w);
 #pragma unroll
-        for (int e = 0; e < V; ++e) y[e] = fmaf(w[e], xp[e], y[e]);
+        for (int e = 0; e < V; ++e) y[e] = fmaf(w[e], x[e], y[e]);
+        if (alone && j < past) di_store<V>(st + (size_t)(past - 1 - j) * C + ch, x);
       }
-      if (n == 1 && past > 0) {  // a single row: the state moves on by one, while x is at hand
-        for (int s = 0; s + 1 < past; ++s) {
-          float o[V];
-#pragma unroll
-          for (int e = 0; e < V; ++e) o[e] = 0.f;
-          if (!from_zero) di_load<V>(st + (size_t)(s + 1) * C + ch, o);
-          di_store<V>(st + (size_t)s * C + ch, o);
-        }
-        di_store<V>(st + (size_t)(past - 1) * C + ch, x);
-      }
-#pragma unroll
-      for (int e = 0; e < V; ++e) y[e] = y[e] / (1.f + expf(-y[e]));
-    };
-    // the new state of channels ch .. after a portion of several rows: its last inputs
-    auto keep = [&](int ch) {
-      for (int s = 0; s < past; ++s) {
-        const int i = n - past + s;
-        float o[V];
-#pragma unroll
-        for (int e = 0; e < V; ++e) o[e] = 0.f;
-        if (i >= 0) di_load<V>(base + (size_t)i * a.stride + ch, o);
-        else if (!from_zero) di_load<V>(st + (size_t)(past + i) * C + ch, o);  // place s + n: not written yet
-        di_store<V>(st + (size_t)s * C + ch, o);
-      }
-    };
-    const int i_end = first ? min(n, max(past, 1)) : i0 + 1;
-    if (job < a.G) {
-      const int kh = job, group = a.H / a.G;
-      const int qc = kh * a.dk, kc = (a.G + kh) * a.dk;
-      constexpr int K = DI_MAX / (32 * V);
-      for (int i = i0; i < i_end; ++i) {
-        float q[K][V], k[K][V];
-        float sq = 0.f, sk = 0.f, qk = 0.f;
-#pragma unroll
-        for (int c = 0; c < K; ++c) {
-          const int d = (lane + 32 * c) * V;
-          if (d < a.dk) {
-            conv(i, qc + d, q[c]);
-            conv(i, kc + d, k[c]);
-#pragma unroll
-            for (int e = 0; e < V; ++e) {
-              sq += q[c][e] * q[c][e];
-              sk += k[c][e] * k[c][e];
-              qk += q[c][e] * k[c][e];
-            }
-          }
-        }
-        sq = warp_sum(sq);
-        sk = warp_sum(sk);
-        qk = warp_sum(qk);
-        const float iq = a.q_scale / sqrtf(sq + 1e-6f), ik = 1.f / sqrtf(sk + 1e-6f);
-        float* row = a.qkv + (size_t)(r0 + i) * C;
-#pragma unroll
-        for (int c = 0; c < K; ++c) {
-          const int d = (lane + 32 * c) * V;
-          if (d < a.dk) {
-#pragma unroll
-            for (int e = 0; e < V; ++e) {
-              q[c][e] *= iq;
-              k[c][e] *= ik;
-            }
-            di_store<V>(row + qc + d, q[c]);
-            di_store<V>(row + kc + d, k[c]);
-          }
-        }
-        for (int h = kh * group + lane; h < (kh + 1) * group; h += 32) {
-          const float* p = base + (size_t)i * a.stride + C + a.H * a.dv + h;
-          const float b = p[0], x = p[a.H] + a.dt_bias[h];
-          const float softplus = fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)));
-          a.scal[(size_t)(r0 + i) * a.H + h] =
-              make_float4(expf(-expf(a.A_log[h]) * softplus), 1.f / (1.f + expf(-b)), qk * iq * ik, 0.f);
-        }
-      }
-      if (first && n > 1 && past > 0)
-        for (int d = lane * V; d < a.dk; d += 32 * V) {
-          keep(qc + d);
-          keep(kc + d);
-        }
-    } else {
-      const int h = job - a.G;
-      const int vc = 2 * a.G * a.dk + h * a.dv;
-      for (int i = i0; i < i_end; ++i)
-        for (int d = lane * V; d < a.dv; d += 32 * V) {
-          float y[V];
-          conv(i, vc + d, y);
-          di_store<V>(a.qkv + (size_t)(r0 + i) * C + vc + d, y);
-        }
-      if (first && n > 1 && past > 0)
-        for (int d = lane * V; d < a.dv; d += 32 * V) keep(vc + d);
     }
+#pragma unroll
+    for (int e = 0; e < V; ++e) y[e] = __fdividef(y[e], 1.f + expf(-y[e]));
+  };
+  // the new state after a portion of several rows: its last inputs, oldest first
+  auto keep = [&](int second, int d) {
+    for (int s = 0; s < past; ++s) {
+      float x[V];
+      input(r1 - r0 - 1, past - 1 - s, second, d, x);  // (place s + rows of the old state: not written yet)
+      di_store<V>(st + (size_t)s * C + (second ? ch1 : ch0) + d, x);
+    }
+  };
+  // decay, step size and k . q of row t, value head h
+  auto numbers = [&](int t, int h, float kq) {
+    const float* p = a.proj + (size_t)t * a.stride + C + a.H * a.dv + h;
+    const float b = p[0], x = p[a.H] + a.dt_bias[h];
+    const float softplus = fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)));
+    a.scal[(size_t)t * a.H + h] = make_float4(expf(-expf(a.A_log[h]) * softplus), 1.f / (1.f + expf(-b)), kq, 0.f);
+  };
+  const int group = a.H / a.G;
+  float kq_mine = 0.f;  // lane r: k . q of the warp's row r
+  unsigned made = 0;    // rows of the warp whose numbers are still to be written
+  for (int t = t_begin; t < t_end; ++t) {
+    if (t >= r1) {
+      seq = a.token_seq[t];
+      r0 = a.cu_q[seq];
+      r1 = a.cu_q[seq + 1];
+      from_zero = a.ctx_lens[seq] - (r1 - r0) == 0;
+      st = a.conv_state ? a.conv_state + (size_t)a.slots[seq] * past * C : nullptr;
+    }
+    const int i0 = t - r0, n = r1 - r0;
+    if (i0 > 0 && i0 < past) continue;  // made by the warp of row 0
+    const int i_end = i0 == 0 ? min(n, max(past, 1)) : i0 + 1;
+    for (int i = i0; i < i_end; ++i) {
+      float* row = a.qkv + (size_t)(r0 + i) * C;
+      if (!is_qk) {
+        for (int d = d_lane; d < len; d += 32 * V) {
+          float y[V];
+          conv(i, 0, d, y);
+          di_store<V>(row + ch0 + d, y);
+        }
+        continue;
+      }
+      float q[NK][V], k[NK][V];
+      float sq = 0.f, sk = 0.f, qk = 0.f;
+#pragma unroll
+      for (int c = 0; c < NK; ++c) {
+        const int d = d_lane + 32 * V * c;
+        if (d < len) {
+          conv(i, 0, d, q[c]);
+          conv(i, 1, d, k[c]);
+#pragma unroll
+          for (int e = 0; e < V; ++e) {
+            sq += q[c][e] * q[c][e];
+            sk += k[c][e] * k[c][e];
+            qk += q[c][e] * k[c][e];
+          }
+        }
+      }
+      sq = warp_sum(sq);
+      sk = warp_sum(sk);
+      qk = warp_sum(qk);
+      const float iq = a.q_scale * rsqrtf(sq + 1e-6f), ik = rsqrtf(sk + 1e-6f);
+#pragma unroll
+      for (int c = 0; c < NK; ++c) {
+        const int d = d_lane + 32 * V * c;
+        if (d < len) {
+#pragma unroll
+          for (int e = 0; e < V; ++e) {
+            q[c][e] *= iq;
+            k[c][e] *= ik;
+          }
+          di_store<V>(row + ch0 + d, q[c]);
+          di_store<V>(row + ch1 + d, k[c]);
+        }
+      }
+      const int r = r0 + i - t_begin;
+      if (r < a.rows) {  // one of this warp's rows: its numbers are written at the end, a lane per row and head
+        if (lane == r) kq_mine = qk * iq * ik;
+        made |= 1u << r;
+      } else {
+        for (int h = job * group + lane; h < (job + 1) * group; h += 32) numbers(r0 + i, h, qk * iq * ik);
+      }
+    }
+    if (i0 == 0 && n > 1)
+      for (int d = d_lane; d < len; d += 32 * V) {
+        keep(0, d);
+        if (is_qk) keep(1, d);
+      }
   }
+  if (is_qk)
+    for (int base = 0; base < a.rows * group; base += 32) {
+      const int idx = base + lane, r = idx / group;
+      const float kq = __shfl_sync(0xffffffffu, kq_mine, r & 31);
+      if (r < a.rows && (made >> r & 1u)) numbers(t_begin + r, job * group + idx - r * group, kq);
+    }
 }
 
 // ------------------------------------------------------------------------------------ recurrence
@@ -217,12 +278,6 @@ struct DeltaRule {
   int H, G, dk, dv;
   int longest;         // longer portions than this are not served here (0: all are)
 };
-
-__device__ __forceinline__ void dr_copy(float* smem, const float* gmem, bool wide) {
-  const uint32_t addr = (uint32_t)__cvta_generic_to_shared(smem);
-  if (wide) asm volatile("cp.async.ca.shared.global [%0], [%1], 16;\n" ::"r"(addr), "l"(gmem));
-  else asm volatile("cp.async.ca.shared.global [%0], [%1], 4;\n" ::"r"(addr), "l"(gmem));
-}
 
 template <int P>
 __global__ void __launch_bounds__(DR_THREADS) delta_rule_kernel(const DeltaRule a) {
@@ -374,7 +429,7 @@ __global__ void __launch_bounds__(DR_THREADS) delta_rule_kernel(const DeltaRule 
 // All in float32 (register-tiled products on the CUDA cores); the decays enter as products of
 // factors in (0, 1], so nothing overflows. A chunk that is not full is filled up with tokens of
 // g = 1, beta = 0 and zero vectors.
-constexpr int DC_L = 64, DC_THREADS = 256, DC_B = 16, DC_B_THREADS = 128, DC_N = 64;
+constexpr int DC_L = 64, DC_THREADS = 256, DC_B = 16, DC_B_THREADS = 256, DC_N = 64;
 
 struct DeltaChunks {
   const float* qkv;    // as DeltaRule
@@ -385,15 +440,17 @@ struct DeltaChunks {
   const int* ctx_lens;
   const int* slots;
   int H, G, dk, dv;
-  int ldk;             // row length of staged q, k, w and state rows: dk up to a multiple of 8, + 4
+  int ld;              // row length of q, k, W and state rows: dk up to a multiple of 16, + 4 (zeros behind dk)
+  int dvp;             // dv up to a multiple of DC_B
   int stages;          // launch B: chunks staged at a time
-  // scratch per (chunk, head)
-  float* w;            // [64, dk]
-  float* u;            // [64, dv]: U, then u
-  float* p;            // [64, 64]
-  float* s0;           // [dv, dk]: the state before the chunk
-  float* coef;         // [2, 64]: G_t, r_(last,t)
+  // scratch per (chunk, head), laid out as the kernels stage it
+  float* wk;           // [2][64][ld]: W, then r_(last,t) k_t
+  float* u;            // [dvp / 16][64][16]: U, then u, in the slices of launch B
+  float* p;            // [64][DC_LDP]
+  float* s0;           // [dvp][ld]: the (transposed) state before the chunk
+  float* g;            // [64]: G_t
 };
+constexpr int DC_LDP = DC_L + 4;
 
 // First chunk of a sequence in the scratch (only sequences of more than one chunk have any), and its chunks.
 __device__ __forceinline__ int dc_first_chunk(const int* cu_q, int seq) {
@@ -405,25 +462,35 @@ __device__ __forceinline__ int dc_first_chunk(const int* cu_q, int seq) {
   return base;
 }
 
-// rows t < tn of `len` values, `stride` apart, into rows of `ld` floats; what is left of 64 rows and of `ld` is zero
+// 64 rows, DC_THREADS / 64 threads each: row t < tn has `len` values (rows `stride` apart); what is left of 64 rows of
+// `ld` floats is zero
 __device__ __forceinline__ void dc_stage(float* dst, int ld, const float* src, long long stride, int tn, int len,
-                                         bool wide, int rows, int tid, int threads) {
+                                         bool wide) {
+  constexpr int PER = DC_THREADS / DC_L;
+  const int t = threadIdx.x / PER, q = threadIdx.x % PER;
+  float* d = dst + t * ld;
+  const float* s = src + (size_t)t * stride;
   if (wide) {
-    const int per = ld / 4, full = len / 4;
-    for (int idx = tid; idx < rows * per; idx += threads) {
-      const int t = idx / per, i = idx - t * per;
-      float* d = dst + (size_t)t * ld + 4 * i;
-      if (t < tn && i < full) dr_copy(d, src + (size_t)t * stride + 4 * i, true);
-      else *reinterpret_cast<float4*>(d) = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int i = 4 * q; i < ld; i += 4 * PER) {
+      if (t < tn && i < len) dr_copy(d + i, s + i, true);
+      else *reinterpret_cast<float4*>(d + i) = make_float4(0.f, 0.f, 0.f, 0.f);
     }
   } else {
-    for (int idx = tid; idx < rows * ld; idx += threads) {
-      const int t = idx / ld, i = idx - t * ld;
-      float* d = dst + (size_t)t * ld + i;
-      if (t < tn && i < len) dr_copy(d, src + (size_t)t * stride + i, false);
-      else *d = 0.f;
+    for (int i = q; i < ld; i += PER) {
+      if (t < tn && i < len) dr_copy(d + i, s + i, false);
+      else d[i] = 0.f;
     }
   }
+}
+// n floats (a multiple of 4) as they lie
+template <int THREADS>
+__device__ __forceinline__ void dc_stage_flat(float* dst, const float* src, int n) {
+  for (int i = 4 * threadIdx.x; i < n; i += 4 * THREADS) dr_copy(dst + i, src + i, true);
+}
+template <int THREADS>
+__device__ __forceinline__ void dc_store_flat(float* dst, const float* src, int n) {
+  for (int i = 4 * threadIdx.x; i < n; i += 4 * THREADS)
+    *reinterpret_cast<float4*>(dst + i) = *reinterpret_cast<const float4*>(src + i);
 }
 
 // ---- launch A
@@ -438,18 +505,18 @@ __global__ void __launch_bounds__(DC_THREADS, 2) delta_chunk_systems_kernel(cons
     return;
   }
   const size_t at = (size_t)(dc_first_chunk(a.cu_q, seq) + c) * a.H + h;
-  const int dk = a.dk, dv = a.dv, ld = a.ldk, tid = threadIdx.x;
+  const int dk = a.dk, dv = a.dv, ld = a.ld, dvp = a.dvp, tid = threadIdx.x;
   const int kh = h / (a.H / a.G), C = 2 * a.G * dk + a.H * dv;
   const int t0 = r0 + c * DC_L, tn = min(DC_L, n - c * DC_L);
-  float* ks = dc_smem;                 // [64][ld]
-  float* qs = ks + DC_L * ld;          // [64][ld]
-  float* ms = qs + DC_L * ld;          // [64][68]: r, then M
-  float* gs = ms + DC_L * 68;          // g [64], beta [64], G [64]
+  float* ks = dc_smem;                   // [64][ld]: k, then W
+  float* qs = ks + DC_L * ld;            // [64][ld]: q; then v and U, [64][dvp]
+  float* ms = qs + DC_L * max(ld, dvp);  // [64][DC_LDP]: r, then M
+  float* gs = ms + DC_L * DC_LDP;        // g [64], beta [64], G [64], r_(last,t) [64]
   pdl_wait();
-  const float* row0 = a.qkv + (size_t)t0 * C + (size_t)kh * dk;
+  const float* row0 = a.qkv + (size_t)t0 * C;
   const bool wide = dk % 4 == 0 && C % 4 == 0;
-  dc_stage(qs, ld, row0, C, tn, dk, wide, DC_L, tid, DC_THREADS);
-  dc_stage(ks, ld, row0 + (size_t)a.G * dk, C, tn, dk, wide, DC_L, tid, DC_THREADS);
+  dc_stage(qs, ld, row0 + (size_t)kh * dk, C, tn, dk, wide);
+  dc_stage(ks, ld, row0 + (size_t)(a.G + kh) * dk, C, tn, dk, wide);
   asm volatile("cp.async.commit_group;\n" ::);
   if (tid < DC_L) {
     const float4 s = tid < tn ? a.scal[(size_t)(t0 + tid) * a.H + h] : make_float4(1.f, 0.f, 0.f, 0.f);
@@ -461,9 +528,9 @@ __global__ void __launch_bounds__(DC_THREADS, 2) delta_chunk_systems_kernel(cons
     float r = 1.f;
     for (int t = tid; t < DC_L; ++t) {
       if (t > tid) r *= gs[t];
-      ms[t * 68 + tid] = r;
+      ms[t * DC_LDP + tid] = r;
     }
-    a.coef[at * 2 * DC_L + DC_L + tid] = r;
+    gs[3 * DC_L + tid] = r;
   } else if (tid == DC_L) {
     float g = 1.f;
     for (int t = 0; t < DC_L; ++t) {
@@ -473,7 +540,7 @@ __global__ void __launch_bounds__(DC_THREADS, 2) delta_chunk_systems_kernel(cons
   }
   asm volatile("cp.async.wait_group 0;\n" ::);
   __syncthreads();
-  if (tid < DC_L) a.coef[at * 2 * DC_L + tid] = gs[2 * DC_L + tid];
+  if (tid < DC_L) a.g[at * DC_L + tid] = gs[2 * DC_L + tid];
   {
     // thread (ty, tx): rows ty + 16 i, columns tx + 16 j of K K^T and Q K^T, the blocks j <= i
     const int ty = tid >> 4, tx = tid & 15;
@@ -503,7 +570,23 @@ __global__ void __launch_bounds__(DC_THREADS, 2) delta_chunk_systems_kernel(cons
         }
       }
     }
-    float* pg = a.p + at * DC_L * DC_L;
+    __syncthreads();  // q is used up: v takes its place
+    {
+      const int t = tid >> 2;
+      float* d = qs + t * dvp;
+      const float* s = row0 + (size_t)t * C + (size_t)2 * a.G * dk + (size_t)h * dv;
+      const bool wv = wide && dv % 4 == 0;
+      const int step = wv ? 4 : 1;
+      for (int i = (tid & 3) * step; i < dvp; i += 4 * step) {
+        if (t < tn && i < dv) {
+          dr_copy(d + i, s + i, wv);
+        } else {
+          for (int e = 0; e < step; ++e) d[i + e] = 0.f;
+        }
+      }
+    }
+    asm volatile("cp.async.commit_group;\n" ::);
+    float* pg = a.p + at * DC_L * DC_LDP;
 #pragma unroll
     for (int i = 0; i < 4; ++i)
 #pragma unroll
@@ -511,180 +594,201 @@ __global__ void __launch_bounds__(DC_THREADS, 2) delta_chunk_systems_kernel(cons
         const int t = ty + 16 * i, s = tx + 16 * j;
         float m = 0.f, p = 0.f;
         if (s <= t) {
-          const float r = ms[t * 68 + s];
+          const float r = ms[t * DC_LDP + s];
           p = r * qk[i][j];
           if (s < t) m = gs[DC_L + t] * r * kk[i][j];
         }
-        pg[t * DC_L + s] = p;
-        ms[t * 68 + s] = m;  // this thread alone reads and writes the element
+        pg[t * DC_LDP + s] = p;
+        ms[t * DC_LDP + s] = m;  // this thread alone reads and writes the element
       }
   }
-  __syncthreads();
-  // forward substitution, a column of W or U per thread, its 64 values in registers
-  for (int col = tid; col < dk + dv; col += DC_THREADS) {
-    const bool is_w = col < dk;
-    const float* v = a.qkv + (size_t)t0 * C + (size_t)2 * a.G * dk + (size_t)h * dv + (col - dk);
-    float* dst = is_w ? a.w + at * DC_L * dk + col : a.u + at * DC_L * dv + (col - dk);
-    const int dst_stride = is_w ? dk : dv;
-    float x[DC_L];
-#pragma unroll
-    for (int t = 0; t < DC_L; ++t) {
-      float rhs = 0.f;
-      if (is_w) rhs = gs[DC_L + t] * gs[2 * DC_L + t] * ks[t * ld + col];
-      else if (t < tn) rhs = gs[DC_L + t] * v[(size_t)t * C];
-      float e0 = 0.f, e1 = 0.f, e2 = 0.f, e3 = 0.f;
-      const float4* m4 = reinterpret_cast<const float4*>(ms + t * 68);
-#pragma unroll
-      for (int s4 = 0; s4 < (t + 3) / 4; ++s4) {  // entries from t on are zero
-        const float4 m = m4[s4];
-        e0 = fmaf(m.x, x[4 * s4], e0);
-        if (4 * s4 + 1 < t) e1 = fmaf(m.y, x[4 * s4 + 1], e1);
-        if (4 * s4 + 2 < t) e2 = fmaf(m.z, x[4 * s4 + 2], e2);
-        if (4 * s4 + 3 < t) e3 = fmaf(m.w, x[4 * s4 + 3], e3);
-      }
-      x[t] = rhs - ((e0 + e1) + (e2 + e3));
-      dst[(size_t)t * dst_stride] = x[t];
+  {  // r_(last,t) k_t
+    const int t = tid >> 2;
+    const float rho = gs[3 * DC_L + t];
+    float* kg = a.wk + at * 2 * DC_L * ld + (size_t)(DC_L + t) * ld;
+    for (int i = 4 * (tid & 3); i < ld; i += 16) {
+      const float4 k = *reinterpret_cast<const float4*>(ks + t * ld + i);
+      *reinterpret_cast<float4*>(kg + i) = make_float4(rho * k.x, rho * k.y, rho * k.z, rho * k.w);
     }
   }
+  asm volatile("cp.async.wait_group 0;\n" ::);
+  __syncthreads();
+  // Forward substitution in blocks of 16 rows, in place: two columns of W and U per thread (a row of M is
+  // read once for both). What the rows of earlier blocks contribute comes from shared memory, the
+  // block's own 16 values stay in registers.
+  const int columns = dk + dvp, half = (columns + 1) / 2;
+  for (int col = tid; col < half; col += DC_THREADS) {
+    float* x[2];
+    int xs[2];
+    bool is_w[2];
+#pragma unroll
+    for (int v = 0; v < 2; ++v) {
+      const int cc = col + v * half < columns ? col + v * half : col;  // (an odd number: one thread has its column twice)
+      is_w[v] = cc < dk;
+      x[v] = is_w[v] ? ks + cc : qs + (cc - dk);
+      xs[v] = is_w[v] ? ld : dvp;
+    }
+#pragma unroll 1
+    for (int b = 0; b < DC_L; b += 16) {
+      float acc[2][16];
+#pragma unroll
+      for (int i = 0; i < 16; ++i) {
+        const float beta = gs[DC_L + b + i], g = gs[2 * DC_L + b + i];
+#pragma unroll
+        for (int v = 0; v < 2; ++v) acc[v][i] = (is_w[v] ? beta * g : beta) * x[v][(b + i) * xs[v]];
+      }
+#pragma unroll 1
+      for (int s = 0; s < b; s += 4) {
+        float xv[2][4];
+#pragma unroll
+        for (int v = 0; v < 2; ++v)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) xv[v][e] = x[v][(s + e) * xs[v]];
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+          const float4 m = *reinterpret_cast<const float4*>(ms + (b + i) * DC_LDP + s);
+#pragma unroll
+          for (int v = 0; v < 2; ++v) {
+            acc[v][i] = fmaf(-m.x, xv[v][0], acc[v][i]);
+            acc[v][i] = fmaf(-m.y, xv[v][1], acc[v][i]);
+            acc[v][i] = fmaf(-m.z, xv[v][2], acc[v][i]);
+            acc[v][i] = fmaf(-m.w, xv[v][3], acc[v][i]);
+          }
+        }
+      }
+#pragma unroll
+      for (int s = 0; s < 16; s += 4) {
+        // the block's rows s .. s + 3 are finished one after another, the rows below take them off as they come
+#pragma unroll
+        for (int i = s + 1; i < 16; ++i) {
+          const float4 m = *reinterpret_cast<const float4*>(ms + (b + i) * DC_LDP + b + s);
+#pragma unroll
+          for (int v = 0; v < 2; ++v) {
+            acc[v][i] = fmaf(-m.x, acc[v][s], acc[v][i]);
+            if (i > s + 1) acc[v][i] = fmaf(-m.y, acc[v][s + 1], acc[v][i]);
+            if (i > s + 2) acc[v][i] = fmaf(-m.z, acc[v][s + 2], acc[v][i]);
+            if (i > s + 3) acc[v][i] = fmaf(-m.w, acc[v][s + 3], acc[v][i]);
+          }
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < 16; ++i)
+#pragma unroll
+        for (int v = 0; v < 2; ++v) x[v][(b + i) * xs[v]] = acc[v][i];
+    }
+  }
+  __syncthreads();
+  dc_store_flat<DC_THREADS>(a.wk + at * 2 * DC_L * ld, ks, DC_L * ld);
+  float* ug = a.u + at * DC_L * dvp;
+  const int t = tid >> 2, q = 4 * (tid & 3);
+  for (int c0 = 0; c0 < dvp; c0 += DC_B)
+    *reinterpret_cast<float4*>(ug + (size_t)c0 * DC_L + t * DC_B + q) =
+        *reinterpret_cast<const float4*>(qs + t * dvp + c0 + q);
 }
 
 // ---- launch B
 __global__ void __launch_bounds__(DC_B_THREADS) delta_chunk_states_kernel(const DeltaChunks a) {
   extern __shared__ __align__(16) float dc_smem[];
   pdl_trigger();
-  const int dk = a.dk, dv = a.dv, ld = a.ldk, tid = threadIdx.x;
-  const int slices = (dv + DC_B - 1) / DC_B;
-  const int h = blockIdx.x / slices, c0 = (blockIdx.x - h * slices) * DC_B, seq = blockIdx.y;
+  const int dk = a.dk, dv = a.dv, ld = a.ld, tid = threadIdx.x;
+  const int slices = a.dvp / DC_B;
+  const int h = blockIdx.x / slices, slice = blockIdx.x - h * slices, c0 = slice * DC_B, seq = blockIdx.y;
   const int r0 = a.cu_q[seq], n = a.cu_q[seq + 1] - r0;
   if (n <= DC_L) {
     pdl_wait();
     return;
   }
   const int chunks = (n + DC_L - 1) / DC_L;
-  const int kh = h / (a.H / a.G), C = 2 * a.G * dk + a.H * dv;
   const int cols = min(DC_B, dv - c0);
   const size_t first = (size_t)dc_first_chunk(a.cu_q, seq) * a.H + h;
-  const int per = DC_L * (2 * ld + DC_B + 2);  // a staged chunk: W, K [64][ld], U [64][16], the two factors [64]
-  float* Ss = dc_smem + a.stages * per;        // [16][ld]: the state's columns
-  float* Vs = Ss + DC_B * ld;                  // [64][20]: r_(last,t) u_t
-  float* part = Vs + DC_L * 20;                // [64][20]: the sums of the second half of the key dims
-  const bool wide = dk % 4 == 0 && C % 4 == 0, wide_u = dv % 4 == 0;
+  const int per = DC_L * (2 * ld + DC_B);  // a staged chunk: W, r k [64][ld] each, U [64][16]
+  float* Ss = dc_smem + a.stages * per;    // [16][ld]: the state's columns
+  float* part = Ss + DC_B * ld;            // sums of parts: [8][64][20] in the first product, [8][16][32] in the second
   pdl_wait();
-  auto issue = [&](int c) {
-    float* ws = dc_smem + (c % a.stages) * per;
-    float* ks = ws + DC_L * ld;
-    float* us = ks + DC_L * ld;
+  auto issue = [&](int c, float* ws) {
     const size_t at = first + (size_t)c * a.H;
-    const int t0 = r0 + c * DC_L, tn = min(DC_L, n - c * DC_L);
-    dc_stage(ws, ld, a.w + at * DC_L * dk, dk, DC_L, dk, wide, DC_L, tid, DC_B_THREADS);
-    dc_stage(ks, ld, a.qkv + (size_t)t0 * C + (size_t)(a.G + kh) * dk, C, tn, dk, wide, DC_L, tid, DC_B_THREADS);
-    dc_stage(us, DC_B, a.u + at * DC_L * dv + c0, dv, DC_L, cols, wide_u, DC_L, tid, DC_B_THREADS);
-    if (tid < DC_L / 2) dr_copy(us + DC_L * DC_B + 4 * tid, a.coef + at * 2 * DC_L + 4 * tid, true);
+    dc_stage_flat<DC_B_THREADS>(ws, a.wk + at * 2 * DC_L * ld, 2 * DC_L * ld);
+    dc_stage_flat<DC_B_THREADS>(ws + 2 * DC_L * ld, a.u + at * DC_L * a.dvp + (size_t)c0 * DC_L, DC_L * DC_B);
     asm volatile("cp.async.commit_group;\n" ::);
   };
-  issue(0);
+  issue(0, dc_smem);
   float* st = a.state + (((size_t)a.slots[seq] * a.H + h) * dv + c0) * dk;
   const bool read = a.ctx_lens[seq] - n > 0;
-  for (int idx = tid; idx < DC_B * ld; idx += DC_B_THREADS) {
-    const int c = idx / ld, d = idx - c * ld;
-    Ss[idx] = (read && c < cols && d < dk) ? __ldcg(st + (size_t)c * dk + d) : 0.f;
-  }
-  const int grp = tid >> 6, cg = tid & 3, rg = (tid & 63) >> 2;  // first product: half of the key dims, columns, rows
-  const int d_half = (ld - 4) / 2;
+  for (int j = tid >> 5; j < DC_B; j += DC_B_THREADS / 32)
+    for (int d = tid & 31; d < ld; d += 32)
+      Ss[j * ld + d] = (read && j < cols && d < dk) ? __ldcg(st + (size_t)j * dk + d) : 0.f;
+  // first product: a warp has an eighth of the key dims, its lanes rows rg + 8 i and columns cg + 4 j
+  const int warp = tid >> 5, cg = tid & 3, rg = (tid & 31) >> 2;
+  const int eighth = ((ld - 4) / 4 + 7) / 8 * 4, d0 = min(warp * eighth, ld - 4), d1 = min(d0 + eighth, ld - 4);
+  // second product: a warp covers 32 key dims x 16 columns (tiles of four x four) and a part of the rows
+  const int dims = (ld - 4 + 31) / 32;
+  const int parts = dims == 1 ? 8 : dims == 2 ? 4 : dims <= 4 ? 2 : 1;
+  const int tpart = warp / dims, trows = DC_L / parts;
+  const int td = (warp - tpart * dims) * 32 + (tid & 7) * 4, tj = ((tid >> 3) & 3) * 4;
   for (int c = 0; c < chunks; ++c) {
+    float* ws = dc_smem + (a.stages > 1 ? (c & 1) * per : 0);
     if (a.stages > 1 && c + 1 < chunks) {
-      issue(c + 1);
+      issue(c + 1, dc_smem + ((c + 1) & 1) * per);
       asm volatile("cp.async.wait_group 1;\n" ::);
     } else {
       asm volatile("cp.async.wait_group 0;\n" ::);
     }
     __syncthreads();
-    const float* ws = dc_smem + (c % a.stages) * per;
     const float* ks = ws + DC_L * ld;
-    float* us = dc_smem + (c % a.stages) * per + 2 * DC_L * ld;
-    const float* gam = us + DC_L * DC_B;  // G_t, then r_(last,t)
+    float* us = ws + 2 * DC_L * ld;
     const size_t at = first + (size_t)c * a.H;
-    float* s0 = a.s0 + (at * dv + c0) * dk;
-    if (dk % 4 == 0) {
-      for (int idx = tid; idx < cols * (dk / 4); idx += DC_B_THREADS) {
-        const int j = idx / (dk / 4), d = (idx - j * (dk / 4)) * 4;
-        *reinterpret_cast<float4*>(s0 + (size_t)j * dk + d) = *reinterpret_cast<const float4*>(Ss + j * ld + d);
-      }
-    } else {
-      for (int idx = tid; idx < cols * dk; idx += DC_B_THREADS) {
-        const int j = idx / dk, d = idx - j * dk;
-        s0[(size_t)j * dk + d] = Ss[j * ld + d];
-      }
-    }
-    float acc[4][4];
+    const float whole = __ldg(a.g + at * DC_L + DC_L - 1);
+    dc_store_flat<DC_B_THREADS>(a.s0 + (at * a.dvp + c0) * ld, Ss, DC_B * ld);
+    float acc[8][4];
 #pragma unroll
-    for (int i = 0; i < 4; ++i)
+    for (int i = 0; i < 8; ++i)
 #pragma unroll
       for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
-    {
-      const float* wp = ws + rg * ld + grp * d_half;
-      const float* sp = Ss + cg * ld + grp * d_half;
-#pragma unroll 2
-      for (int d = 0; d < d_half; d += 4) {
-        float4 w[4], s[4];
+    for (int d = d0; d < d1; d += 4) {
+      float4 s[4];
 #pragma unroll
-        for (int i = 0; i < 4; ++i) w[i] = *reinterpret_cast<const float4*>(wp + 16 * i * ld + d);
+      for (int j = 0; j < 4; ++j) s[j] = *reinterpret_cast<const float4*>(Ss + (cg + 4 * j) * ld + d);
 #pragma unroll
-        for (int j = 0; j < 4; ++j) s[j] = *reinterpret_cast<const float4*>(sp + 4 * j * ld + d);
-#pragma unroll
-        for (int i = 0; i < 4; ++i)
-#pragma unroll
-          for (int j = 0; j < 4; ++j) {
-            acc[i][j] = fmaf(w[i].x, s[j].x, acc[i][j]);
-            acc[i][j] = fmaf(w[i].y, s[j].y, acc[i][j]);
-            acc[i][j] = fmaf(w[i].z, s[j].z, acc[i][j]);
-            acc[i][j] = fmaf(w[i].w, s[j].w, acc[i][j]);
-          }
-      }
-    }
-    if (grp == 1) {
-#pragma unroll
-      for (int i = 0; i < 4; ++i)
-#pragma unroll
-        for (int j = 0; j < 4; ++j) part[(rg + 16 * i) * 20 + cg + 4 * j] = acc[i][j];
-    }
-    __syncthreads();
-    if (grp == 0) {
-#pragma unroll
-      for (int i = 0; i < 4; ++i) {
-        const int t = rg + 16 * i;
-        const float rho = gam[DC_L + t];
+      for (int i = 0; i < 8; ++i) {
+        const float4 w = *reinterpret_cast<const float4*>(ws + (rg + 8 * i) * ld + d);
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
-          const int cc = cg + 4 * j;
-          const float u = us[t * DC_B + cc] - (acc[i][j] + part[t * 20 + cc]);
-          us[t * DC_B + cc] = u;
-          Vs[t * 20 + cc] = rho * u;
+          acc[i][j] = fmaf(w.x, s[j].x, acc[i][j]);
+          acc[i][j] = fmaf(w.y, s[j].y, acc[i][j]);
+          acc[i][j] = fmaf(w.z, s[j].z, acc[i][j]);
+          acc[i][j] = fmaf(w.w, s[j].w, acc[i][j]);
         }
       }
     }
+#pragma unroll
+    for (int i = 0; i < 8; ++i)
+#pragma unroll
+      for (int j = 0; j < 4; ++j) part[(warp * DC_L + rg + 8 * i) * 20 + cg + 4 * j] = acc[i][j];
     __syncthreads();
     {
-      float* ug = a.u + at * DC_L * dv + c0;
-      for (int idx = tid; idx < DC_L * cols; idx += DC_B_THREADS) {
-        const int t = idx / cols, cc = idx - t * cols;
-        ug[(size_t)t * dv + cc] = us[t * DC_B + cc];
+      const int t = tid >> 2, q = 4 * (tid & 3);
+      float4 u = *reinterpret_cast<const float4*>(us + t * DC_B + q);
+#pragma unroll
+      for (int g = 0; g < 8; ++g) {
+        const float4 v = *reinterpret_cast<const float4*>(part + (g * DC_L + t) * 20 + q);
+        u.x -= v.x; u.y -= v.y; u.z -= v.z; u.w -= v.w;
       }
+      *reinterpret_cast<float4*>(us + t * DC_B + q) = u;
     }
-    const float whole = gam[DC_L - 1];
-    // the next state: tiles of four key dims x four columns
-    for (int tile = tid; tile < (ld - 4 + 31) / 32 * 32; tile += DC_B_THREADS) {
-      const int d = (tile >> 5) * 32 + (tile & 7) * 4, j0 = ((tile >> 3) & 3) * 4;  // a warp: 32 dims x 16 columns
-      if (d >= ld - 4) continue;
+    __syncthreads();
+    dc_store_flat<DC_B_THREADS>(a.u + at * DC_L * a.dvp + (size_t)c0 * DC_L, us, DC_L * DC_B);
+    if (tpart < parts) {
       float s[4][4];  // [column][dim]
 #pragma unroll
       for (int j = 0; j < 4; ++j)
 #pragma unroll
         for (int e = 0; e < 4; ++e) s[j][e] = 0.f;
-#pragma unroll 4
-      for (int t = 0; t < DC_L; ++t) {
-        const float4 k = *reinterpret_cast<const float4*>(ks + t * ld + d);
-        const float4 v = *reinterpret_cast<const float4*>(Vs + t * 20 + j0);
+      const float* kp = ks + tpart * trows * ld + min(td, ld - 4);  // (dims beyond the row's: the zeros behind it)
+      const float* up = us + tpart * trows * DC_B + tj;
+#pragma unroll 8
+      for (int t = 0; t < trows; ++t, kp += ld, up += DC_B) {
+        const float4 k = *reinterpret_cast<const float4*>(kp);
+        const float4 v = *reinterpret_cast<const float4*>(up);
         const float vv[4] = {v.x, v.y, v.z, v.w};
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
@@ -695,24 +799,30 @@ __global__ void __launch_bounds__(DC_B_THREADS) delta_chunk_states_kernel(const 
         }
       }
 #pragma unroll
-      for (int j = 0; j < 4; ++j) {
-        float4* p = reinterpret_cast<float4*>(Ss + (j0 + j) * ld + d);
-        const float4 o = *p;
-        *p = make_float4(fmaf(whole, o.x, s[j][0]), fmaf(whole, o.y, s[j][1]), fmaf(whole, o.z, s[j][2]),
-                         fmaf(whole, o.w, s[j][3]));
+      for (int j = 0; j < 4; ++j) store4<float>(part + (warp * DC_B + tj + j) * 32 + (tid & 7) * 4, s[j]);
+    }
+    __syncthreads();
+    for (int b = tid >> 7; b < dims; b += 2) {
+      const int j = (tid >> 3) & 15, d = b * 32 + (tid & 7) * 4;
+      if (d >= ld - 4) continue;
+      float4* p = reinterpret_cast<float4*>(Ss + j * ld + d);
+      float4 o = *p;
+      o.x *= whole; o.y *= whole; o.z *= whole; o.w *= whole;
+      for (int g = 0; g < parts; ++g) {
+        const float4 v = *reinterpret_cast<const float4*>(part + ((g * dims + b) * DC_B + j) * 32 + (tid & 7) * 4);
+        o.x += v.x; o.y += v.y; o.z += v.z; o.w += v.w;
       }
+      *p = o;
     }
     __syncthreads();  // the state is whole, and the staged chunk is free
-    if (a.stages == 1 && c + 1 < chunks) issue(c + 1);
+    if (a.stages == 1 && c + 1 < chunks) issue(c + 1, dc_smem);
   }
-  for (int idx = tid; idx < cols * dk; idx += DC_B_THREADS) {
-    const int c = idx / dk, d = idx - c * dk;
-    st[(size_t)c * dk + d] = Ss[c * ld + d];
-  }
+  for (int j = tid >> 5; j < cols; j += DC_B_THREADS / 32)
+    for (int d = tid & 31; d < dk; d += 32) st[(size_t)j * dk + d] = Ss[j * ld + d];
 }
 
 // ---- launch C
-__global__ void __launch_bounds__(DC_THREADS) delta_chunk_outputs_kernel(const DeltaChunks a) {
+__global__ void __launch_bounds__(DC_THREADS, 3) delta_chunk_outputs_kernel(const DeltaChunks a) {
   extern __shared__ __align__(16) float dc_smem[];
   pdl_trigger();
   const int slices = (a.dv + DC_N - 1) / DC_N;
@@ -724,14 +834,14 @@ __global__ void __launch_bounds__(DC_THREADS) delta_chunk_outputs_kernel(const D
     return;
   }
   const size_t at = (size_t)(dc_first_chunk(a.cu_q, seq) + c) * a.H + h;
-  const int dk = a.dk, dv = a.dv, ld = a.ldk, tid = threadIdx.x;
+  const int dk = a.dk, dv = a.dv, ld = a.ld, tid = threadIdx.x;
   const int kh = h / (a.H / a.G), C = 2 * a.G * dk + a.H * dv;
-  const int t0 = r0 + c * DC_L, tn = min(DC_L, n - c * DC_L), cols = min(DC_N, dv - c0);
-  float* qs = dc_smem;            // [64][ld]; then P [64][68]
-  float* ss = qs + DC_L * ld;     // [64][ld]: columns of the state; then u [64][68]
+  const int t0 = r0 + c * DC_L, tn = min(DC_L, n - c * DC_L), cols = min(DC_N, a.dvp - c0);
+  float* qs = dc_smem;            // [64][ld]; then P [64][DC_LDP]
+  float* ss = qs + DC_L * ld;     // [64][ld]: columns of the state; then u, up to four slices of [64][16]
   pdl_wait();
-  dc_stage(qs, ld, a.qkv + (size_t)t0 * C + (size_t)kh * dk, C, tn, dk, dk % 4 == 0 && C % 4 == 0, DC_L, tid, DC_THREADS);
-  dc_stage(ss, ld, a.s0 + (at * dv + c0) * dk, dk, cols, dk, dk % 4 == 0, DC_N, tid, DC_THREADS);
+  dc_stage(qs, ld, a.qkv + (size_t)t0 * C + (size_t)kh * dk, C, tn, dk, dk % 4 == 0 && C % 4 == 0);
+  dc_stage_flat<DC_THREADS>(ss, a.s0 + (at * a.dvp + c0) * ld, cols * ld);
   asm volatile("cp.async.commit_group;\n" ::);
   asm volatile("cp.async.wait_group 0;\n" ::);
   __syncthreads();
@@ -741,6 +851,7 @@ __global__ void __launch_bounds__(DC_THREADS) delta_chunk_outputs_kernel(const D
   for (int i = 0; i < 4; ++i)
 #pragma unroll
     for (int j = 0; j < 4; ++j) acc[i][j] = 0.f;
+  // (columns beyond `cols` read what lies there: their sums are never stored)
 #pragma unroll 2
   for (int d = 0; d < ld - 4; d += 4) {
     float4 q[4], s[4];
@@ -760,13 +871,13 @@ __global__ void __launch_bounds__(DC_THREADS) delta_chunk_outputs_kernel(const D
   }
   __syncthreads();
   float* ps = dc_smem;
-  float* us = ps + DC_L * 68;
-  dc_stage(ps, 68, a.p + at * DC_L * DC_L, DC_L, DC_L, DC_L, true, DC_L, tid, DC_THREADS);
-  dc_stage(us, 68, a.u + at * DC_L * dv + c0, dv, DC_L, cols, dv % 4 == 0, DC_L, tid, DC_THREADS);
+  float* us = ps + DC_L * DC_LDP;
+  dc_stage_flat<DC_THREADS>(ps, a.p + at * DC_L * DC_LDP, DC_L * DC_LDP);
+  dc_stage_flat<DC_THREADS>(us, a.u + at * DC_L * a.dvp + (size_t)c0 * DC_L, cols * DC_L);
   asm volatile("cp.async.commit_group;\n" ::);
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
-    const float g = __ldg(a.coef + at * 2 * DC_L + ty + 16 * i);
+    const float g = __ldg(a.g + at * DC_L + ty + 16 * i);
 #pragma unroll
     for (int j = 0; j < 4; ++j) acc[i][j] *= g;
   }
@@ -780,10 +891,10 @@ __global__ void __launch_bounds__(DC_THREADS) delta_chunk_outputs_kernel(const D
 #pragma unroll
       for (int e = 0; e < 4; ++e)
 #pragma unroll
-        for (int j = 0; j < 4; ++j) u[e][j] = us[(s + e) * 68 + tx + 16 * j];
+        for (int j = 0; j < 4; ++j) u[e][j] = us[(j * DC_L + s + e) * DC_B + tx];
 #pragma unroll
       for (int i = b; i < 4; ++i) {
-        const float4 p = *reinterpret_cast<const float4*>(ps + (ty + 16 * i) * 68 + s);
+        const float4 p = *reinterpret_cast<const float4*>(ps + (ty + 16 * i) * DC_LDP + s);
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           acc[i][j] = fmaf(p.x, u[0][j], acc[i][j]);
@@ -800,7 +911,7 @@ __global__ void __launch_bounds__(DC_THREADS) delta_chunk_outputs_kernel(const D
     if (t >= tn) continue;
 #pragma unroll
     for (int j = 0; j < 4; ++j)
-      if (tx + 16 * j < cols)
+      if (c0 + tx + 16 * j < dv)
         a.out[(size_t)(t0 + t) * ((size_t)a.H * dv) + (size_t)h * dv + c0 + tx + 16 * j] = acc[i][j];
   }
 }
@@ -831,7 +942,29 @@ extern "C" int lse_delta_inputs(const float* proj, long long stride, const float
   // 16-byte accesses: every head starts on one in the projection, the taps, the kept inputs and the result
   const bool vec = dk % 4 == 0 && dv % 4 == 0 && stride % 4 == 0 && aligned(proj) && aligned(conv) &&
                    aligned(conv_state) && aligned(qkv);
-  launch(vec ? delta_inputs_kernel<4> : delta_inputs_kernel<1>, grid, DI_WARPS * 32, 0, stream, a);
+  const size_t smem = (size_t)DI_WARPS * (a.rows + taps - 1) * (2 * dk > dv ? 2 * dk : dv) * sizeof(float);
+  const bool staged = vec && a.rows > 1 && smem <= 96 * 1024;
+#define LSE_DI_LAUNCH(KERNEL, BYTES)                                                                              \
+  do {                                                                                                            \
+    if ((BYTES) > 48 * 1024 &&                                                                                    \
+        cudaFuncSetAttribute(KERNEL, cudaFuncAttributeMaxDynamicSharedMemorySize, 96 * 1024) != cudaSuccess)      \
+      return LSE_LAUNCH_FAILED;                                                                                   \
+    launch(KERNEL, grid, DI_WARPS * 32, BYTES, stream, a);                                                        \
+  } while (0)
+#define LSE_DI(TAPS)                                                          \
+  do {                                                                        \
+    if (staged && dk <= 128) LSE_DI_LAUNCH((delta_inputs_kernel<4, TAPS, 1, true>), smem); \
+    else if (staged) LSE_DI_LAUNCH((delta_inputs_kernel<4, TAPS, 2, true>), smem);         \
+    else if (vec && dk <= 128) LSE_DI_LAUNCH((delta_inputs_kernel<4, TAPS, 1, false>), 0); \
+    else if (vec) LSE_DI_LAUNCH((delta_inputs_kernel<4, TAPS, 2, false>), 0);              \
+    else LSE_DI_LAUNCH((delta_inputs_kernel<1, TAPS, 8, false>), 0);                       \
+  } while (0)
+  if (taps == 4) LSE_DI(4);
+  else if (taps == 3) LSE_DI(3);
+  else if (taps == 2) LSE_DI(2);
+  else LSE_DI(0);
+#undef LSE_DI
+#undef LSE_DI_LAUNCH
   return LSE_CHECK_LAUNCH();
 }
 
@@ -852,7 +985,8 @@ static int launch_delta_rule(const DeltaRule& a, int num_seqs, cudaStream_t stre
 
 // Floats of scratch that one chunk of a portion longer than DC_L tokens needs.
 static size_t chunk_floats(int H, int dk, int dv) {
-  return (size_t)H * (DC_L * (size_t)(dk + dv + DC_L + 2) + (size_t)dv * dk);
+  const size_t ld = (dk + 15) / 16 * 16 + 4, dvp = (dv + DC_B - 1) / DC_B * DC_B;
+  return (size_t)H * (DC_L * (2 * ld + dvp + DC_LDP + 1) + dvp * ld);
 }
 
 extern "C" int lse_delta_rule_chunk(void) { return DC_L; }
@@ -871,26 +1005,28 @@ static int launch_delta_chunks(const DeltaRule& r, int num_seqs, int max_chunks,
   DeltaChunks a;
   a.qkv = r.qkv; a.scal = r.scal; a.state = r.state; a.out = r.out; a.cu_q = r.cu_q; a.ctx_lens = r.ctx_lens;
   a.slots = r.slots; a.H = r.H; a.G = r.G; a.dk = r.dk; a.dv = r.dv;
-  a.ldk = (r.dk + 7) / 8 * 8 + 4;
+  a.ld = (r.dk + 15) / 16 * 16 + 4;
+  a.dvp = (r.dv + DC_B - 1) / DC_B * DC_B;
   const size_t units = (size_t)total_chunks * r.H;
-  // the parts that are read as 16-byte vectors whatever the sizes are come first
-  a.coef = scratch;
-  a.p = a.coef + units * 2 * DC_L;
-  a.w = a.p + units * DC_L * DC_L;
-  a.u = a.w + units * DC_L * r.dk;
-  a.s0 = a.u + units * DC_L * r.dv;
+  a.g = scratch;
+  a.p = a.g + units * DC_L;
+  a.u = a.p + units * DC_L * DC_LDP;
+  a.wk = a.u + units * DC_L * a.dvp;
+  a.s0 = a.wk + units * 2 * DC_L * a.ld;
   if (r.H > 65535 || max_chunks > 65535) return LSE_BAD_ARGUMENT;
-  const size_t smem_a = (size_t)(2 * DC_L * a.ldk + DC_L * 68 + 3 * DC_L) * sizeof(float);
-  const size_t per = (size_t)DC_L * (2 * a.ldk + DC_B + 2), rest = (size_t)DC_B * a.ldk + 2 * DC_L * 20;
+  const size_t smem_a =
+      (size_t)(DC_L * a.ld + DC_L * (a.ld > a.dvp ? a.ld : a.dvp) + DC_L * DC_LDP + 4 * DC_L) * sizeof(float);
+  const size_t per = (size_t)DC_L * (2 * a.ld + DC_B), rest = (size_t)DC_B * a.ld + 8 * DC_L * 20;
   a.stages = (2 * per + rest) * sizeof(float) <= 227 * 1024 ? 2 : 1;
   const size_t smem_b = (a.stages * per + rest) * sizeof(float);
-  size_t smem_c = (size_t)2 * DC_L * a.ldk * sizeof(float);
-  if (smem_c < (size_t)2 * DC_L * 68 * sizeof(float)) smem_c = (size_t)2 * DC_L * 68 * sizeof(float);
+  size_t smem_c = (size_t)2 * DC_L * a.ld * sizeof(float);
+  const size_t second = (size_t)DC_L * (DC_LDP + DC_N) * sizeof(float);  // what the second product stages in the same place
+  if (smem_c < second) smem_c = second;
   if (!allow_smem(delta_chunk_systems_kernel, smem_a) || !allow_smem(delta_chunk_states_kernel, smem_b) ||
       !allow_smem(delta_chunk_outputs_kernel, smem_c))
     return LSE_LAUNCH_FAILED;
   launch(delta_chunk_systems_kernel, dim3(max_chunks, r.H, num_seqs), DC_THREADS, smem_a, stream, a);
-  launch(delta_chunk_states_kernel, dim3(r.H * ((r.dv + DC_B - 1) / DC_B), num_seqs), DC_B_THREADS, smem_b, stream, a);
+  launch(delta_chunk_states_kernel, dim3(r.H * (a.dvp / DC_B), num_seqs), DC_B_THREADS, smem_b, stream, a);
   const int slices = r.H * ((r.dv + DC_N - 1) / DC_N);
   if (slices > 65535) return LSE_BAD_ARGUMENT;
   launch(delta_chunk_outputs_kernel, dim3(max_chunks, slices, num_seqs), DC_THREADS, smem_c, stream, a);
