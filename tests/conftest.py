@@ -488,3 +488,132 @@ def write_lanilorn(folder, name):
 @pytest.fixture(scope="session")
 def lanilorn_dirs(tmp_path_factory):
     return {name: write_lanilorn(tmp_path_factory.mktemp(f"lanilorn-{name}"), name) for name in LANILORN_TINY}
+
+
+# ----------------------------------------------------------------------------- Miberax
+def _mib(left, right, mlp):
+    """left: (heads, kv_heads, dim, vdim, scale, chunk, rot or None); right: (heads, kv_heads, dim, vdim, conv)."""
+    h, g, d, v, scale, chunk, rot = left
+    m = {"heads": h, "kv_heads": g, "dim": d, "vdim": v, "scale": scale}
+    if chunk:
+        m["mask"] = {"size": chunk}
+    if rot:
+        base, dims, factor = rot
+        m["rot"] = {"base": base, "dims": dims}
+        if factor != 1.0:
+            m["rot"]["scaling"] = {"factor": factor}
+    return {"type": "parallel", "mlp": mlp, "mixer": {
+        "left": m, "right": dict(zip(("heads", "kv_heads", "dim", "vdim", "conv"), right))}}
+
+
+def _gmoe(experts, top, ff, limit, scale, groups=None, identity=0, shared=None):
+    router = {"experts": experts, "top": top, "scale": scale}
+    if groups:
+        router["groups"] = {"count": groups[0], "keep": groups[1]}
+    if identity:
+        router["identity"] = identity
+    d = {"kind": "moe", "router": router, "expert": {"ff": ff, "limit": limit}}
+    if shared:
+        d["shared"] = {"ff": shared[0], "limit": shared[1]}
+    return d
+
+
+MIBERAX_TINY = {
+    # values wider than keys on the left, narrower on the right; a third of each head rotated; a chunk
+    # that is no multiple of the page; grouped key heads on both sides; groups of experts of which
+    # some are kept; an identity expert; a layer without feed-forward
+    "M1": dict(seed=5, page_tokens=16, config={
+        "architecture": "Miberax", "vocab": 163, "width": 96, "norm": {"eps": 1e-5, "groups": 4},
+        "layers": [_mib((4, 2, 24, 40, 0.3, 21, (10000.0, 8, 2.0)), (4, 2, 32, 16, 4), _dense(112)),
+                   _mib((3, 1, 32, 16, 0.25, 40, (500.0, 32, 8.0)), (2, 1, 16, 40, 2),
+                        _gmoe(5, 2, 24, 0.8, 1.5, groups=(3, 2), identity=1, shared=(40, 1.3))),
+                   _mib((2, 2, 16, 16, 0.35, 16, (50.0, 16, 1.0)), (3, 3, 24, 24, 3), None)]}),
+    # sizes that are multiples of nothing; norms of whole rows; a chunk shorter than a page and one of a
+    # single token; a convolution of one tap and one of five; no rotation; no shared expert; every
+    # expert chosen; one group of one expert each; several identity experts
+    "M2": dict(seed=12, page_tokens=8, config={
+        "architecture": "Miberax", "vocab": 131, "width": 70, "norm": {"eps": 1e-6, "groups": 1},
+        "layers": [_mib((3, 3, 18, 10, 0.3, 5, (300.0, 6, 3.0)), (5, 1, 10, 14, 1), _gmoe(4, 4, 10, 0.5, 0.7)),
+                   _mib((2, 1, 20, 12, 0.3, 1, None), (2, 2, 22, 9, 5), _dense(50)),
+                   _mib((5, 1, 12, 12, 0.4, 33, (1000.0, 12, 4.0)), (3, 1, 7, 20, 3),
+                        _gmoe(5, 3, 14, 2.0, 3.0, groups=(8, 4), identity=3, shared=(12, 0.4)))]}),
+    # the head sizes of larger models; chunks of one and of several pages; attention without a mask; a wide
+    # key of the delta rule; norms of two parts; many experts in groups
+    "M3": dict(seed=20, page_tokens=32, sharp=5, config={
+        "architecture": "Miberax", "vocab": 300, "width": 128, "norm": {"eps": 1e-5, "groups": 2},
+        "layers": [_mib((8, 2, 64, 64, 0.125, 32, (20000.0, 64, 4.0)), (2, 2, 128, 64, 4), _dense(192)),
+                   _mib((4, 4, 32, 48, 0.2, 0, (10000.0, 16, 1.0)), (4, 1, 64, 64, 4),
+                        _gmoe(14, 3, 48, 1.1, 2.2, groups=(4, 2), identity=2, shared=(64, 0.9))),
+                   _mib((2, 1, 48, 32, 0.2, 96, (700.0, 24, 2.0)), (1, 1, 160, 32, 2), _dense(80))]}),
+}
+
+
+def write_miberax(folder, name):
+    """A random folder whose attention is sharp, whose decays, step sizes and convolutions differ clearly
+    from head to head and channel to channel, and whose norms and coefficients are drawn wide, so that
+    leaving one of them out, a key too many or a lost state changes the logits clearly.
+
+    No routing decision is a close call (a model computed in bfloat16 must pick the same experts as the
+    float64 one): the last dims of the residual stream carry, for every token, one of evenly spaced
+    levels per expert, in an order that depends on the token; no layer writes those dims, and each
+    router row reads its expert's dim beside small random weights on all the others. (An identity
+    expert hands those dims on and so stretches them, which leaves the gaps between levels wide.)"""
+    from safetensors.torch import load_file, save_file
+
+    from llmserve_b200.config.miberax import MiberaxConfig
+    from llmserve_b200.weights import write_random_model
+
+    spec = MIBERAX_TINY[name]
+    write_random_model(folder, MiberaxConfig.from_dict(spec["config"]), spec["seed"])
+    f = folder / "model.safetensors"
+    t = load_file(str(f))
+    g = torch.Generator().manual_seed(spec["seed"] + 1)
+    for k, v in t.items():
+        r = torch.rand(v.shape, generator=g)
+        if k.endswith("A_log"):
+            t[k] = (2.5 * r - 2.0).to(v.dtype)
+        elif k.endswith("dt_bias"):
+            t[k] = (4 * r - 4.0).to(v.dtype)
+        elif k.endswith(".conv"):
+            t[k] = (1.6 * r - 0.5).to(v.dtype)
+        elif k.endswith("mlp.act"):
+            t[k] = (1.4 * (r - 0.3)).to(v.dtype)
+        elif v.dim() == 1:  # norm weights (and the correction, set below)
+            t[k] = (0.5 + r).to(v.dtype)
+        elif k == "embed":
+            t[k] = (v.float() * 40).to(v.dtype)
+        elif k.endswith(("left.q", "left.k")):
+            t[k] = (v.float() * spec.get("sharp", 10)).to(v.dtype)
+        elif k.endswith(("right.a", "right.b")):
+            t[k] = (v.float() * 15).to(v.dtype)
+        else:
+            t[k] = (v.float() * 8).to(v.dtype)
+    cfg = spec["config"]
+    width = cfg["width"]
+    moe = [(i, l["mlp"]["router"]) for i, l in enumerate(cfg["layers"]) if l["mlp"] and l["mlp"]["kind"] == "moe"]
+    counts = [r["experts"] + r.get("identity", 0) for _, r in moe]
+    most = max(counts)
+    step = next(m for m in (3, 5, 7, 11) if all(most % q or m % q for q in (2, 3, 5, 7, 11)))
+    dims = [width - most + e for e in range(most)]
+    tok = torch.arange(cfg["vocab"])[:, None]
+    levels = 1.5 * (((tok * 7 + step * torch.arange(most)[None, :]) % most).float() - (most - 1) / 2)
+    t["embed"][:, dims] = levels.to(t["embed"].dtype)
+    for k in t:
+        if k.endswith("down"):
+            t[k][dims, :] = 0
+        elif k.endswith((".left.out", ".right.out")):
+            t[k][dims] = 0
+    for (i, r), n in zip(moe, counts):
+        t[f"l{i}.norm2"][dims] = 1
+        router = torch.randn(n, width, generator=g) * 0.002
+        router[torch.arange(n), dims[:n]] = 0.8
+        t[f"l{i}.mlp.router"] = router.to(torch.bfloat16)
+        # a correction that moves a choice here and there: below the gap between two scores where it counts
+        t[f"l{i}.mlp.correction"] = (0.01 * (torch.rand(n, generator=g) - 0.5)).to(torch.bfloat16)
+    save_file(t, str(f))
+    return folder
+
+
+@pytest.fixture(scope="session")
+def miberax_dirs(tmp_path_factory):
+    return {name: write_miberax(tmp_path_factory.mktemp(f"miberax-{name}"), name) for name in MIBERAX_TINY}
