@@ -21,16 +21,14 @@ namespace lse {
 // ------------------------------------------------------------------------------------ inputs
 // Columns of a row of the projection, from its column 0: q (G heads of dk) | k (G of dk) | v (H of dv)
 // | gate (H of dv) | b (H) | a (H). One warp per (`rows` neighbouring rows, job): G jobs that make a key
-// head's q and k and the numbers of its value heads, then H jobs that make a value head's v. With
-// several rows a warp finds the inputs that neighbouring rows share in its SM's cache.
+// head's q and k and the numbers of its value heads, then H jobs that make a value head's v.
 //
 // The convolution of row i of a portion reads rows i - taps + 1 .. i, the first taps - 1 rows also
 // the inputs kept from the step before (state [slots, taps - 1, channels], oldest first). The warp
 // of a portion's row 0 makes all of these first rows and then writes the new state of its
-// channels, so nobody else touches them. V channels per lane and visit, at most NK visits for a
-// key head. TAPS:
-// the number of taps (0: any; their inputs are then fetched one after another). STAGED: the inputs of
-// all rows of the warp are fetched together into shared memory.
+// channels, so nobody else touches them. V channels per lane and visit, at most NK visits for a key
+// head. TAPS: the number of taps (0: any; their inputs are then fetched one after another). STAGED:
+// the inputs of all rows of the warp are fetched together into shared memory.
 constexpr int DI_WARPS = 4, DI_MAX = 256;  // DI_MAX: largest key size
 
 struct DeltaInputs {
@@ -430,6 +428,7 @@ __global__ void __launch_bounds__(DR_THREADS) delta_rule_kernel(const DeltaRule 
 // factors in (0, 1], so nothing overflows. A chunk that is not full is filled up with tokens of
 // g = 1, beta = 0 and zero vectors.
 constexpr int DC_L = 64, DC_THREADS = 256, DC_B = 16, DC_B_THREADS = 256, DC_N = 64;
+constexpr int DC_MAX_DV = 512;  // value sizes whose rows fit launch A's shared memory; longer ones run token by token
 
 struct DeltaChunks {
   const float* qkv;    // as DeltaRule
@@ -992,10 +991,13 @@ static size_t chunk_floats(int H, int dk, int dv) {
 extern "C" int lse_delta_rule_chunk(void) { return DC_L; }
 extern "C" size_t lse_delta_rule_chunk_floats(int H, int dk, int dv) { return chunk_floats(H, dk, dv); }
 
-template <typename K>
-static bool allow_smem(K kernel, size_t bytes) {
-  return bytes <= 48 * 1024 ||
-         cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes) == cudaSuccess;
+template <auto KERNEL>
+static bool allow_smem(size_t bytes) {
+  static size_t allowed = 48 * 1024;
+  if (bytes <= allowed) return true;
+  if (cudaFuncSetAttribute(KERNEL, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes) != cudaSuccess) return false;
+  allowed = bytes;
+  return true;
 }
 
 // The portions of more than DC_L tokens: max_chunks bounds the chunks of any sequence, total_chunks
@@ -1022,8 +1024,8 @@ static int launch_delta_chunks(const DeltaRule& r, int num_seqs, int max_chunks,
   size_t smem_c = (size_t)2 * DC_L * a.ld * sizeof(float);
   const size_t second = (size_t)DC_L * (DC_LDP + DC_N) * sizeof(float);  // what the second product stages in the same place
   if (smem_c < second) smem_c = second;
-  if (!allow_smem(delta_chunk_systems_kernel, smem_a) || !allow_smem(delta_chunk_states_kernel, smem_b) ||
-      !allow_smem(delta_chunk_outputs_kernel, smem_c))
+  if (!allow_smem<delta_chunk_systems_kernel>(smem_a) || !allow_smem<delta_chunk_states_kernel>(smem_b) ||
+      !allow_smem<delta_chunk_outputs_kernel>(smem_c))
     return LSE_LAUNCH_FAILED;
   launch(delta_chunk_systems_kernel, dim3(max_chunks, r.H, num_seqs), DC_THREADS, smem_a, stream, a);
   launch(delta_chunk_states_kernel, dim3(r.H * (a.dvp / DC_B), num_seqs), DC_B_THREADS, smem_b, stream, a);
@@ -1042,8 +1044,9 @@ extern "C" int lse_delta_rule(const float* qkv, const float* scal, float* state,
   DeltaRule a;
   a.qkv = qkv; a.scal = reinterpret_cast<const float4*>(scal); a.state = state; a.out = out; a.cu_q = cu_q;
   a.ctx_lens = ctx_lens; a.slots = slots; a.H = H; a.G = G; a.dk = dk; a.dv = dv;
-  a.longest = max_chunks > 1 ? DC_L : 0;
-  if (max_chunks > 1) {
+  const bool chunked = max_chunks > 1 && dv <= DC_MAX_DV;
+  a.longest = chunked ? DC_L : 0;
+  if (chunked) {
     const int code = launch_delta_chunks(a, num_seqs, max_chunks, scratch, total_chunks, stream);
     if (code != LSE_OK || !short_too) return code;
   }

@@ -237,7 +237,7 @@ def delta_plain(c, proj, before, S0):
     return o.reshape(n, H * dv), x[x.shape[0] - (c.taps - 1) :], S.transpose(1, 2)
 
 
-SIZES = [(4, 2, 64, 32, 4), (3, 3, 20, 12, 3), (2, 1, 128, 128, 4), (1, 1, 256, 40, 2), (5, 5, 16, 24, 1), (2, 2, 48, 72, 5),
+SIZES = [(1, 1, 16, 520, 2), (4, 2, 64, 32, 4), (3, 3, 20, 12, 3), (2, 1, 128, 128, 4), (1, 1, 256, 40, 2), (5, 5, 16, 24, 1), (2, 2, 48, 72, 5),
          (4, 4, 12, 10, 4), (3, 1, 7, 9, 4), (2, 1, 132, 136, 4), (1, 1, 64, 256, 3)]
 
 
