@@ -132,6 +132,18 @@ def _register_builtin() -> None:
             checkpoint_layout=miberax_checkpoint_layout,
         )
     )
+    from ..models.tanupel import tanupel_checkpoint_layout, tanupel_plan
+    from .tanupel import TanupelConfig
+
+    register_architecture(
+        Architecture(
+            name="Tanupel",
+            model_type="tanupel",
+            config_cls=TanupelConfig,
+            plan=tanupel_plan,
+            checkpoint_layout=tanupel_checkpoint_layout,
+        )
+    )
 
 
 _register_builtin()

@@ -107,7 +107,8 @@ __device__ __forceinline__ float head_factor(const LseAttnArgs& a, int head) {
 constexpr int SIMT_QT = 32;
 constexpr int SIMT_KT = (D <= 128) ? 32 : 16;
 
-template <typename T>
+// CAP (here and in the single-token kernels): the scores are soft-capped
+template <typename T, bool CAP>
 __global__ void __launch_bounds__(128) prefill_simt_kernel(const LseAttnArgs a, int page_shift) {
   constexpr int QT = SIMT_QT, KT = SIMT_KT, DPT = D / 4, VEC = Num<T>::kVec, NCHUNK = D / VEC;
   __shared__ float ks[KT][D];
@@ -140,6 +141,7 @@ __global__ void __launch_bounds__(128) prefill_simt_kernel(const LseAttnArgs a, 
   const T* kp = (const T*)a.k_pages;
   const T* vp = (const T*)a.v_pages;
   const int kept = kept_keys(a, k_first);
+  const SoftCap softcap(CAP ? a.softcap : 0.f);
   const int kept_tiles_end = (kept + KT - 1) / KT * KT, window_tile = (k_first / KT) * KT;
 
   for (int k0 = kept > 0 ? 0 : window_tile; k0 < k_end; k0 = next_tile(k0, KT, kept_tiles_end, window_tile)) {
@@ -175,6 +177,7 @@ __global__ void __launch_bounds__(128) prefill_simt_kernel(const LseAttnArgs a, 
       for (int i = 0; i < DPT; ++i) d = fmaf(qreg[i], ks[jj][sub + 4 * i], d);
       d += __shfl_xor_sync(0xffffffffu, d, 1);
       d += __shfl_xor_sync(0xffffffffu, d, 2);
+      if constexpr (CAP) d = softcap(d);
       const int j = k0 + jj;
       const bool ok = row_valid && j <= qpos && (j >= q_first || j < a.keep_first);
       s[jj] = ok ? d - slope * (float)(qpos - j) : -INFINITY;
@@ -288,8 +291,10 @@ __global__ void __launch_bounds__(MMA_THREADS, (LSE_HEAD_DIM <= 64 ? 2 : 1)) pre
   float m_r[2] = {-INFINITY, -INFINITY}, l_r[2] = {0.f, 0.f};
   // With score options the scores are finished (factor, distance penalty) when they are masked,
   // and only the change to base 2 is left to the exponent's multiply-add.
-  const bool options = a.head_scale || a.slopes || a.chunk > 0 || a.sinks || a.keep_first > 0;
+  const bool options = a.head_scale || a.slopes || a.chunk > 0 || a.sinks || a.keep_first > 0 || a.softcap > 0.f;
+  const SoftCap softcap(a.softcap);
   const float qk_factor = head_factor(a, head);
+  const float finish = a.softcap > 0.f ? 1.f : qk_factor;  // (a capped score is a finished one)
   const float slope = a.slopes ? a.slopes[head] : 0.f;
   const int kept = kept_keys(a, k_first);
   const int kept_tiles_end = (kept + KT - 1) / KT * KT;
@@ -348,6 +353,12 @@ __global__ void __launch_bounds__(MMA_THREADS, (LSE_HEAD_DIM <= 64 ? 2 : 1)) pre
         mma_bf16(s[nb + 1], qf[kk], b[2], b[3]);
       }
     }
+    if (a.softcap > 0.f) {
+#pragma unroll
+      for (int nb = 0; nb < NB; ++nb)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) s[nb][e] = softcap(s[nb][e] * qk_factor);
+    }
     // running maximum; only tiles on the diagonal, at a window's edge or at the context's start
     // need the per-element mask (rows past the portion compute garbage that is never stored)
     const bool full_tile = !options && k0 >= k_first && k0 + KT - 1 <= qmin_w &&
@@ -366,7 +377,7 @@ __global__ void __launch_bounds__(MMA_THREADS, (LSE_HEAD_DIM <= 64 ? 2 : 1)) pre
           const int rr = e >> 1;
           const int j = k0 + nb * 8 + t4 * 2 + (e & 1);
           const bool ok = valid_r[rr] && j <= qpos_r[rr] && (j >= qfirst_r[rr] || j < a.keep_first);
-          const float sc = options ? s[nb][e] * qk_factor - slope * (float)(qpos_r[rr] - j) : s[nb][e];
+          const float sc = options ? s[nb][e] * finish - slope * (float)(qpos_r[rr] - j) : s[nb][e];
           s[nb][e] = ok ? sc : -INFINITY;
           tmax[rr] = fmaxf(tmax[rr], s[nb][e]);
         }
@@ -521,7 +532,7 @@ __device__ __noinline__ void merge_partitions(const float* __restrict__ parts, i
   }
 }
 
-template <typename T, int GT>
+template <typename T, int GT, bool CAP>
 __global__ void __launch_bounds__(DEC_WARPS * 32)
 decode_split_kernel(const LseAttnArgs a, int page_shift) {
   using S = DecodeShape<T>;
@@ -581,6 +592,7 @@ decode_split_kernel(const LseAttnArgs a, int page_shift) {
     }
   }
 
+  const SoftCap softcap(CAP ? a.softcap : 0.f);
   // U passes of the warp are in flight together: all their loads are issued before any arithmetic.
   constexpr int U = (GT * CPL <= 2) ? 4 : 2;
   for (int j0 = lo + warp * KPI; j0 < hi; j0 += DEC_WARPS * KPI * U) {
@@ -623,6 +635,7 @@ decode_split_kernel(const LseAttnArgs a, int page_shift) {
             d[u] = fmaf(qreg[gq][c][e], Num<T>::to_float(kv[u][c].v[e]), d[u]);
 #pragma unroll
         for (int o = LPK / 2; o > 0; o >>= 1) d[u] += __shfl_xor_sync(0xffffffffu, d[u], o);
+        if constexpr (CAP) d[u] = softcap(d[u]);
         d[u] -= slope[gq] * (float)(ctx - 1 - key_of(j0 + u * DEC_WARPS * KPI + slot));  // the distance penalty
         if (ok[u]) m_new = fmaxf(m_new, d[u]);  // ok is uniform over the LPK lanes of a key
       }
@@ -756,6 +769,7 @@ decode_split_kernel(const LseAttnArgs a, int page_shift) {
 // in the kernel above.
 constexpr int DM_HEADS = 16;
 
+template <bool CAP>
 __global__ void __launch_bounds__(DEC_WARPS * 32)
 decode_mma_kernel(const LseAttnArgs a, int page_shift) {
   using T = bf16;
@@ -775,6 +789,8 @@ decode_mma_kernel(const LseAttnArgs a, int page_shift) {
   const int lo = k_first + split * per;
   const int hi = min(ctx, lo + per);
 
+  const SoftCap softcap(CAP ? a.softcap : 0.f);
+  auto score = [&](float qk) { return CAP ? softcap(qk * a.scale) : qk * a.scale; };
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, t = lane & 3;
   const int* table = a.block_tables + (size_t)seq * a.table_stride;
@@ -868,7 +884,7 @@ decode_mma_kernel(const LseAttnArgs a, int page_shift) {
           const bool ok = key >= lo && key < hi;
 #pragma unroll
           for (int r = 0; r < 2; ++r) {
-            const float v = ok ? sc[nt][2 * r + e] * a.scale : -INFINITY;
+            const float v = ok ? score(sc[nt][2 * r + e]) : -INFINITY;
             sc[nt][2 * r + e] = v;
             mx[r] = fmaxf(mx[r], v);
           }
@@ -999,7 +1015,7 @@ __device__ __forceinline__ uint32_t movmatrix_trans(uint32_t x) {
 // from shared memory (the tile loop stops one key earlier); the block that finishes last for a
 // (sequence, key/value head) clears the sums it stands for. This saves the
 // rotation kernel between the projection and the attention of a step of single tokens.
-template <bool EARLY, bool FUSED>
+template <bool EARLY, bool FUSED, bool CAP>
 __global__ void __launch_bounds__(DEC_WARPS * 32, EARLY ? 4 : ((FUSED && D == 64) ? 7 : 0))  // 0: the compiler's own choice
 // (head size 64: 72 registers, 7 blocks per SM; the form that makes its own queries needs the promise to stay there)
 decode_mma8_kernel(const LseAttnArgs a, int page_shift) {
@@ -1029,6 +1045,8 @@ decode_mma8_kernel(const LseAttnArgs a, int page_shift) {
   const bool owns_new = FUSED && hi_all == ctx && hi_all > lo;
   const int hi = owns_new ? hi_all - 1 : hi_all;  // keys [lo, hi) come from the pages
 
+  const SoftCap softcap(CAP ? a.softcap : 0.f);
+  auto score = [&](float qk) { return CAP ? softcap(qk * a.scale) : qk * a.scale; };
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, t = lane & 3;
   const int* table = a.block_tables + (size_t)seq * a.table_stride;
@@ -1217,8 +1235,8 @@ decode_mma8_kernel(const LseAttnArgs a, int page_shift) {
       float corr[2], p[2][2];
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
-        const float s0 = ok0 ? sc[e] * a.scale : -INFINITY;
-        const float s1 = ok1 ? sc[2 + e] * a.scale : -INFINITY;
+        const float s0 = ok0 ? score(sc[e]) : -INFINITY;
+        const float s1 = ok1 ? score(sc[2 + e]) : -INFINITY;
         float mx = fmaxf(m_run[e], fmaxf(s0, s1));
         mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 4));
         mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 8));
@@ -1271,7 +1289,7 @@ decode_mma8_kernel(const LseAttnArgs a, int page_shift) {
     for (int e = 0; e < 2; ++e) {
       const int head = 2 * t + e;
       const float of_head = __shfl_sync(0xffffffffu, dot, 4 * head);
-      const float sc_new = head < G ? of_head * a.scale : -INFINITY;
+      const float sc_new = head < G ? score(of_head) : -INFINITY;
       const float mx = fmaxf(m_run[e], sc_new);
       const float m_fin = (mx == -INFINITY) ? 0.f : mx;
       corr[e] = Exp<T>::f(m_run[e] - m_fin);
@@ -1408,7 +1426,7 @@ __device__ __forceinline__ uint32_t piece(int r, int c) {
 
 // PER: tiles in flight per warp. Every warp is its own producer: lane 0 asks for the warp's tile
 // k + PER into the slot that tile k has just been read from, so no warp waits for another.
-template <int PER>
+template <int PER, bool CAP>
 __global__ void __launch_bounds__(DEC_WARPS * 32)
 decode_ring_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                    const LseAttnArgs a, int page_shift) {
@@ -1441,6 +1459,8 @@ decode_ring_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
   const int first_tile = lo >> 4;
   const int n_tiles = hi > lo ? ((hi - 1) >> 4) - first_tile + 1 : 0;
 
+  const SoftCap softcap(CAP ? a.softcap : 0.f);
+  auto score = [&](float qk) { return CAP ? softcap(qk * a.scale) : qk * a.scale; };
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int g = lane >> 2, t = lane & 3;
   const int n_mine = n_tiles > warp ? (n_tiles - warp + DEC_WARPS - 1) / DEC_WARPS : 0;  // tiles warp, warp + 4, ...
@@ -1550,8 +1570,8 @@ decode_ring_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_const
     float corr[2], p[2][2];
 #pragma unroll
     for (int e = 0; e < 2; ++e) {
-      const float s0 = ok0 ? sc[e] * a.scale : -INFINITY;
-      const float s1 = ok1 ? sc[2 + e] * a.scale : -INFINITY;
+      const float s0 = ok0 ? score(sc[e]) : -INFINITY;
+      const float s1 = ok1 ? score(sc[2 + e]) : -INFINITY;
       float mx = fmaxf(m_run[e], fmaxf(s0, s1));
       mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 4));
       mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 8));
@@ -1660,7 +1680,7 @@ static int shift_of(int n) {
 static bool args_ok(const LseAttnArgs* a) {
   return a && (a->dtype == LSE_F32 || a->dtype == LSE_BF16) && a->num_heads > 0 &&
          a->num_kv_heads > 0 && a->num_heads % a->num_kv_heads == 0 && a->page_tokens > 0 &&
-         a->window >= 0 && a->chunk >= 0 && a->keep_first >= 0 && !(a->keep_first > 0 && a->chunk > 0) &&
+         a->window >= 0 && a->chunk >= 0 && a->keep_first >= 0 && a->softcap >= 0.f && !(a->keep_first > 0 && a->chunk > 0) &&
          (a->q || a->qkv_sums) && a->out && a->k_pages && a->v_pages && a->block_tables &&
          a->ctx_lens && a->cu_q && (a->out_f32 == 0 || (a->out_f32 == 1 && !a->qkv_sums));
 }
@@ -1669,6 +1689,8 @@ template <typename T>
 static int launch_decode(const LseAttnArgs* a, cudaStream_t stream) {
   const int G = a->num_heads / a->num_kv_heads;
   const int ps = shift_of(a->page_tokens);
+  const bool cap = a->softcap > 0.f;
+  if (cap && a->qkv_sums) return LSE_BAD_ARGUMENT;  // (the form that makes its own queries has no cap)
   // served by the CUDA-core kernel only (sinks: also by the tensor-core kernel for groups of up to 8)
   const bool options = a->head_scale || a->slopes || a->chunk > 0 || ((a->sinks || a->out_f32) && G > 8) ||
                        (a->keep_first > 0 && a->window > 0);
@@ -1706,7 +1728,9 @@ static int launch_decode(const LseAttnArgs* a, cudaStream_t stream) {
       constexpr int smem = PER * DEC_WARPS * 2 * ring::TILE_BYTES + 1024;
       static bool configured = false;
       if (!configured) {
-        if (cudaFuncSetAttribute(decode_ring_kernel<PER>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+        if (cudaFuncSetAttribute(decode_ring_kernel<PER, false>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                 smem) != cudaSuccess ||
+            cudaFuncSetAttribute(decode_ring_kernel<PER, true>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                  smem) != cudaSuccess)
           return LSE_LAUNCH_FAILED;
         configured = true;
@@ -1715,22 +1739,22 @@ static int launch_decode(const LseAttnArgs* a, cudaStream_t stream) {
       if (!tma::make_map_bf16(&mk, a->k_pages, pool_rows, D, D, 16) ||
           !tma::make_map_bf16(&mv, a->v_pages, pool_rows, D, D, 16))
         return LSE_LAUNCH_FAILED;
-      launch(decode_ring_kernel<PER>, mgrid, DEC_WARPS * 32, smem, stream, mk, mv, *a, ps);
+      launch(cap ? decode_ring_kernel<PER, true> : decode_ring_kernel<PER, false>, mgrid, DEC_WARPS * 32, smem, stream, mk, mv, *a, ps);
       return cudaPeekAtLastError() == cudaSuccess ? LSE_OK : LSE_LAUNCH_FAILED;
     }
     if (G <= 8) {
       // a grid that leaves the SMs part empty can afford the registers of an early first tile
       const bool small = blocks <= 4LL * sms;
       if (a->qkv_sums) {
-        if (small) launch(decode_mma8_kernel<true, true>, mgrid, DEC_WARPS * 32, 0, stream, *a, ps);
-        else launch(decode_mma8_kernel<false, true>, mgrid, DEC_WARPS * 32, 0, stream, *a, ps);
+        if (small) launch(decode_mma8_kernel<true, true, false>, mgrid, DEC_WARPS * 32, 0, stream, *a, ps);
+        else launch(decode_mma8_kernel<false, true, false>, mgrid, DEC_WARPS * 32, 0, stream, *a, ps);
       } else {
-        if (small) launch(decode_mma8_kernel<true, false>, mgrid, DEC_WARPS * 32, 0, stream, *a, ps);
-        else launch(decode_mma8_kernel<false, false>, mgrid, DEC_WARPS * 32, 0, stream, *a, ps);
+        if (small) launch(cap ? decode_mma8_kernel<true, false, true> : decode_mma8_kernel<true, false, false>, mgrid, DEC_WARPS * 32, 0, stream, *a, ps);
+        else launch(cap ? decode_mma8_kernel<false, false, true> : decode_mma8_kernel<false, false, false>, mgrid, DEC_WARPS * 32, 0, stream, *a, ps);
       }
     }
 #if LSE_HEAD_DIM == 64
-    else launch(decode_mma_kernel, mgrid, DEC_WARPS * 32, 0, stream, *a, ps);
+    else launch(cap ? decode_mma_kernel<true> : decode_mma_kernel<false>, mgrid, DEC_WARPS * 32, 0, stream, *a, ps);
 #endif
     return cudaPeekAtLastError() == cudaSuccess ? LSE_OK : LSE_LAUNCH_FAILED;
   }
@@ -1741,9 +1765,9 @@ static int launch_decode(const LseAttnArgs* a, cudaStream_t stream) {
   if (grid.y > 65535 || grid.z > 65535) return LSE_BAD_ARGUMENT;
   if (a->num_splits > 1 && (size_t)grid.y * grid.z > (size_t)LSE_ATTN_COUNTERS) return LSE_BAD_ARGUMENT;
   if (a->num_splits > MERGE_SPLITS) return LSE_BAD_ARGUMENT;
-  if (gt == 1) launch(decode_split_kernel<T, 1>, grid, DEC_WARPS * 32, 0, stream, *a, ps);
-  else if (gt == 2) launch(decode_split_kernel<T, 2>, grid, DEC_WARPS * 32, 0, stream, *a, ps);
-  else launch(decode_split_kernel<T, 4>, grid, DEC_WARPS * 32, 0, stream, *a, ps);
+  if (gt == 1) launch(cap ? decode_split_kernel<T, 1, true> : decode_split_kernel<T, 1, false>, grid, DEC_WARPS * 32, 0, stream, *a, ps);
+  else if (gt == 2) launch(cap ? decode_split_kernel<T, 2, true> : decode_split_kernel<T, 2, false>, grid, DEC_WARPS * 32, 0, stream, *a, ps);
+  else launch(cap ? decode_split_kernel<T, 4, true> : decode_split_kernel<T, 4, false>, grid, DEC_WARPS * 32, 0, stream, *a, ps);
   return cudaPeekAtLastError() == cudaSuccess ? LSE_OK : LSE_LAUNCH_FAILED;
 }
 
@@ -1778,17 +1802,17 @@ extern "C" int lse_attn_decode_blocks_per_sm(int dtype, int num_heads, int num_k
   if (num_heads <= 0 || num_kv_heads <= 0 || num_heads % num_kv_heads) return 0;
   const int G = num_heads / num_kv_heads;
 #if LSE_HEAD_DIM == 64 || LSE_HEAD_DIM == 128
-  if (dtype == LSE_BF16 && G <= 8) return blocks_per_sm(decode_mma8_kernel<false, false>);
+  if (dtype == LSE_BF16 && G <= 8) return blocks_per_sm(decode_mma8_kernel<false, false, false>);
 #endif
 #if LSE_HEAD_DIM == 64
-  if (dtype == LSE_BF16 && G <= 16) return blocks_per_sm(decode_mma_kernel);
+  if (dtype == LSE_BF16 && G <= 16) return blocks_per_sm(decode_mma_kernel<false>);
 #endif
   const int gt = G == 1 ? 1 : (G == 2 ? 2 : 4);
   if (dtype == LSE_BF16)
-    return gt == 1 ? blocks_per_sm(decode_split_kernel<bf16, 1>)
-                   : gt == 2 ? blocks_per_sm(decode_split_kernel<bf16, 2>) : blocks_per_sm(decode_split_kernel<bf16, 4>);
-  return gt == 1 ? blocks_per_sm(decode_split_kernel<float, 1>)
-                 : gt == 2 ? blocks_per_sm(decode_split_kernel<float, 2>) : blocks_per_sm(decode_split_kernel<float, 4>);
+    return gt == 1 ? blocks_per_sm(decode_split_kernel<bf16, 1, false>)
+                   : gt == 2 ? blocks_per_sm(decode_split_kernel<bf16, 2, false>) : blocks_per_sm(decode_split_kernel<bf16, 4, false>);
+  return gt == 1 ? blocks_per_sm(decode_split_kernel<float, 1, false>)
+                 : gt == 2 ? blocks_per_sm(decode_split_kernel<float, 2, false>) : blocks_per_sm(decode_split_kernel<float, 4, false>);
 }
 
 extern "C" int lse_attn_decode_takes_sums(int dtype, int num_heads, int num_kv_heads) {
@@ -1806,7 +1830,8 @@ extern "C" int lse_attn_prefill(const LseAttnArgs* a, cudaStream_t stream) {
   const int ps = shift_of(a->page_tokens);
   dim3 grid(a->num_heads, a->num_tiles);
   if (a->dtype == LSE_F32) {
-    prefill_simt_kernel<float><<<grid, 128, 0, stream>>>(*a, ps);
+    if (a->softcap > 0.f) prefill_simt_kernel<float, true><<<grid, 128, 0, stream>>>(*a, ps);
+    else prefill_simt_kernel<float, false><<<grid, 128, 0, stream>>>(*a, ps);
 #if LSE_HEAD_DIM == 64
   } else if (a->force_simt == 0 && a->num_rows > 0 && a->num_pages > 0 && atc::supported(a) &&
              !(a->head_scale || a->slopes || a->chunk > 0 || a->sinks || a->keep_first > 0 || a->out_f32)) {
@@ -1816,7 +1841,8 @@ extern "C" int lse_attn_prefill(const LseAttnArgs* a, cudaStream_t stream) {
 #endif
   } else if (!kHasMma || a->force_simt == 1) {
     // the caller built tiles of SIMT_QT rows in this case
-    prefill_simt_kernel<bf16><<<grid, 128, 0, stream>>>(*a, ps);
+    if (a->softcap > 0.f) prefill_simt_kernel<bf16, true><<<grid, 128, 0, stream>>>(*a, ps);
+    else prefill_simt_kernel<bf16, false><<<grid, 128, 0, stream>>>(*a, ps);
   } else {
 #if LSE_HEAD_DIM <= 128
     constexpr int smem = (MMA_QT + 4 * MMA_KT) * (D + 8) * (int)sizeof(bf16);

@@ -54,7 +54,7 @@ struct LseAttnArgs {
   const float* rope_sin;
   // Options of the score, all off when null / 0. With any of them on, the CUDA-core kernels and
   // the mma.sync kernel for portions serve the call (lse_attn_decode_takes_sums() does not hold).
-  //   s_ij = scale * head_scale[h] * q_i . k_j - slopes[h] * (i - j)
+  //   s_ij = softcap(scale * head_scale[h] * q_i . k_j) - slopes[h] * (i - j)
   //   chunk > 0: query i reads key j only if i / chunk == j / chunk (absolute positions)
   const float* head_scale;  // [num_heads] or null
   const float* slopes;      // [num_heads] or null
@@ -71,6 +71,9 @@ struct LseAttnArgs {
   // kernels, the mma.sync kernel for portions and the tensor-core single-token kernel for groups
   // of up to 8 heads.
   int out_f32;
+  //   softcap > 0: the scaled score s becomes softcap * tanh(s / softcap) (before the distance penalty).
+  //   Every kernel serves it, except single tokens straight from qkv_sums.
+  float softcap;
 };
 
 #define LSE_ATTN_COUNTERS 65536  // words at the start of the scratch: one counter per (sequence, head group)

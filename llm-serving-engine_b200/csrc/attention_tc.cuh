@@ -117,6 +117,8 @@ struct Params {
   int* error_flag;
 };
 
+// CAP: the scores are scaled and soft-capped as they leave tensor memory.
+template <bool CAP>
 __global__ void __launch_bounds__(THREADS, 2)
 prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                   const __grid_constant__ CUtensorMap map_v, const Params p) {
@@ -289,7 +291,8 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
     const bool row_valid = r < rows_here;
     const uint32_t lane_base = tmem + ((uint32_t)(wq * 32) << 16);
     const uint32_t o_col = lane_base + COL_O + st * O_COLS;
-    const float sl2 = a.scale * 1.4426950408889634f;
+    const float sl2 = (CAP ? 1.f : a.scale) * 1.4426950408889634f;
+    const lse::SoftCap softcap(CAP ? a.softcap : 0.f);
     float m_run = -INFINITY, l_run = 0.f;
     bool ok = true;
     for (int it = 0; it < n_tiles && !failed; ++it) {
@@ -300,6 +303,10 @@ prefill_tc_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_consta
       uint32_t sv[32];
       tmem_ld32(s_buf, sv);
       asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
+      if constexpr (CAP) {
+#pragma unroll
+        for (int j = 0; j < 32; ++j) sv[j] = __float_as_uint(softcap(__uint_as_float(sv[j]) * a.scale));
+      }
       const int k0 = it * KT + 32 * st;
       // four independent chains for the maximum and for the sum: a single chain of dependent
       // operations would leave the warp waiting on its own results
@@ -430,7 +437,8 @@ inline bool supported(const LseAttnArgs* a) {
 }
 
 // total_rows: rows of the query tensor; pool_rows: pages * kv_heads * page_tokens.
-inline int launch_prefill(const LseAttnArgs* a, long long total_rows, long long pool_rows,
+template <bool CAP>
+inline int launch_prefill_form(const LseAttnArgs* a, long long total_rows, long long pool_rows,
                           int* error_flag, cudaStream_t stream) {
   CUtensorMap mq, mk, mv;
   const int box_rows = a->page_tokens < KT ? a->page_tokens : KT;
@@ -447,15 +455,21 @@ inline int launch_prefill(const LseAttnArgs* a, long long total_rows, long long 
   constexpr int smem = Q_BYTES + 2 * STAGES * KV_BYTES + (2 * STAGES + 9) * 8 + 16 + 1024;
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(prefill_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) !=
+    if (cudaFuncSetAttribute(prefill_tc_kernel<CAP>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) !=
         cudaSuccess)
       return LSE_LAUNCH_FAILED;
     configured = true;
   }
   dim3 grid(a->num_heads, a->num_tiles);
-  return lse::launch(prefill_tc_kernel, grid, THREADS, smem, stream, mq, mk, mv, p) == cudaSuccess
+  return lse::launch(prefill_tc_kernel<CAP>, grid, THREADS, smem, stream, mq, mk, mv, p) == cudaSuccess
              ? LSE_OK
              : LSE_LAUNCH_FAILED;
+}
+
+inline int launch_prefill(const LseAttnArgs* a, long long total_rows, long long pool_rows,
+                          int* error_flag, cudaStream_t stream) {
+  return a->softcap > 0.f ? launch_prefill_form<true>(a, total_rows, pool_rows, error_flag, stream)
+                          : launch_prefill_form<false>(a, total_rows, pool_rows, error_flag, stream);
 }
 
 }  // namespace atc

@@ -76,15 +76,53 @@ void done(int code, const char* what) {
   }
 }
 
-void embedding(const Tensor& ids, const Tensor& table, Tensor& out) {
+void embedding(const Tensor& ids, const Tensor& table, Tensor& out, double scale) {
   check_i32(ids, "ids");
   check_cuda(table, "table");
   check_f32(out, "out");
   TORCH_CHECK(table.dim() == 2 && out.dim() == 2 && ids.dim() == 1, "embedding: bad ranks");
   TORCH_CHECK(out.size(0) == ids.size(0) && out.size(1) == table.size(1), "embedding: bad shapes");
   done(lse_embedding(ids.data_ptr<int>(), table.data_ptr(), dtype_code(table, "table"),
-                     out.data_ptr<float>(), (int)ids.size(0), (int)table.size(1), stream()),
+                     out.data_ptr<float>(), (int)ids.size(0), (int)table.size(1), stream(), (float)scale),
        "embedding");
+}
+
+// x += sum of c[i] * y[i] (float32 tensors or fixed-point sums) + row; with weight also out = norm(x)
+void sum_add_rmsnorm(Tensor& x, const std::vector<Tensor>& y, const std::vector<double>& c, const OptTensor& row,
+                     const OptTensor& weight, double eps, const OptTensor& out) {
+  check_f32(x, "x");
+  TORCH_CHECK(x.dim() == 2 && y.size() == c.size() && y.size() <= 4, "sum_add_rmsnorm: at most four tensors, a factor each");
+  const void* ptrs[4] = {};
+  float factors[4] = {};
+  int codes[4] = {};
+  for (size_t i = 0; i < y.size(); ++i) {
+    check_cuda(y[i], "y");
+    TORCH_CHECK(y[i].sizes() == x.sizes(), "sum_add_rmsnorm: every tensor needs x's shape");
+    codes[i] = dtype_code(y[i], "y");
+    TORCH_CHECK(codes[i] == LSE_F32 || codes[i] == LSE_FIXED64, "sum_add_rmsnorm: float32 tensors or sums");
+    ptrs[i] = y[i].data_ptr();
+    factors[i] = (float)c[i];
+  }
+  const float *rp = nullptr, *wp = nullptr;
+  if (row) {
+    check_f32(*row, "row");
+    TORCH_CHECK(row->numel() == x.size(1), "sum_add_rmsnorm: row needs x's width");
+    rp = row->data_ptr<float>();
+  }
+  void* op = nullptr;
+  int oc = LSE_F32;
+  if (weight) {
+    check_f32(*weight, "weight");
+    TORCH_CHECK(weight->numel() == x.size(1) && out, "sum_add_rmsnorm: weight needs x's width, and an output");
+    wp = weight->data_ptr<float>();
+    check_cuda(*out, "out");
+    TORCH_CHECK(out->sizes() == x.sizes(), "sum_add_rmsnorm: out shape differs from x");
+    op = out->data_ptr();
+    oc = dtype_code(*out, "out");
+  }
+  done(lse_sum_add_rmsnorm(x.data_ptr<float>(), ptrs, factors, codes, (int)y.size(), rp, wp, (float)eps, op, oc,
+                           (int)x.size(0), (int)x.size(1), stream()),
+       "sum_add_rmsnorm");
 }
 
 void add_rmsnorm(Tensor& x, const OptTensor& residual, const Tensor& weight, double eps,
@@ -324,7 +362,8 @@ void paged_attention(const Tensor& q, Tensor& out, const Tensor& k_pages, const 
                      const Tensor& cu_q, const OptTensor& tiles, int64_t num_tiles,
                      const OptTensor& decode_seqs, int64_t num_decode, int64_t num_splits,
                      const OptTensor& scratch, int64_t force_kernel, const OptTensor& head_scale,
-                     const OptTensor& slopes, int64_t chunk, const OptTensor& sinks, int64_t keep_first) {
+                     const OptTensor& slopes, int64_t chunk, const OptTensor& sinks, int64_t keep_first,
+                     double softcap) {
   const AttnLib& lib = attn_lib(D);
   TORCH_CHECK(q.is_cuda() && q.dim() == 2 && q.stride(1) == 1 && q.size(1) >= num_heads * D,
               "paged_attention: q must be [T, >= heads*head_dim] with unit column stride");
@@ -386,6 +425,8 @@ void paged_attention(const Tensor& q, Tensor& out, const Tensor& k_pages, const 
   a.chunk = (int)chunk;
   TORCH_CHECK(keep_first >= 0 && !(keep_first > 0 && chunk > 0), "paged_attention: keep_first must not be negative, and not with chunks");
   a.keep_first = (int)keep_first;
+  TORCH_CHECK(softcap >= 0, "paged_attention: softcap must not be negative");
+  a.softcap = (float)softcap;
   if (sinks) {
     check_f32(*sinks, "sinks");
     TORCH_CHECK(sinks->numel() == num_heads, "paged_attention: sinks needs one value per head");
@@ -511,7 +552,7 @@ void head_linear(const Tensor& a, int64_t col0, const Tensor& w, Tensor& out, in
 
 void moe_route(const Tensor& h, const Tensor& router, int64_t E, int64_t top, Tensor& idx, Tensor& wts,
                const OptTensor& gate, const OptTensor& bias, int64_t mode, int64_t groups, int64_t keep,
-               double scale) {
+               double scale, bool normalise) {
   check_cuda(h, "h");
   check_f32(router, "router");
   check_i32(idx, "idx");
@@ -529,7 +570,8 @@ void moe_route(const Tensor& h, const Tensor& router, int64_t E, int64_t top, Te
   }
   done(lse_moe_route(h.data_ptr(), out_code(h, "h"), router.data_ptr<float>(), (int)T, (int)W, (int)E,
                      has_gate, (int)top, idx.data_ptr<int>(), wts.data_ptr<float>(), g, stream(),
-                     opt_f32(bias, E, "router bias"), (int)mode, (int)groups, (int)keep, (float)scale),
+                     opt_f32(bias, E, "router bias"), (int)mode, (int)groups, (int)keep, (float)scale,
+                     normalise ? 1 : 0),
        "moe_route");
 }
 
@@ -603,7 +645,7 @@ void expert_linear(const Tensor& a, const Tensor& w, Tensor& out, const Tensor& 
 
 void moe_combine(const Tensor& y, const Tensor& work, int64_t E, int64_t top, const OptTensor& shared_out,
                  const OptTensor& gate, Tensor& out, bool accumulate, const OptTensor& wts,
-                 const OptTensor& h) {
+                 const OptTensor& h, double scale) {
   check_f32(y, "y");
   check_i32(work, "work");
   check_f32(out, "out");
@@ -630,7 +672,7 @@ void moe_combine(const Tensor& y, const Tensor& work, int64_t E, int64_t top, co
   }
   done(lse_moe_combine(y.data_ptr<float>(), work.data_ptr<int>() + E + 1 + n, (int)top, sp, gp,
                        out.data_ptr<float>(), accumulate ? 1 : 0, (int)T, (int)W, stream(), opt_f32(wts, n, "experts' weights"),
-                       hp, hc),
+                       hp, hc, (float)scale),
        "moe_combine");
 }
 
@@ -639,6 +681,16 @@ void cast_f32(const Tensor& x, Tensor& out) {
   check_cuda(out, "out");
   TORCH_CHECK(out.numel() == x.numel(), "cast: sizes differ");
   done(lse_cast(x.data_ptr<float>(), out.data_ptr(), out_code(out, "out"), x.numel(), stream()), "cast");
+}
+
+void cast_columns(const Tensor& x, int64_t col0, Tensor& out) {
+  check_f32(x, "x");
+  check_cuda(out, "out");
+  TORCH_CHECK(x.dim() == 2 && out.dim() == 2 && out.size(0) == x.size(0) && col0 >= 0 && col0 + out.size(1) <= x.size(1),
+              "cast_columns: out must be [T, columns of x from col0 on]");
+  done(lse_cast_columns(x.data_ptr<float>() + col0, x.size(1), out.data_ptr(), out_code(out, "out"), (int)out.size(0),
+                        (int)out.size(1), stream()),
+       "cast_columns");
 }
 
 void token_shift(const Tensor& x, const Tensor& mix, Tensor& state, Tensor& out, const Tensor& token_seq,
@@ -788,7 +840,7 @@ void norm_rope_kv_write(const Tensor& qkv, Tensor& q_out, int64_t nq, int64_t nk
 void delta_inputs(const Tensor& proj, int64_t col0, const Tensor& conv, const OptTensor& conv_state, const Tensor& A_log,
                   const Tensor& dt_bias, const Tensor& token_seq, const Tensor& cu_q, const Tensor& ctx_lens,
                   const Tensor& slots, Tensor& qkv, Tensor& scal, int64_t H, int64_t G, int64_t dk, int64_t dv,
-                  double q_scale) {
+                  double q_scale, const OptTensor& z, const OptTensor& decay) {
   check_f32(proj, "proj");
   check_f32(conv, "conv");
   check_f32(A_log, "A_log");
@@ -801,9 +853,22 @@ void delta_inputs(const Tensor& proj, int64_t col0, const Tensor& conv, const Op
   check_f32(scal, "scal");
   TORCH_CHECK(H > 0 && G > 0 && H % G == 0 && dk > 0 && dk <= 256 && dv > 0, "delta_inputs: bad head counts or sizes");
   const int64_t T = proj.size(0), C = 2 * G * dk + H * dv;
-  TORCH_CHECK(proj.dim() == 2 && col0 >= 0 && col0 + C + H * dv + 2 * H <= proj.size(1), "delta_inputs: columns outside proj");
+  TORCH_CHECK(proj.dim() == 2 && col0 >= 0 && col0 + C + (z ? H : H * dv + 2 * H) <= proj.size(1),
+              "delta_inputs: columns outside proj");
   TORCH_CHECK(conv.dim() == 2 && conv.size(0) >= 1 && conv.size(1) == C, "delta_inputs: conv must be [taps, channels]");
-  TORCH_CHECK(A_log.numel() == H && dt_bias.numel() == H, "delta_inputs: one A_log and dt_bias per head");
+  TORCH_CHECK(A_log.numel() == H && dt_bias.numel() == (z ? H * dk : H),
+              "delta_inputs: one A_log per head, one dt_bias per decay");
+  const float* zp = nullptr;
+  float* dp = nullptr;
+  if (z) {
+    check_f32(*z, "z");
+    TORCH_CHECK(decay.has_value(), "delta_inputs: decays per channel need their output");
+    check_f32(*decay, "decay");
+    TORCH_CHECK(z->dim() == 2 && z->size(0) == T && z->size(1) >= H * dk && decay->numel() == T * H * dk,
+                "delta_inputs: z must be [T, >= heads * key_dim], decay [T, heads * key_dim]");
+    zp = z->data_ptr<float>();
+    dp = decay->data_ptr<float>();
+  }
   TORCH_CHECK(qkv.dim() == 2 && qkv.size(0) == T && qkv.size(1) == C && scal.numel() == T * H * 4,
               "delta_inputs: qkv must be [T, channels], scal [T, heads, 4]");
   TORCH_CHECK(token_seq.numel() >= T && cu_q.numel() == ctx_lens.numel() + 1 && slots.numel() >= ctx_lens.numel(),
@@ -820,13 +885,13 @@ void delta_inputs(const Tensor& proj, int64_t col0, const Tensor& conv, const Op
   done(lse_delta_inputs(proj.data_ptr<float>() + col0, proj.size(1), conv.data_ptr<float>(), (int)taps, st,
                         A_log.data_ptr<float>(), dt_bias.data_ptr<float>(), token_seq.data_ptr<int>(), cu_q.data_ptr<int>(),
                         ctx_lens.data_ptr<int>(), slots.data_ptr<int>(), qkv.data_ptr<float>(), scal.data_ptr<float>(),
-                        (int)T, (int)H, (int)G, (int)dk, (int)dv, (float)q_scale, stream()),
+                        (int)T, (int)H, (int)G, (int)dk, (int)dv, (float)q_scale, stream(), zp, z ? (long long)z->size(1) : 0, dp),
        "delta_inputs");
 }
 
 void delta_rule(const Tensor& qkv, const Tensor& scal, Tensor& state, Tensor& out, const Tensor& cu_q,
                 const Tensor& ctx_lens, const Tensor& slots, int64_t H, int64_t G, int64_t dk, int64_t dv,
-                int64_t max_chunks, const OptTensor& scratch, bool short_too) {
+                int64_t max_chunks, const OptTensor& scratch, bool short_too, const OptTensor& decay) {
   check_f32(qkv, "qkv");
   check_f32(scal, "scal");
   check_state(state, "state", dk);
@@ -843,6 +908,12 @@ void delta_rule(const Tensor& qkv, const Tensor& scal, Tensor& state, Tensor& ou
               "delta_rule: state must be [slots, heads, value_dim, key_dim]");
   TORCH_CHECK(cu_q.numel() == ctx_lens.numel() + 1 && slots.numel() >= ctx_lens.numel(),
               "delta_rule: per-sequence arrays disagree");
+  const float* dp = nullptr;
+  if (decay) {
+    check_f32(*decay, "decay");
+    TORCH_CHECK(decay->numel() == T * H * dk, "delta_rule: decay must be [T, heads * key_dim]");
+    dp = decay->data_ptr<float>();
+  }
   float* sp = nullptr;
   int64_t total = 0;
   if (max_chunks > 1) {
@@ -850,13 +921,13 @@ void delta_rule(const Tensor& qkv, const Tensor& scal, Tensor& state, Tensor& ou
     total = T / lse_delta_rule_chunk() + ctx_lens.numel();
     TORCH_CHECK(scratch.has_value(), "delta_rule: long portions need the scratch");
     check_f32(*scratch, "scratch");
-    TORCH_CHECK(scratch->numel() >= total * (int64_t)lse_delta_rule_chunk_floats((int)H, (int)dk, (int)dv),
+    TORCH_CHECK(scratch->numel() >= total * (int64_t)lse_delta_rule_chunk_floats((int)H, (int)dk, (int)dv, decay ? 1 : 0),
                 "delta_rule: the scratch is too small");
     sp = scratch->data_ptr<float>();
   }
   done(lse_delta_rule(qkv.data_ptr<float>(), scal.data_ptr<float>(), state.data_ptr<float>(), out.data_ptr<float>(),
                       cu_q.data_ptr<int>(), ctx_lens.data_ptr<int>(), slots.data_ptr<int>(), (int)ctx_lens.numel(),
-                      (int)H, (int)G, (int)dk, (int)dv, stream(), (int)max_chunks, sp, (int)total, short_too ? 1 : 0),
+                      (int)H, (int)G, (int)dk, (int)dv, stream(), (int)max_chunks, sp, (int)total, short_too ? 1 : 0, dp),
        "delta_rule");
 }
 
@@ -1335,7 +1406,8 @@ void differential_combine(const Tensor& a, const Tensor& gate, int64_t gate_col0
 }
 
 PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
-  m.def("embedding", &embedding);
+  m.def("embedding", &embedding, py::arg("ids"), py::arg("table"), py::arg("out"), py::arg("scale") = 1.0);
+  m.def("sum_add_rmsnorm", &sum_add_rmsnorm);
   m.def("add_rmsnorm", &add_rmsnorm, py::arg("x"), py::arg("residual"), py::arg("weight"), py::arg("eps"),
         py::arg("out"), py::arg("rows"), py::arg("groups") = 1);
   m.def("rope_kv_write", &rope_kv_write);
@@ -1357,7 +1429,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
         py::arg("block_tables"), py::arg("ctx_lens"), py::arg("cu_q"), py::arg("tiles"), py::arg("num_tiles"),
         py::arg("decode_seqs"), py::arg("num_decode"), py::arg("num_splits"), py::arg("scratch"),
         py::arg("force_kernel"), py::arg("head_scale"), py::arg("slopes"), py::arg("chunk"),
-        py::arg("sinks") = py::none(), py::arg("keep_first") = 0);
+        py::arg("sinks") = py::none(), py::arg("keep_first") = 0, py::arg("softcap") = 0.0);
   m.def("hashed_pair_add", &hashed_pair_add);
   m.def("sinusoid_add", &sinusoid_add);
   m.def("latent_write", &latent_write);
@@ -1365,31 +1437,36 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
         py::arg("a_head_cols") = 0, py::arg("out_head_cols") = 0);
   m.def("moe_route", &moe_route, py::arg("h"), py::arg("router"), py::arg("num_experts"), py::arg("top"),
         py::arg("idx"), py::arg("wts"), py::arg("gate"), py::arg("bias") = py::none(), py::arg("mode") = 0,
-        py::arg("groups") = 1, py::arg("keep") = 1, py::arg("scale") = 1.0);
+        py::arg("groups") = 1, py::arg("keep") = 1, py::arg("scale") = 1.0, py::arg("normalise") = true);
   m.def("moe_max_tiles", &moe_max_tiles);
   m.def("moe_tile_rows", &moe_tile_rows);
   m.def("moe_sort", &moe_sort);
   m.def("expert_linear", &expert_linear);
   m.def("moe_combine", &moe_combine, py::arg("y"), py::arg("work"), py::arg("num_experts"), py::arg("top"),
         py::arg("shared_out"), py::arg("gate"), py::arg("out"), py::arg("accumulate"), py::arg("wts") = py::none(),
-        py::arg("h") = py::none());
+        py::arg("h") = py::none(), py::arg("scale") = 1.0);
   m.def("latent_rope_write", &latent_rope_write);
   m.def("latent_query_rope", &latent_query_rope);
   m.def("sigmoid_gate_mul", &sigmoid_gate_mul);
   m.def("act_rows", &act_rows);
   m.def("cast_f32", &cast_f32);
+  m.def("cast_columns", &cast_columns);
   m.def("token_shift", &token_shift);
   m.def("rmsnorm_add", &rmsnorm_add, py::arg("x"), py::arg("a"), py::arg("b"), py::arg("wa"), py::arg("wb"),
         py::arg("ca"), py::arg("cb"), py::arg("eps_in"), py::arg("w"), py::arg("eps"), py::arg("out"),
         py::arg("then_w"), py::arg("then_eps"), py::arg("then_groups") = 1);
-  m.def("delta_inputs", &delta_inputs);
+  m.def("delta_inputs", &delta_inputs, py::arg("proj"), py::arg("col0"), py::arg("conv"), py::arg("conv_state"),
+        py::arg("A_log"), py::arg("dt_bias"), py::arg("token_seq"), py::arg("cu_q"), py::arg("ctx_lens"),
+        py::arg("slots"), py::arg("qkv"), py::arg("scal"), py::arg("H"), py::arg("G"), py::arg("dk"), py::arg("dv"),
+        py::arg("q_scale"), py::arg("z") = py::none(), py::arg("decay") = py::none());
   m.def("delta_rule", &delta_rule, py::arg("qkv"), py::arg("scal"), py::arg("state"), py::arg("out"), py::arg("cu_q"),
         py::arg("ctx_lens"), py::arg("slots"), py::arg("H"), py::arg("G"), py::arg("dk"), py::arg("dv"),
-        py::arg("max_chunks") = 1, py::arg("scratch") = py::none(), py::arg("short_too") = true);
+        py::arg("max_chunks") = 1, py::arg("scratch") = py::none(), py::arg("short_too") = true,
+        py::arg("decay") = py::none());
   m.def("delta_rule_chunk", []() { return (int64_t)lse_delta_rule_chunk(); });
-  m.def("delta_rule_chunk_floats", [](int64_t H, int64_t dk, int64_t dv) {
-    return (int64_t)lse_delta_rule_chunk_floats((int)H, (int)dk, (int)dv);
-  });
+  m.def("delta_rule_chunk_floats", [](int64_t H, int64_t dk, int64_t dv, bool channels) {
+    return (int64_t)lse_delta_rule_chunk_floats((int)H, (int)dk, (int)dv, channels ? 1 : 0);
+  }, py::arg("H"), py::arg("dk"), py::arg("dv"), py::arg("channels") = false);
   m.def("mix_normed", &mix_normed);
   m.def("gated_group_norm", &gated_group_norm);
   m.def("norm_rope_kv_write", &norm_rope_kv_write);

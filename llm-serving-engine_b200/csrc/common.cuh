@@ -125,6 +125,15 @@ __device__ __forceinline__ float block_sum(float v, float* scratch) {
   return warp_sum(t);
 }
 
+// cap * tanh(s / cap) by tanh(y) = 1 - 2 / (1 + e^(2 y)): exact at both ends, an absolute error of a few ulps of cap
+struct SoftCap {
+  float cap, to_exp;  // to_exp: 2 log2(e) / cap
+  __device__ __forceinline__ explicit SoftCap(float c) : cap(c), to_exp(c > 0.f ? 2.8853900817779268f / c : 0.f) {}
+  __device__ __forceinline__ float operator()(float s) const {
+    return fmaf(-2.f * cap, __fdividef(1.f, 1.f + exp2f(s * to_exp)), cap);
+  }
+};
+
 // Page and offset of a token position. page_shift >= 0 when page_tokens is a power of two.
 __device__ __forceinline__ void page_of(int pos, int page_tokens, int page_shift, int& idx, int& off) {
   if (page_shift >= 0) {

@@ -2,11 +2,13 @@
 //
 //   per head, with unit vectors k, q (q also scaled), a decay g and a step size beta per token:
 //   S <- g S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q            S [dk, dv], float32
+//   g is one number per head, or one per head and key channel (row d of S is multiplied by g_d)
 //
 //   delta_inputs   what enters the recurrence, from the projections of a step's tokens: the short
 //                  causal convolution over time per channel (its last inputs kept per request),
 //                  silu, unit norms, the query's factor, beta = sigmoid(b),
-//                  g = exp(-exp(A_log) softplus(a + dt_bias)) and the product k . q
+//                  g = exp(-exp(A_log) softplus(a + dt_bias)) (a, dt_bias and g per head, or per
+//                  head and key channel) and the product k . q
 //   delta_rule     the recurrence
 //
 // All arithmetic is float32. A request's states live in row slots[seq] of [slots, ...] tensors; a
@@ -21,7 +23,9 @@ namespace lse {
 // ------------------------------------------------------------------------------------ inputs
 // Columns of a row of the projection, from its column 0: q (G heads of dk) | k (G of dk) | v (H of dv)
 // | gate (H of dv) | b (H) | a (H). One warp per (`rows` neighbouring rows, job): G jobs that make a key
-// head's q and k and the numbers of its value heads, then H jobs that make a value head's v.
+// head's q and k and the numbers of its value heads, then H jobs that make a value head's v. With
+// decays per channel there is no gate in the row and `a` comes as a tensor of its own (z); H
+// more jobs make a value head's dk decays.
 //
 // The convolution of row i of a portion reads rows i - taps + 1 .. i, the first taps - 1 rows also
 // the inputs kept from the step before (state [slots, taps - 1, channels], oldest first). The warp
@@ -37,17 +41,26 @@ struct DeltaInputs {
   const float* conv;    // [taps, C], C = 2 G dk + H dv; the last row is the current token's
   float* conv_state;    // [slots, taps - 1, C], or null when taps == 1
   const float* A_log;   // [H]
-  const float* dt_bias; // [H]
+  const float* dt_bias; // [H], or [H, dk] beside z
   const int* token_seq;
   const int* cu_q;
   const int* ctx_lens;
   const int* slots;
   float* qkv;           // [T, C]
-  float4* scal;         // [T, H]: (g, beta, k . q, 0)
+  float4* scal;         // [T, H]: (g, beta, k . q, 0); g = 1 beside z
   int T, H, G, dk, dv, taps;
   int rows;             // rows per warp
   float q_scale;
+  int b_col;            // column of b; a, where it is part of the row, is at b_col + H
+  const float* z;       // decays per channel: [T, H dk], rows z_stride apart; null: one decay per head
+  long long z_stride;
+  float* decay;         // [T, H dk], with z
 };
+
+__device__ __forceinline__ float dr_decay(float A, float x) {  // A = exp(A_log)
+  const float softplus = fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)));
+  return expf(-A * softplus);
+}
 
 __device__ __forceinline__ void dr_copy(float* smem, const float* gmem, bool wide) {
   const uint32_t addr = (uint32_t)__cvta_generic_to_shared(smem);
@@ -87,7 +100,24 @@ __global__ void __launch_bounds__(DI_WARPS * 32) delta_inputs_kernel(const Delta
   bool from_zero = a.ctx_lens[seq] - (r1 - r0) == 0;
   float* st = a.conv_state ? a.conv_state + (size_t)a.slots[seq] * past * C : nullptr;
   pdl_wait();
-  if (job >= a.G + a.H) return;
+  if (job >= a.G + a.H) {
+    const int h = job - a.G - a.H;
+    if (!a.z || h >= a.H) return;
+    const float A = expf(a.A_log[h]);  // a value head's decays, channel by channel
+    for (int t = t_begin; t < t_end; ++t) {
+      const float* zp = a.z + (size_t)t * a.z_stride + (size_t)h * a.dk;
+      float* out = a.decay + ((size_t)t * a.H + h) * a.dk;
+      for (int d = d_lane; d < a.dk; d += 32 * V) {
+        float x[V], bias[V];
+        di_load<V>(zp + d, x);
+        di_load<V>(a.dt_bias + (size_t)h * a.dk + d, bias);
+#pragma unroll
+        for (int e = 0; e < V; ++e) x[e] = dr_decay(A, x[e] + bias[e]);
+        di_store<V>(out + d, x);
+      }
+    }
+    return;
+  }
   // STAGED: all inputs of the warp's rows (and of the rows just before them) are on their way together; a lane reads
   // back only what it copied itself
   const int s_begin = max(0, t_begin - past), width = max(2 * a.dk, a.dv);
@@ -167,10 +197,9 @@ __global__ void __launch_bounds__(DI_WARPS * 32) delta_inputs_kernel(const Delta
   };
   // decay, step size and k . q of row t, value head h
   auto numbers = [&](int t, int h, float kq) {
-    const float* p = a.proj + (size_t)t * a.stride + C + a.H * a.dv + h;
-    const float b = p[0], x = p[a.H] + a.dt_bias[h];
-    const float softplus = fmaxf(x, 0.f) + log1pf(expf(-fabsf(x)));
-    a.scal[(size_t)t * a.H + h] = make_float4(expf(-expf(a.A_log[h]) * softplus), 1.f / (1.f + expf(-b)), kq, 0.f);
+    const float* p = a.proj + (size_t)t * a.stride + a.b_col + h;
+    const float g = a.z ? 1.f : dr_decay(expf(a.A_log[h]), p[a.H] + a.dt_bias[h]);
+    a.scal[(size_t)t * a.H + h] = make_float4(g, 1.f / (1.f + expf(-p[0])), kq, 0.f);
   };
   const int group = a.H / a.G;
   float kq_mine = 0.f;  // lane r: k . q of the warp's row r
@@ -263,6 +292,8 @@ __global__ void __launch_bounds__(DI_WARPS * 32) delta_inputs_kernel(const Delta
 // which leaves one reduction over the P lanes on a token's critical path.
 // q, k, v and the three numbers of DR_TT tokens are staged per pass, the next pass on its way
 // (cp.async) while this one is computed. The state is stored transposed, [slot][head][dv][dk].
+// CH: decays per channel, staged beside q and k; the rows of S are multiplied first and the
+// number per head is 1.
 constexpr int DR_ROWS = 16, DR_THREADS = 128, DR_TT = 16;
 
 struct DeltaRule {
@@ -275,14 +306,15 @@ struct DeltaRule {
   const int* slots;
   int H, G, dk, dv;
   int longest;         // longer portions than this are not served here (0: all are)
+  const float* decay;  // [T, H dk]: a decay per channel; null: scal's number per head
 };
 
-template <int P>
+template <int P, bool CH>
 __global__ void __launch_bounds__(DR_THREADS) delta_rule_kernel(const DeltaRule a) {
   constexpr int CB = DR_THREADS / P;        // columns of this block
   constexpr int LD = P * DR_ROWS;           // a staged q or k row
   constexpr int R4 = DR_ROWS / 4;
-  constexpr int PER = 2 * DR_TT * LD + DR_TT * CB + DR_TT * 4;  // floats per buffer
+  constexpr int PER = (CH ? 3 : 2) * DR_TT * LD + DR_TT * CB + DR_TT * 4;  // floats per buffer
   extern __shared__ __align__(16) float dr_smem[];
   float* os = dr_smem + 2 * PER;            // [DR_TT][CB] outputs of a pass
   pdl_trigger();
@@ -325,6 +357,13 @@ __global__ void __launch_bounds__(DR_THREADS) delta_rule_kernel(const DeltaRule 
     }
     for (int tt = threadIdx.x; tt < tn; tt += DR_THREADS)
       dr_copy(ss + tt * 4, reinterpret_cast<const float*>(a.scal + (size_t)(r0 + t0 + tt) * H + h), true);
+    if constexpr (CH) {
+      float* gs = ss + DR_TT * 4;
+      for (int idx = threadIdx.x; idx < tn * ku; idx += DR_THREADS) {
+        const int tt = idx / ku, i = (idx - tt * ku) * kstep;
+        dr_copy(gs + tt * LD + i, a.decay + ((size_t)(r0 + t0 + tt) * H + h) * dk + i, wide_k);
+      }
+    }
     asm volatile("cp.async.commit_group;\n" ::);
   };
   issue(0, 0);
@@ -359,13 +398,18 @@ __global__ void __launch_bounds__(DR_THREADS) delta_rule_kernel(const DeltaRule 
     const float4* ss = reinterpret_cast<const float4*>(vs + DR_TT * CB);
     const float4* k4 = reinterpret_cast<const float4*>(ks) + p;
     const float4* q4 = reinterpret_cast<const float4*>(qs) + p;
+    const float4* g4 = reinterpret_cast<const float4*>(vs + DR_TT * CB + DR_TT * 4) + p;
 #pragma unroll 2
-    for (int tt = 0; tt < tn; ++tt, k4 += LD / 4, q4 += LD / 4) {
+    for (int tt = 0; tt < tn; ++tt, k4 += LD / 4, q4 += LD / 4, g4 += CH ? LD / 4 : 0) {
       float kv[DR_ROWS];
       float kd0 = 0.f, kd1 = 0.f, qd0 = 0.f, qd1 = 0.f;
 #pragma unroll
       for (int r = 0; r < R4; ++r) {
         const float4 k = k4[r * P], q = q4[r * P];
+        if constexpr (CH) {
+          const float4 g = g4[r * P];
+          S[4 * r] *= g.x; S[4 * r + 1] *= g.y; S[4 * r + 2] *= g.z; S[4 * r + 3] *= g.w;
+        }
         kv[4 * r] = k.x; kv[4 * r + 1] = k.y; kv[4 * r + 2] = k.z; kv[4 * r + 3] = k.w;
         kd0 = fmaf(S[4 * r], k.x, kd0);
         kd1 = fmaf(S[4 * r + 1], k.y, kd1);
@@ -383,10 +427,17 @@ __global__ void __launch_bounds__(DR_THREADS) delta_rule_kernel(const DeltaRule 
         qd += __shfl_xor_sync(0xffffffffu, qd, o);
       }
       const float4 sc = ss[tt];
-      const float u = sc.y * (vs[tt * CB + jl] - sc.x * kd);
+      if constexpr (CH) {
+        const float u = sc.y * (vs[tt * CB + jl] - kd);
 #pragma unroll
-      for (int r = 0; r < DR_ROWS; ++r) S[r] = fmaf(kv[r], u, sc.x * S[r]);
-      if (p == 0) os[tt * CB + jl] = fmaf(sc.z, u, sc.x * qd);
+        for (int r = 0; r < DR_ROWS; ++r) S[r] = fmaf(kv[r], u, S[r]);
+        if (p == 0) os[tt * CB + jl] = fmaf(sc.z, u, qd);
+      } else {
+        const float u = sc.y * (vs[tt * CB + jl] - sc.x * kd);
+#pragma unroll
+        for (int r = 0; r < DR_ROWS; ++r) S[r] = fmaf(kv[r], u, sc.x * S[r]);
+        if (p == 0) os[tt * CB + jl] = fmaf(sc.z, u, sc.x * qd);
+      }
     }
     __syncthreads();  // the outputs are there, and the buffer is free for the pass after the next
     for (int idx = threadIdx.x; idx < tn * cols; idx += DR_THREADS) {
@@ -427,6 +478,10 @@ __global__ void __launch_bounds__(DR_THREADS) delta_rule_kernel(const DeltaRule 
 // All in float32 (register-tiled products on the CUDA cores); the decays enter as products of
 // factors in (0, 1], so nothing overflows. A chunk that is not full is filled up with tokens of
 // g = 1, beta = 0 and zero vectors.
+//
+// With a decay per channel (CH) the products k_s . k_t and k_s . q_t are taken with every channel
+// multiplied by its own r_ts, and G_t k_t, G_t q_t and r_(last,t) k_t channel by channel. Launch A has
+// a form of its own for it; C then reads G q as A left it.
 constexpr int DC_L = 64, DC_THREADS = 256, DC_B = 16, DC_B_THREADS = 256, DC_N = 64;
 constexpr int DC_MAX_DV = 512;  // value sizes whose rows fit launch A's shared memory; longer ones run token by token
 
@@ -438,6 +493,7 @@ struct DeltaChunks {
   const int* cu_q;
   const int* ctx_lens;
   const int* slots;
+  const float* decay;  // [T, H dk] (CH)
   int H, G, dk, dv;
   int ld;              // row length of q, k, W and state rows: dk up to a multiple of 16, + 4 (zeros behind dk)
   int dvp;             // dv up to a multiple of DC_B
@@ -447,7 +503,8 @@ struct DeltaChunks {
   float* u;            // [dvp / 16][64][16]: U, then u, in the slices of launch B
   float* p;            // [64][DC_LDP]
   float* s0;           // [dvp][ld]: the (transposed) state before the chunk
-  float* g;            // [64]: G_t
+  float* g;            // [64]: G_t; CH: [ld]: G_last of every channel
+  float* qg;           // CH: [64][ld]: G q
 };
 constexpr int DC_LDP = DC_L + 4;
 
@@ -490,6 +547,75 @@ template <int THREADS>
 __device__ __forceinline__ void dc_store_flat(float* dst, const float* src, int n) {
   for (int i = 4 * threadIdx.x; i < n; i += 4 * THREADS)
     *reinterpret_cast<float4*>(dst + i) = *reinterpret_cast<const float4*>(src + i);
+}
+
+// (I + M) X = factor X, unit lower triangular, X = the dk columns of W in ks (rows ld apart) and the dvp columns of U
+// in qs; M in ms (rows DC_LDP apart, its strictly lower part is read); factor(is W, row) scales the right-hand sides.
+template <typename F>
+__device__ __forceinline__ void dc_solve(float* ks, int ld, int dk, float* qs, int dvp, const float* ms, F factor) {
+  // Forward substitution in blocks of 16 rows, in place: two columns of W and U per thread (a row of M is
+  // read once for both). What the rows of earlier blocks contribute comes from shared memory, the
+  // block's own 16 values stay in registers.
+  const int columns = dk + dvp, half = (columns + 1) / 2;
+  for (int col = (int)threadIdx.x; col < half; col += DC_THREADS) {
+    float* x[2];
+    int xs[2];
+    bool is_w[2];
+#pragma unroll
+    for (int v = 0; v < 2; ++v) {
+      const int cc = col + v * half < columns ? col + v * half : col;  // (an odd number: one thread has its column twice)
+      is_w[v] = cc < dk;
+      x[v] = is_w[v] ? ks + cc : qs + (cc - dk);
+      xs[v] = is_w[v] ? ld : dvp;
+    }
+#pragma unroll 1
+    for (int b = 0; b < DC_L; b += 16) {
+      float acc[2][16];
+#pragma unroll
+      for (int i = 0; i < 16; ++i) {
+#pragma unroll
+        for (int v = 0; v < 2; ++v) acc[v][i] = factor(is_w[v], b + i) * x[v][(b + i) * xs[v]];
+      }
+#pragma unroll 1
+      for (int s = 0; s < b; s += 4) {
+        float xv[2][4];
+#pragma unroll
+        for (int v = 0; v < 2; ++v)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) xv[v][e] = x[v][(s + e) * xs[v]];
+#pragma unroll
+        for (int i = 0; i < 16; ++i) {
+          const float4 m = *reinterpret_cast<const float4*>(ms + (b + i) * DC_LDP + s);
+#pragma unroll
+          for (int v = 0; v < 2; ++v) {
+            acc[v][i] = fmaf(-m.x, xv[v][0], acc[v][i]);
+            acc[v][i] = fmaf(-m.y, xv[v][1], acc[v][i]);
+            acc[v][i] = fmaf(-m.z, xv[v][2], acc[v][i]);
+            acc[v][i] = fmaf(-m.w, xv[v][3], acc[v][i]);
+          }
+        }
+      }
+#pragma unroll
+      for (int s = 0; s < 16; s += 4) {
+        // the block's rows s .. s + 3 are finished one after another, the rows below take them off as they come
+#pragma unroll
+        for (int i = s + 1; i < 16; ++i) {
+          const float4 m = *reinterpret_cast<const float4*>(ms + (b + i) * DC_LDP + b + s);
+#pragma unroll
+          for (int v = 0; v < 2; ++v) {
+            acc[v][i] = fmaf(-m.x, acc[v][s], acc[v][i]);
+            if (i > s + 1) acc[v][i] = fmaf(-m.y, acc[v][s + 1], acc[v][i]);
+            if (i > s + 2) acc[v][i] = fmaf(-m.z, acc[v][s + 2], acc[v][i]);
+            if (i > s + 3) acc[v][i] = fmaf(-m.w, acc[v][s + 3], acc[v][i]);
+          }
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < 16; ++i)
+#pragma unroll
+        for (int v = 0; v < 2; ++v) x[v][(b + i) * xs[v]] = acc[v][i];
+    }
+  }
 }
 
 // ---- launch A
@@ -612,70 +738,235 @@ __global__ void __launch_bounds__(DC_THREADS, 2) delta_chunk_systems_kernel(cons
   }
   asm volatile("cp.async.wait_group 0;\n" ::);
   __syncthreads();
-  // Forward substitution in blocks of 16 rows, in place: two columns of W and U per thread (a row of M is
-  // read once for both). What the rows of earlier blocks contribute comes from shared memory, the
-  // block's own 16 values stay in registers.
-  const int columns = dk + dvp, half = (columns + 1) / 2;
-  for (int col = tid; col < half; col += DC_THREADS) {
-    float* x[2];
-    int xs[2];
-    bool is_w[2];
+  dc_solve(ks, ld, dk, qs, dvp, ms, [&](bool is_w, int i) { return is_w ? gs[DC_L + i] * gs[2 * DC_L + i] : gs[DC_L + i]; });
+  __syncthreads();
+  dc_store_flat<DC_THREADS>(a.wk + at * 2 * DC_L * ld, ks, DC_L * ld);
+  float* ug = a.u + at * DC_L * dvp;
+  const int t = tid >> 2, q = 4 * (tid & 3);
+  for (int c0 = 0; c0 < dvp; c0 += DC_B)
+    *reinterpret_cast<float4*>(ug + (size_t)c0 * DC_L + t * DC_B + q) =
+        *reinterpret_cast<const float4*>(qs + t * dvp + c0 + q);
+}
+
+// ---- launch A, decays per channel
+// The chunk is four blocks of 16 tokens. With F_t the product of a block's decays up to and with t, E_s that of
+// the decays behind s in its block and B_b a whole block's, a token t of block i and a token s of an
+// earlier block j have r_ts = F_t (B_(j+1) .. B_(i-1)) E_s: two products of factors in (0, 1], so a dot
+// product of scaled vectors, (F k)_t . B (E k)_s, gives M and P between blocks. Within a block there is no
+// such split that cannot underflow: there r_ts k_s is multiplied up token by token, a column s at a time.
+// NR: pieces of four channels that a thread has of a column there (8 threads share a column).
+constexpr int DC_BLOCK = 16, DC_BLOCKS = DC_L / DC_BLOCK;
+
+static size_t channel_systems_floats(int ld, int dvp) {
+  const int third = ld > DC_LDP ? ld : DC_LDP;
+  return (size_t)DC_L * (ld + (ld > dvp ? ld : dvp) + third) + DC_BLOCKS * ld + DC_L + DC_BLOCKS * DC_BLOCK * DC_BLOCK;
+}
+
+template <int NR>
+__global__ void __launch_bounds__(DC_THREADS, 2) delta_channel_systems_kernel(const DeltaChunks a) {
+  extern __shared__ __align__(16) float dc_smem[];
+  pdl_trigger();
+  const int c = blockIdx.x, h = blockIdx.y, seq = blockIdx.z;
+  const int r0 = a.cu_q[seq], n = a.cu_q[seq + 1] - r0;
+  const int chunks = n > DC_L ? (n + DC_L - 1) / DC_L : 0;
+  if (c >= chunks) {
+    pdl_wait();
+    return;
+  }
+  const size_t at = (size_t)(dc_first_chunk(a.cu_q, seq) + c) * a.H + h;
+  const int dk = a.dk, dv = a.dv, ld = a.ld, dvp = a.dvp, tid = threadIdx.x;
+  const int kh = h / (a.H / a.G), C = 2 * a.G * dk + a.H * dv;
+  const int t0 = r0 + c * DC_L, tn = min(DC_L, n - c * DC_L);
+  float* ks = dc_smem;                        // [64][ld]: k, then F k, then W
+  float* qs = ks + DC_L * ld;                 // [64][ld]: q, then F q; then v and U, [64][dvp]
+  float* gs = qs + DC_L * max(ld, dvp);       // [64][ld]: g, then E k; then M, [64][DC_LDP]
+  float* bs = gs + DC_L * max(ld, DC_LDP);    // [4][ld]: B
+  float* betas = bs + DC_BLOCKS * ld;         // [64]
+  float* diag = betas + DC_L;                 // [4][16][16]: M within the blocks
+  pdl_wait();
+  const float* row0 = a.qkv + (size_t)t0 * C;
+  const bool wide = dk % 4 == 0 && C % 4 == 0;
+  dc_stage(qs, ld, row0 + (size_t)kh * dk, C, tn, dk, wide);
+  dc_stage(ks, ld, row0 + (size_t)(a.G + kh) * dk, C, tn, dk, wide);
+  dc_stage(gs, ld, a.decay + ((size_t)t0 * a.H + h) * dk, (long long)a.H * dk, tn, dk, wide);
+  asm volatile("cp.async.commit_group;\n" ::);
+  if (tid < DC_L) betas[tid] = tid < tn ? a.scal[(size_t)(t0 + tid) * a.H + h].y : 0.f;
+  __syncwarp();
+  if (const int t = tid >> 2; t >= tn)  // tokens that fill the chunk up do not decay (this warp has zeroed the row)
+    for (int i = tid & 3; i < ld; i += 4) gs[t * ld + i] = 1.f;
+  asm volatile("cp.async.wait_group 0;\n" ::);
+  __syncthreads();
+  float* pg = a.p + at * DC_L * DC_LDP;
+  {
+    // within the blocks: a thread has the pieces slice, slice + 8, ... of the columns s and s + 8 of its block
+    const int slice = tid & 7, b = tid >> 6, s = (tid >> 3) & 7;
+    const float* kb = ks + b * DC_BLOCK * ld;
+    const float* qb = qs + b * DC_BLOCK * ld;
+    const float* gb = gs + b * DC_BLOCK * ld;
+    float run[2][NR][4];
 #pragma unroll
-    for (int v = 0; v < 2; ++v) {
-      const int cc = col + v * half < columns ? col + v * half : col;  // (an odd number: one thread has its column twice)
-      is_w[v] = cc < dk;
-      x[v] = is_w[v] ? ks + cc : qs + (cc - dk);
-      xs[v] = is_w[v] ? ld : dvp;
-    }
-#pragma unroll 1
-    for (int b = 0; b < DC_L; b += 16) {
-      float acc[2][16];
+    for (int v = 0; v < 2; ++v)
 #pragma unroll
-      for (int i = 0; i < 16; ++i) {
-        const float beta = gs[DC_L + b + i], g = gs[2 * DC_L + b + i];
-#pragma unroll
-        for (int v = 0; v < 2; ++v) acc[v][i] = (is_w[v] ? beta * g : beta) * x[v][(b + i) * xs[v]];
+      for (int r = 0; r < NR; ++r) {
+        const int d = 4 * (slice + 8 * r);
+        float4 k = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (d < ld - 4) k = *reinterpret_cast<const float4*>(kb + (s + 8 * v) * ld + d);
+        run[v][r][0] = k.x; run[v][r][1] = k.y; run[v][r][2] = k.z; run[v][r][3] = k.w;
       }
 #pragma unroll 1
-      for (int s = 0; s < b; s += 4) {
-        float xv[2][4];
+    for (int t = 0; t < DC_BLOCK; ++t) {
+      float acc[2][2] = {{0.f, 0.f}, {0.f, 0.f}};  // [column][with k_t, with q_t]
 #pragma unroll
-        for (int v = 0; v < 2; ++v)
+      for (int r = 0; r < NR; ++r) {
+        const int d = 4 * (slice + 8 * r);
+        if (d >= ld - 4) continue;
+        const float4 g = *reinterpret_cast<const float4*>(gb + t * ld + d);
+        const float4 k = *reinterpret_cast<const float4*>(kb + t * ld + d);
+        const float4 q = *reinterpret_cast<const float4*>(qb + t * ld + d);
 #pragma unroll
-          for (int e = 0; e < 4; ++e) xv[v][e] = x[v][(s + e) * xs[v]];
-#pragma unroll
-        for (int i = 0; i < 16; ++i) {
-          const float4 m = *reinterpret_cast<const float4*>(ms + (b + i) * DC_LDP + s);
-#pragma unroll
-          for (int v = 0; v < 2; ++v) {
-            acc[v][i] = fmaf(-m.x, xv[v][0], acc[v][i]);
-            acc[v][i] = fmaf(-m.y, xv[v][1], acc[v][i]);
-            acc[v][i] = fmaf(-m.z, xv[v][2], acc[v][i]);
-            acc[v][i] = fmaf(-m.w, xv[v][3], acc[v][i]);
+        for (int v = 0; v < 2; ++v) {
+          if (v == 1 && t < 8) continue;  // its columns have not begun
+          if (t > s + 8 * v) {
+            run[v][r][0] *= g.x; run[v][r][1] *= g.y; run[v][r][2] *= g.z; run[v][r][3] *= g.w;
           }
+          acc[v][0] = fmaf(run[v][r][0], k.x, acc[v][0]);
+          acc[v][1] = fmaf(run[v][r][0], q.x, acc[v][1]);
+          acc[v][0] = fmaf(run[v][r][1], k.y, acc[v][0]);
+          acc[v][1] = fmaf(run[v][r][1], q.y, acc[v][1]);
+          acc[v][0] = fmaf(run[v][r][2], k.z, acc[v][0]);
+          acc[v][1] = fmaf(run[v][r][2], q.z, acc[v][1]);
+          acc[v][0] = fmaf(run[v][r][3], k.w, acc[v][0]);
+          acc[v][1] = fmaf(run[v][r][3], q.w, acc[v][1]);
         }
       }
-#pragma unroll
-      for (int s = 0; s < 16; s += 4) {
-        // the block's rows s .. s + 3 are finished one after another, the rows below take them off as they come
-#pragma unroll
-        for (int i = s + 1; i < 16; ++i) {
-          const float4 m = *reinterpret_cast<const float4*>(ms + (b + i) * DC_LDP + b + s);
-#pragma unroll
-          for (int v = 0; v < 2; ++v) {
-            acc[v][i] = fmaf(-m.x, acc[v][s], acc[v][i]);
-            if (i > s + 1) acc[v][i] = fmaf(-m.y, acc[v][s + 1], acc[v][i]);
-            if (i > s + 2) acc[v][i] = fmaf(-m.z, acc[v][s + 2], acc[v][i]);
-            if (i > s + 3) acc[v][i] = fmaf(-m.w, acc[v][s + 3], acc[v][i]);
-          }
-        }
+      // four sums over eight lanes: every step halves what a lane still carries
+      const bool hi4 = slice & 4, hi2 = slice & 2;
+      float x0 = hi4 ? acc[1][0] : acc[0][0], x1 = hi4 ? acc[1][1] : acc[0][1];
+      x0 += __shfl_xor_sync(0xffffffffu, hi4 ? acc[0][0] : acc[1][0], 4);
+      x1 += __shfl_xor_sync(0xffffffffu, hi4 ? acc[0][1] : acc[1][1], 4);
+      float y = hi2 ? x1 : x0;
+      y += __shfl_xor_sync(0xffffffffu, hi2 ? x0 : x1, 2);
+      y += __shfl_xor_sync(0xffffffffu, y, 1);
+      if (!(slice & 1)) {
+        const int col = s + (hi4 ? 8 : 0), row = b * DC_BLOCK + t;
+        if (hi2) pg[row * DC_LDP + b * DC_BLOCK + col] = col <= t ? y : 0.f;
+        else diag[(b * DC_BLOCK + t) * DC_BLOCK + col] = betas[row] * y;  // (read for col < t only)
       }
-#pragma unroll
-      for (int i = 0; i < 16; ++i)
-#pragma unroll
-        for (int v = 0; v < 2; ++v) x[v][(b + i) * xs[v]] = acc[v][i];
     }
   }
+  __syncthreads();
+  for (int idx = tid; idx < DC_BLOCKS * (ld - 4); idx += DC_THREADS) {  // a channel of a block
+    const int b = idx / (ld - 4), d = idx - b * (ld - 4);
+    float* kp = ks + b * DC_BLOCK * ld + d;
+    float* qp = qs + b * DC_BLOCK * ld + d;
+    float* gp = gs + b * DC_BLOCK * ld + d;
+    float k[DC_BLOCK], g[DC_BLOCK];
+#pragma unroll
+    for (int t = 0; t < DC_BLOCK; ++t) {
+      k[t] = kp[t * ld];
+      g[t] = gp[t * ld];
+    }
+    float f = 1.f, e = 1.f;
+#pragma unroll
+    for (int t = 0; t < DC_BLOCK; ++t) {
+      f *= g[t];
+      kp[t * ld] = k[t] * f;
+      qp[t * ld] *= f;
+    }
+    bs[b * ld + d] = f;
+#pragma unroll
+    for (int t = DC_BLOCK - 1; t >= 0; --t) {
+      gp[t * ld] = k[t] * e;
+      e *= g[t];
+    }
+  }
+  for (int i = tid; i < DC_L * 4; i += DC_THREADS) gs[(i >> 2) * ld + ld - 4 + (i & 3)] = 0.f;  // (the row's filling)
+  if (tid < DC_BLOCKS * 4) bs[(tid >> 2) * ld + ld - 4 + (tid & 3)] = 0.f;
+  __syncthreads();
+  const int ty = tid >> 4, tx = tid & 15;
+  float kk[6], qk[6];  // blocks (1,0) (2,0) (2,1) (3,0) (3,1) (3,2): rows ty + 16 i, columns tx + 16 j
+#pragma unroll
+  for (int i = 0; i < 6; ++i) kk[i] = qk[i] = 0.f;
+  for (int d = 0; d < ld - 4; d += 4) {
+    auto row = [&](const float* m, int r) { return *reinterpret_cast<const float4*>(m + r * ld + d); };
+    auto mul = [](const float4& x, const float4& y) { return make_float4(x.x * y.x, x.y * y.y, x.z * y.z, x.w * y.w); };
+    auto dot = [](const float4& x, const float4& y, float& acc) {
+      acc = fmaf(x.x, y.x, acc);
+      acc = fmaf(x.y, y.y, acc);
+      acc = fmaf(x.z, y.z, acc);
+      acc = fmaf(x.w, y.w, acc);
+    };
+    const float4 b1 = row(bs, 1), b2 = row(bs, 2);
+    const float4 c10 = row(gs, tx), c21 = row(gs, tx + 16), c32 = row(gs, tx + 32);
+    const float4 c20 = mul(c10, b1), c31 = mul(c21, b2), c30 = mul(c20, b2);
+    const float4 k1 = row(ks, ty + 16), k2 = row(ks, ty + 32), k3 = row(ks, ty + 48);
+    const float4 q1 = row(qs, ty + 16), q2 = row(qs, ty + 32), q3 = row(qs, ty + 48);
+    dot(k1, c10, kk[0]); dot(q1, c10, qk[0]);
+    dot(k2, c20, kk[1]); dot(q2, c20, qk[1]);
+    dot(k2, c21, kk[2]); dot(q2, c21, qk[2]);
+    dot(k3, c30, kk[3]); dot(q3, c30, qk[3]);
+    dot(k3, c31, kk[4]); dot(q3, c31, qk[4]);
+    dot(k3, c32, kk[5]); dot(q3, c32, qk[5]);
+  }
+#pragma unroll
+  for (int i = 1, e = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < i; ++j, ++e) pg[(ty + 16 * i) * DC_LDP + tx + 16 * j] = qk[e];
+  __syncthreads();
+  {
+    // G q and r_(last,t) k out, and the right-hand side of W: beta G k
+    const int t = tid >> 2, b = t / DC_BLOCK;
+    const float beta = betas[t];
+    float* kg = a.wk + at * 2 * DC_L * ld + (size_t)(DC_L + t) * ld;
+    float* qg = a.qg + (at * DC_L + t) * ld;
+    for (int i = 4 * (tid & 3); i < ld; i += 16) {
+      float4 before = make_float4(1.f, 1.f, 1.f, 1.f), behind = before;
+#pragma unroll
+      for (int o = 0; o < DC_BLOCKS; ++o) {
+        const float4 w = *reinterpret_cast<const float4*>(bs + o * ld + i);
+        if (o < b) { before.x *= w.x; before.y *= w.y; before.z *= w.z; before.w *= w.w; }
+        if (o > b) { behind.x *= w.x; behind.y *= w.y; behind.z *= w.z; behind.w *= w.w; }
+      }
+      const float4 e = *reinterpret_cast<const float4*>(gs + t * ld + i);
+      const float4 q = *reinterpret_cast<const float4*>(qs + t * ld + i);
+      float4* kp = reinterpret_cast<float4*>(ks + t * ld + i);
+      const float4 k = *kp;
+      *reinterpret_cast<float4*>(kg + i) = make_float4(e.x * behind.x, e.y * behind.y, e.z * behind.z, e.w * behind.w);
+      *reinterpret_cast<float4*>(qg + i) = make_float4(q.x * before.x, q.y * before.y, q.z * before.z, q.w * before.w);
+      *kp = make_float4(beta * before.x * k.x, beta * before.y * k.y, beta * before.z * k.z, beta * before.w * k.w);
+      if (t == 0) {
+        const float4 w = *reinterpret_cast<const float4*>(bs + i);
+        *reinterpret_cast<float4*>(a.g + at * ld + i) =
+            make_float4(w.x * behind.x, w.y * behind.y, w.z * behind.z, w.w * behind.w);
+      }
+    }
+  }
+  __syncthreads();
+  float* ms = gs;
+  {
+    const int t = tid >> 2;
+    float* d = qs + t * dvp;
+    const float* s = row0 + (size_t)t * C + (size_t)2 * a.G * dk + (size_t)h * dv;
+    const bool wv = wide && dv % 4 == 0;
+    const int step = wv ? 4 : 1;
+    for (int i = (tid & 3) * step; i < dvp; i += 4 * step) {
+      if (t < tn && i < dv) {
+        dr_copy(d + i, s + i, wv);
+      } else {
+        for (int e = 0; e < step; ++e) d[i + e] = 0.f;
+      }
+    }
+  }
+  asm volatile("cp.async.commit_group;\n" ::);
+#pragma unroll
+  for (int i = 1, e = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < i; ++j, ++e) ms[(ty + 16 * i) * DC_LDP + tx + 16 * j] = betas[ty + 16 * i] * kk[e];
+#pragma unroll
+  for (int i = 0; i < 4; ++i) ms[(ty + 16 * i) * DC_LDP + tx + 16 * i] = diag[(16 * i + ty) * DC_BLOCK + tx];
+  asm volatile("cp.async.wait_group 0;\n" ::);
+  __syncthreads();
+  dc_solve(ks, ld, dk, qs, dvp, ms, [&](bool is_w, int i) { return is_w ? 1.f : betas[i]; });
   __syncthreads();
   dc_store_flat<DC_THREADS>(a.wk + at * 2 * DC_L * ld, ks, DC_L * ld);
   float* ug = a.u + at * DC_L * dvp;
@@ -686,6 +977,7 @@ __global__ void __launch_bounds__(DC_THREADS, 2) delta_chunk_systems_kernel(cons
 }
 
 // ---- launch B
+template <bool CH>
 __global__ void __launch_bounds__(DC_B_THREADS) delta_chunk_states_kernel(const DeltaChunks a) {
   extern __shared__ __align__(16) float dc_smem[];
   pdl_trigger();
@@ -736,7 +1028,7 @@ __global__ void __launch_bounds__(DC_B_THREADS) delta_chunk_states_kernel(const 
     const float* ks = ws + DC_L * ld;
     float* us = ws + 2 * DC_L * ld;
     const size_t at = first + (size_t)c * a.H;
-    const float whole = __ldg(a.g + at * DC_L + DC_L - 1);
+    const float whole = CH ? 1.f : __ldg(a.g + at * DC_L + DC_L - 1);
     dc_store_flat<DC_B_THREADS>(a.s0 + (at * a.dvp + c0) * ld, Ss, DC_B * ld);
     float acc[8][4];
 #pragma unroll
@@ -806,7 +1098,12 @@ __global__ void __launch_bounds__(DC_B_THREADS) delta_chunk_states_kernel(const 
       if (d >= ld - 4) continue;
       float4* p = reinterpret_cast<float4*>(Ss + j * ld + d);
       float4 o = *p;
-      o.x *= whole; o.y *= whole; o.z *= whole; o.w *= whole;
+      if constexpr (CH) {
+        const float4 w = __ldg(reinterpret_cast<const float4*>(a.g + at * ld + d));
+        o.x *= w.x; o.y *= w.y; o.z *= w.z; o.w *= w.w;
+      } else {
+        o.x *= whole; o.y *= whole; o.z *= whole; o.w *= whole;
+      }
       for (int g = 0; g < parts; ++g) {
         const float4 v = *reinterpret_cast<const float4*>(part + ((g * dims + b) * DC_B + j) * 32 + (tid & 7) * 4);
         o.x += v.x; o.y += v.y; o.z += v.z; o.w += v.w;
@@ -821,6 +1118,7 @@ __global__ void __launch_bounds__(DC_B_THREADS) delta_chunk_states_kernel(const 
 }
 
 // ---- launch C
+template <bool CH>
 __global__ void __launch_bounds__(DC_THREADS, 3) delta_chunk_outputs_kernel(const DeltaChunks a) {
   extern __shared__ __align__(16) float dc_smem[];
   pdl_trigger();
@@ -839,7 +1137,8 @@ __global__ void __launch_bounds__(DC_THREADS, 3) delta_chunk_outputs_kernel(cons
   float* qs = dc_smem;            // [64][ld]; then P [64][DC_LDP]
   float* ss = qs + DC_L * ld;     // [64][ld]: columns of the state; then u, up to four slices of [64][16]
   pdl_wait();
-  dc_stage(qs, ld, a.qkv + (size_t)t0 * C + (size_t)kh * dk, C, tn, dk, dk % 4 == 0 && C % 4 == 0);
+  if constexpr (CH) dc_stage_flat<DC_THREADS>(qs, a.qg + at * DC_L * ld, DC_L * ld);
+  else dc_stage(qs, ld, a.qkv + (size_t)t0 * C + (size_t)kh * dk, C, tn, dk, dk % 4 == 0 && C % 4 == 0);
   dc_stage_flat<DC_THREADS>(ss, a.s0 + (at * a.dvp + c0) * ld, cols * ld);
   asm volatile("cp.async.commit_group;\n" ::);
   asm volatile("cp.async.wait_group 0;\n" ::);
@@ -874,11 +1173,13 @@ __global__ void __launch_bounds__(DC_THREADS, 3) delta_chunk_outputs_kernel(cons
   dc_stage_flat<DC_THREADS>(ps, a.p + at * DC_L * DC_LDP, DC_L * DC_LDP);
   dc_stage_flat<DC_THREADS>(us, a.u + at * DC_L * a.dvp + (size_t)c0 * DC_L, cols * DC_L);
   asm volatile("cp.async.commit_group;\n" ::);
+  if constexpr (!CH) {
 #pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    const float g = __ldg(a.g + at * DC_L + ty + 16 * i);
+    for (int i = 0; i < 4; ++i) {
+      const float g = __ldg(a.g + at * DC_L + ty + 16 * i);
 #pragma unroll
-    for (int j = 0; j < 4; ++j) acc[i][j] *= g;
+      for (int j = 0; j < 4; ++j) acc[i][j] *= g;
+    }
   }
   asm volatile("cp.async.wait_group 0;\n" ::);
   __syncthreads();
@@ -923,24 +1224,27 @@ extern "C" int lse_delta_inputs(const float* proj, long long stride, const float
                                 float* conv_state, const float* A_log, const float* dt_bias, const int* token_seq,
                                 const int* cu_q, const int* ctx_lens, const int* slots, float* qkv, float* scal,
                                 int T, int H, int G, int dk, int dv, float q_scale,
-                                cudaStream_t stream) {
+                                cudaStream_t stream, const float* z, long long z_stride, float* decay) {
   if (T <= 0) return LSE_OK;
   if (H <= 0 || G <= 0 || H % G || dk <= 0 || dk > DI_MAX || dv <= 0 || taps < 1 || (taps > 1 && !conv_state) ||
-      stride < 2LL * G * dk + 2LL * H * dv + 2LL * H)
+      stride < 2LL * G * dk + (z ? 1LL : 2LL) * H * (dv + 1) || (z && (!decay || z_stride < (long long)H * dk)))
     return LSE_BAD_ARGUMENT;
   DeltaInputs a;
   a.proj = proj; a.stride = stride; a.conv = conv; a.conv_state = taps > 1 ? conv_state : nullptr;
   a.A_log = A_log; a.dt_bias = dt_bias; a.token_seq = token_seq; a.cu_q = cu_q; a.ctx_lens = ctx_lens;
   a.slots = slots; a.qkv = qkv; a.scal = reinterpret_cast<float4*>(scal);
   a.T = T; a.H = H; a.G = G; a.dk = dk; a.dv = dv; a.taps = taps; a.q_scale = q_scale;
-  const int jobs = (G + H + DI_WARPS - 1) / DI_WARPS;
+  a.b_col = 2 * G * dk + (z ? 1 : 2) * H * dv;
+  a.z = z; a.z_stride = z_stride; a.decay = z ? decay : nullptr;
+  const int jobs = (G + (z ? 2 : 1) * H + DI_WARPS - 1) / DI_WARPS;
   a.rows = (long long)T * jobs >= 16384 ? 8 : (long long)T * jobs >= 4096 ? 2 : 1;
   const dim3 grid((T + a.rows - 1) / a.rows, jobs);
   if (grid.y > 65535) return LSE_BAD_ARGUMENT;
   auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
   // 16-byte accesses: every head starts on one in the projection, the taps, the kept inputs and the result
   const bool vec = dk % 4 == 0 && dv % 4 == 0 && stride % 4 == 0 && aligned(proj) && aligned(conv) &&
-                   aligned(conv_state) && aligned(qkv);
+                   aligned(conv_state) && aligned(qkv) &&
+                   (!z || (z_stride % 4 == 0 && aligned(z) && aligned(dt_bias) && aligned(decay)));
   const size_t smem = (size_t)DI_WARPS * (a.rows + taps - 1) * (2 * dk > dv ? 2 * dk : dv) * sizeof(float);
   const bool staged = vec && a.rows > 1 && smem <= 96 * 1024;
 #define LSE_DI_LAUNCH(KERNEL, BYTES)                                                                              \
@@ -967,29 +1271,40 @@ extern "C" int lse_delta_inputs(const float* proj, long long stride, const float
   return LSE_CHECK_LAUNCH();
 }
 
-template <int P>
-static int launch_delta_rule(const DeltaRule& a, int num_seqs, cudaStream_t stream) {
+template <int P, bool CH>
+static int launch_delta_rule_form(const DeltaRule& a, int num_seqs, cudaStream_t stream) {
   constexpr int CB = DR_THREADS / P;
   constexpr size_t smem =
-      (2 * (2 * DR_TT * P * DR_ROWS + DR_TT * CB + DR_TT * 4) + DR_TT * CB) * sizeof(float);
+      (2 * ((CH ? 3 : 2) * DR_TT * P * DR_ROWS + DR_TT * CB + DR_TT * 4) + DR_TT * CB) * sizeof(float);
   static bool configured = false;
   if (smem > 48 * 1024 && !configured) {
-    if (cudaFuncSetAttribute(delta_rule_kernel<P>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+    if (cudaFuncSetAttribute(delta_rule_kernel<P, CH>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
       return LSE_LAUNCH_FAILED;
     configured = true;
   }
-  launch(delta_rule_kernel<P>, dim3(a.H * ((a.dv + CB - 1) / CB), num_seqs), DR_THREADS, smem, stream, a);
+  launch(delta_rule_kernel<P, CH>, dim3(a.H * ((a.dv + CB - 1) / CB), num_seqs), DR_THREADS, smem, stream, a);
   return LSE_CHECK_LAUNCH();
+}
+template <int P>
+static int launch_delta_rule(const DeltaRule& a, int num_seqs, cudaStream_t stream) {
+  return a.decay ? launch_delta_rule_form<P, true>(a, num_seqs, stream) : launch_delta_rule_form<P, false>(a, num_seqs, stream);
 }
 
 // Floats of scratch that one chunk of a portion longer than DC_L tokens needs.
-static size_t chunk_floats(int H, int dk, int dv) {
+static size_t chunk_floats(int H, int dk, int dv, bool channels) {
   const size_t ld = (dk + 15) / 16 * 16 + 4, dvp = (dv + DC_B - 1) / DC_B * DC_B;
-  return (size_t)H * (DC_L * (2 * ld + dvp + DC_LDP + 1) + dvp * ld);
+  return (size_t)H * (DC_L * (2 * ld + dvp + DC_LDP) + dvp * ld + (channels ? (DC_L + 1) * ld : DC_L));
+}
+// Does launch A's working space for decays per channel fit a block? (If not, such portions run token by token.)
+static bool channel_chunks_fit(int dk, int dv) {
+  const int ld = (dk + 15) / 16 * 16 + 4, dvp = (dv + DC_B - 1) / DC_B * DC_B;
+  return channel_systems_floats(ld, dvp) * sizeof(float) <= 227 * 1024;
 }
 
 extern "C" int lse_delta_rule_chunk(void) { return DC_L; }
-extern "C" size_t lse_delta_rule_chunk_floats(int H, int dk, int dv) { return chunk_floats(H, dk, dv); }
+extern "C" size_t lse_delta_rule_chunk_floats(int H, int dk, int dv, int channels) {
+  return chunk_floats(H, dk, dv, channels != 0);
+}
 
 template <auto KERNEL>
 static bool allow_smem(size_t bytes) {
@@ -1002,21 +1317,23 @@ static bool allow_smem(size_t bytes) {
 
 // The portions of more than DC_L tokens: max_chunks bounds the chunks of any sequence, total_chunks
 // those of all such sequences together (what the scratch has room for).
+template <bool CH>
 static int launch_delta_chunks(const DeltaRule& r, int num_seqs, int max_chunks, float* scratch, int total_chunks,
                                cudaStream_t stream) {
   DeltaChunks a;
   a.qkv = r.qkv; a.scal = r.scal; a.state = r.state; a.out = r.out; a.cu_q = r.cu_q; a.ctx_lens = r.ctx_lens;
-  a.slots = r.slots; a.H = r.H; a.G = r.G; a.dk = r.dk; a.dv = r.dv;
+  a.slots = r.slots; a.H = r.H; a.G = r.G; a.dk = r.dk; a.dv = r.dv; a.decay = r.decay;
   a.ld = (r.dk + 15) / 16 * 16 + 4;
   a.dvp = (r.dv + DC_B - 1) / DC_B * DC_B;
   const size_t units = (size_t)total_chunks * r.H;
   a.g = scratch;
-  a.p = a.g + units * DC_L;
+  a.p = a.g + units * (CH ? a.ld : DC_L);
   a.u = a.p + units * DC_L * DC_LDP;
   a.wk = a.u + units * DC_L * a.dvp;
   a.s0 = a.wk + units * 2 * DC_L * a.ld;
+  a.qg = CH ? a.s0 + units * a.dvp * a.ld : nullptr;
   if (r.H > 65535 || max_chunks > 65535) return LSE_BAD_ARGUMENT;
-  const size_t smem_a =
+  const size_t smem_a = CH ? channel_systems_floats(a.ld, a.dvp) * sizeof(float) :
       (size_t)(DC_L * a.ld + DC_L * (a.ld > a.dvp ? a.ld : a.dvp) + DC_L * DC_LDP + 4 * DC_L) * sizeof(float);
   const size_t per = (size_t)DC_L * (2 * a.ld + DC_B), rest = (size_t)DC_B * a.ld + 8 * DC_L * 20;
   a.stages = (2 * per + rest) * sizeof(float) <= 227 * 1024 ? 2 : 1;
@@ -1024,30 +1341,47 @@ static int launch_delta_chunks(const DeltaRule& r, int num_seqs, int max_chunks,
   size_t smem_c = (size_t)2 * DC_L * a.ld * sizeof(float);
   const size_t second = (size_t)DC_L * (DC_LDP + DC_N) * sizeof(float);  // what the second product stages in the same place
   if (smem_c < second) smem_c = second;
-  if (!allow_smem<delta_chunk_systems_kernel>(smem_a) || !allow_smem<delta_chunk_states_kernel>(smem_b) ||
-      !allow_smem<delta_chunk_outputs_kernel>(smem_c))
+  if (!allow_smem<delta_chunk_states_kernel<CH>>(smem_b) || !allow_smem<delta_chunk_outputs_kernel<CH>>(smem_c))
     return LSE_LAUNCH_FAILED;
-  launch(delta_chunk_systems_kernel, dim3(max_chunks, r.H, num_seqs), DC_THREADS, smem_a, stream, a);
-  launch(delta_chunk_states_kernel, dim3(r.H * (a.dvp / DC_B), num_seqs), DC_B_THREADS, smem_b, stream, a);
+  const dim3 grid_a(max_chunks, r.H, num_seqs);
+  if constexpr (CH) {
+    const int pieces = (a.ld - 4 + 31) / 32;  // of four channels, per thread
+#define LSE_CHANNELS(NR)                                                                             \
+  do {                                                                                               \
+    if (!allow_smem<delta_channel_systems_kernel<NR>>(smem_a)) return LSE_LAUNCH_FAILED;             \
+    launch(delta_channel_systems_kernel<NR>, grid_a, DC_THREADS, smem_a, stream, a);                 \
+  } while (0)
+    if (pieces <= 1) LSE_CHANNELS(1);
+    else if (pieces <= 2) LSE_CHANNELS(2);
+    else if (pieces <= 4) LSE_CHANNELS(4);
+    else LSE_CHANNELS(8);
+#undef LSE_CHANNELS
+  } else {
+    if (!allow_smem<delta_chunk_systems_kernel>(smem_a)) return LSE_LAUNCH_FAILED;
+    launch(delta_chunk_systems_kernel, grid_a, DC_THREADS, smem_a, stream, a);
+  }
+  launch(delta_chunk_states_kernel<CH>, dim3(r.H * (a.dvp / DC_B), num_seqs), DC_B_THREADS, smem_b, stream, a);
   const int slices = r.H * ((r.dv + DC_N - 1) / DC_N);
   if (slices > 65535) return LSE_BAD_ARGUMENT;
-  launch(delta_chunk_outputs_kernel, dim3(max_chunks, slices, num_seqs), DC_THREADS, smem_c, stream, a);
+  launch(delta_chunk_outputs_kernel<CH>, dim3(max_chunks, slices, num_seqs), DC_THREADS, smem_c, stream, a);
   return LSE_CHECK_LAUNCH();
 }
 
 extern "C" int lse_delta_rule(const float* qkv, const float* scal, float* state, float* out, const int* cu_q,
                               const int* ctx_lens, const int* slots, int num_seqs, int H, int G, int dk, int dv,
-                              cudaStream_t stream, int max_chunks, float* scratch, int total_chunks, int short_too) {
+                              cudaStream_t stream, int max_chunks, float* scratch, int total_chunks, int short_too,
+                              const float* decay) {
   if (num_seqs <= 0) return LSE_OK;
   if (max_chunks > 1 && (!scratch || total_chunks < 2)) return LSE_BAD_ARGUMENT;
   if (H <= 0 || G <= 0 || H % G || dk <= 0 || dk > DI_MAX || dv <= 0 || num_seqs > 65535) return LSE_BAD_ARGUMENT;
   DeltaRule a;
   a.qkv = qkv; a.scal = reinterpret_cast<const float4*>(scal); a.state = state; a.out = out; a.cu_q = cu_q;
-  a.ctx_lens = ctx_lens; a.slots = slots; a.H = H; a.G = G; a.dk = dk; a.dv = dv;
-  const bool chunked = max_chunks > 1 && dv <= DC_MAX_DV;
+  a.ctx_lens = ctx_lens; a.slots = slots; a.H = H; a.G = G; a.dk = dk; a.dv = dv; a.decay = decay;
+  const bool chunked = max_chunks > 1 && dv <= DC_MAX_DV && (!decay || channel_chunks_fit(dk, dv));
   a.longest = chunked ? DC_L : 0;
   if (chunked) {
-    const int code = launch_delta_chunks(a, num_seqs, max_chunks, scratch, total_chunks, stream);
+    const int code = decay ? launch_delta_chunks<true>(a, num_seqs, max_chunks, scratch, total_chunks, stream)
+                           : launch_delta_chunks<false>(a, num_seqs, max_chunks, scratch, total_chunks, stream);
     if (code != LSE_OK || !short_too) return code;
   }
   const int lanes = (dk + DR_ROWS - 1) / DR_ROWS;

@@ -18,9 +18,16 @@
 
 extern "C" {
 
-// out[t, :] = float(table[ids[t], :])                      out float32 [T, H]
+// out[t, :] = float(table[ids[t], :]) * scale              out float32 [T, H]
 int lse_embedding(const int* ids, const void* table, int table_dtype, float* out, int T, int H,
-                  cudaStream_t stream);
+                  cudaStream_t stream, float scale = 1.f);
+
+// x[t] += sum_i c[i] * y[i][t] (+ row), in place; with a weight also out[t] = x[t] / rms(x[t]) * weight.
+// n <= 4 tensors y[i] [T, H] of dtypes[i]: LSE_F32, or LSE_FIXED64 sums (cleared as they are read);
+// row float32 [H] or null; weight null: no norm, out is not written.
+int lse_sum_add_rmsnorm(float* x, const void* const* y, const float* c, const int* dtypes, int n,
+                        const float* row, const float* weight, float eps, void* out, int out_dtype, int T,
+                        int H, cudaStream_t stream);
 
 // Residual add and RMS norm.
 //   rows == nullptr: for every row t < T: if residual: x[t] += residual[t] (in place, float32);
@@ -126,6 +133,8 @@ int lse_ban_tokens(float* logits, int V, const int* row, const int* token, int n
 
 // out = x in out_dtype
 int lse_cast(const float* x, void* out, int out_dtype, long long n, cudaStream_t stream);
+// out[t, i] = x[t * stride + i] for i < cols: columns of a wider float32 matrix as one of their own
+int lse_cast_columns(const float* x, long long stride, void* out, int out_dtype, int T, int cols, cudaStream_t stream);
 
 // out[t] = x[t] + (x[t-1] - x[t]) * mix, with x[t-1] from state[slots[seq]] for a sequence's first
 // row; afterwards state[slots[seq]] = the sequence's last row of x.   x float32 [T, W]
@@ -198,10 +207,13 @@ int lse_decay_linear_attention(const float* proj, long long stride, float* out, 
 //   first), then silu; q and k divided by sqrt(sum of squares + 1e-6) per head, q times q_scale.
 //   scal [T, H, 4] = (exp(-exp(A_log) softplus(a + dt_bias)), sigmoid(b), k . q, 0)
 // qkv [T, 2 G dk + H dv]. dk <= 256.
+// With z (float32 [T, H*dk], rows z_stride apart): a decay per head and key channel, decay [T, H*dk] =
+// exp(-exp(A_log[h]) softplus(z + dt_bias[h*dk + i])); the row of proj is then q | k | v | b, and scal's first number 1.
 int lse_delta_inputs(const float* proj, long long stride, const float* conv, int taps,
                      float* conv_state, const float* A_log, const float* dt_bias, const int* token_seq,
                      const int* cu_q, const int* ctx_lens, const int* slots, float* qkv, float* scal,
-                     int T, int H, int G, int dk, int dv, float q_scale, cudaStream_t stream);
+                     int T, int H, int G, int dk, int dv, float q_scale, cudaStream_t stream,
+                     const float* z = nullptr, long long z_stride = 0, float* decay = nullptr);
 
 // S <- g S; u = beta (v - S^T k); S <- S + k u^T; out = S^T q per head and token, float32, with qkv and
 // scal as lse_delta_inputs leaves them; state [slots, H, dv, dk]; out [T, H*dv]. dk <= 256.
@@ -209,12 +221,13 @@ int lse_delta_inputs(const float* proj, long long stride, const float* conv, int
 // a bound on any sequence's chunks, is above one: scratch then holds total_chunks times
 // lse_delta_rule_chunk_floats() floats, total_chunks at least the chunks of all such sequences
 // together; short_too: the step may also hold shorter portions (one more launch).
+// decay [T, H*dk]: row d of S is multiplied by decay[t, h*dk + d] instead of scal's number (null: that number).
 int lse_delta_rule_chunk(void);
-size_t lse_delta_rule_chunk_floats(int H, int dk, int dv);
+size_t lse_delta_rule_chunk_floats(int H, int dk, int dv, int channels = 0);  // channels: with decay
 int lse_delta_rule(const float* qkv, const float* scal, float* state, float* out, const int* cu_q,
                    const int* ctx_lens, const int* slots, int num_seqs, int H, int G, int dk, int dv,
                    cudaStream_t stream, int max_chunks = 1, float* scratch = nullptr, int total_chunks = 0,
-                   int short_too = 1);
+                   int short_too = 1, const float* decay = nullptr);
 
 // ---- several residual streams, rows of q/k/v prepared a token at a time, differential attention
 // (streams_mixers.cu). The residual state is float32 [T, S * W]: a token's S streams of W values.
@@ -297,7 +310,8 @@ int lse_head_linear(const void* a, int a_dtype, long long a_stride, long long a_
 //     first, the lower index on a tie). mode 0: wts = sigmoid(z) of the chosen; mode 1: wts = the
 //     softmax over the chosen z alone. mode 2: s = softmax(z) over all E; chosen by the largest
 //     s + bias among the `keep` best of `groups` equal groups of neighbours (a group's score is its
-//     largest s + bias; bias is no part of z); wts = s / (sum of the chosen s + 1e-20) * scale.
+//     largest s + bias; bias is no part of z); wts = s / (sum of the chosen s + 1e-20) * scale, or s * scale
+//     without `normalise`.
 //     With has_gate, gate[t] = sigmoid(router[E] . h).
 //   lse_moe_sort: the n = T * top choices sorted by expert: offsets [E + 1], perm [n] (sorted row ->
 //     choice), pos_of [n] (choice -> sorted row), and tiles of at most lse_moe_tile_rows() rows of one
@@ -310,10 +324,12 @@ int lse_head_linear(const void* a, int a_dtype, long long a_stride, long long a_
 //     (kinds 1 and 2 multiply the float32 sums by a_scale, which is the same product).
 //   lse_moe_combine: out[t] (+)= sum_k wts[t*top + k] * y[pos_of[t*top + k]] (+ gate[t] * shared_out[t]);
 //     wts null: 1; gate null: 1. A choice with pos_of < 0 adds wts * h[t] (h [T, W]; null: nothing).
+//     The whole sum is multiplied by `scale` before it is added or stored.
 int lse_moe_tile_rows(void);
 int lse_moe_route(const void* h, int h_dtype, const float* router, int T, int W, int E, int has_gate,
                   int top, int* idx, float* wts, float* gate, cudaStream_t stream,
-                  const float* bias = nullptr, int mode = 0, int groups = 1, int keep = 1, float scale = 1.f);
+                  const float* bias = nullptr, int mode = 0, int groups = 1, int keep = 1, float scale = 1.f,
+                  int normalise = 1);
 int lse_moe_sort(const int* idx, int n, int E, int tile_rows, int* offsets, int* perm, int* pos_of,
                  int* tile_batch, int* tile_row0, int* num_tiles, cudaStream_t stream);
 // out[r] = a[perm[r] / top] for the n sorted rows (bfloat16, K a multiple of 8)
@@ -333,7 +349,7 @@ int lse_expert_linear(const void* a, int a_dtype, long long a_stride, const int*
                       const int* num_tiles, int max_tiles, int kind, cudaStream_t stream);
 int lse_moe_combine(const float* y, const int* pos_of, int top, const float* shared_out,
                     const float* gate, float* out, int accumulate, int T, int W, cudaStream_t stream,
-                    const float* wts = nullptr, const void* h = nullptr, int h_dtype = LSE_F32);
+                    const float* wts = nullptr, const void* h = nullptr, int h_dtype = LSE_F32, float scale = 1.f);
 
 // Latent attention with a rotated key part (rotary_latent.cu). cos/sin: float32 [positions, rot/2];
 // neighbouring dims (2i, 2i+1) are a pair; of a part's Dr dims the first rot are turned.

@@ -362,15 +362,31 @@ __global__ void __launch_bounds__(MM_THREADS) rows_gemm_mma_kernel(const RowsGem
 // in a fixed order, so a row's result does not depend on the batch.
 constexpr int GV_WARPS = 8, GV_ROWS = 4, GV_CPW = 4, GV_COLS = GV_WARPS * GV_CPW;  // columns per block
 
-template <typename TO, int RN>
-__device__ __forceinline__ void gemv_rows(const RowsGemm& g, const bf16* a, const bf16* w, TO* out,
+__device__ __forceinline__ void load8(const bf16* p, float (&v)[8]) {
+  const Vec16<bf16> t = load16(p);
+#pragma unroll
+  for (int e = 0; e < 8; ++e) v[e] = __bfloat162float(t.v[e]);
+}
+__device__ __forceinline__ void load8(const float* p, float (&v)[8]) {
+  float lo[4], hi[4];
+  load4<float>(p, lo);
+  load4<float>(p + 4, hi);
+#pragma unroll
+  for (int e = 0; e < 4; ++e) {
+    v[e] = lo[e];
+    v[e + 4] = hi[e];
+  }
+}
+
+template <typename TO, typename TA, int RN>
+__device__ __forceinline__ void gemv_rows(const RowsGemm& g, const TA* a, const bf16* w, TO* out,
                                           const int* srow, const float* sscale, int m0, int r0, int rows,
                                           int n, int lane) {
   const int K = g.K, N = g.N;
   const bf16* wr[GV_CPW];
 #pragma unroll
   for (int c = 0; c < GV_CPW; ++c) wr[c] = w + (size_t)min(n + c, N - 1) * K;
-  const bf16* ar[RN];
+  const TA* ar[RN];
 #pragma unroll
   for (int r = 0; r < RN; ++r) ar[r] = a + (size_t)srow[min(r0 + r, rows - 1)] * g.a_stride;
   float acc[GV_CPW][RN];
@@ -389,11 +405,13 @@ __device__ __forceinline__ void gemv_rows(const RowsGemm& g, const bf16* a, cons
     }
 #pragma unroll
     for (int r = 0; r < RN; ++r) {
-      const Vec16<bf16> a0 = load16(ar[r] + k), a1 = load16(ar[r] + (more ? k2 : k));
+      float a0[8], a1[8];
+      load8(ar[r] + k, a0);
+      load8(ar[r] + (more ? k2 : k), a1);
 #pragma unroll
       for (int e = 0; e < 8; ++e) {
-        const float x0 = __bfloat162float(a0.v[e]);
-        const float x1 = more ? __bfloat162float(a1.v[e]) : 0.f;
+        const float x0 = a0[e];
+        const float x1 = more ? a1[e] : 0.f;
 #pragma unroll
         for (int c = 0; c < GV_CPW; ++c) {
           acc[c][r] = fmaf(x0, __bfloat162float(wv[0][c].v[e]), acc[c][r]);
@@ -412,7 +430,7 @@ __device__ __forceinline__ void gemv_rows(const RowsGemm& g, const bf16* a, cons
     }
 }
 
-template <typename TO>
+template <typename TO, typename TA>
 __global__ void __launch_bounds__(GV_WARPS * 32, 2) rows_gemv_kernel(const RowsGemm g) {
   pdl_trigger();
   pdl_wait();  // everything below reads what kernels before this one wrote
@@ -436,7 +454,7 @@ __global__ void __launch_bounds__(GV_WARPS * 32, 2) rows_gemv_kernel(const RowsG
   __syncthreads();
   const int rows = m_end - m0;
   if (rows <= 0) return;
-  const bf16* a = (const bf16*)g.a + g.a_col0 + (long long)batch * g.a_batch_cols;
+  const TA* a = (const TA*)g.a + g.a_col0 + (long long)batch * g.a_batch_cols;
   const bf16* w = (const bf16*)g.w + (long long)batch * g.w_batch_stride;
   TO* out = (TO*)g.out + (long long)batch * g.out_batch_cols;
   const int warp = tid >> 5, lane = tid & 31;
@@ -444,9 +462,9 @@ __global__ void __launch_bounds__(GV_WARPS * 32, 2) rows_gemv_kernel(const RowsG
   if (n >= g.N) return;
   for (int r0 = 0; r0 < rows; r0 += GV_ROWS) {
     const int left = rows - r0;
-    if (left == 1) gemv_rows<TO, 1>(g, a, w, out, srow, sscale, m0, r0, rows, n, lane);
-    else if (left == 2) gemv_rows<TO, 2>(g, a, w, out, srow, sscale, m0, r0, rows, n, lane);
-    else gemv_rows<TO, GV_ROWS>(g, a, w, out, srow, sscale, m0, r0, rows, n, lane);
+    if (left == 1) gemv_rows<TO, TA, 1>(g, a, w, out, srow, sscale, m0, r0, rows, n, lane);
+    else if (left == 2) gemv_rows<TO, TA, 2>(g, a, w, out, srow, sscale, m0, r0, rows, n, lane);
+    else gemv_rows<TO, TA, GV_ROWS>(g, a, w, out, srow, sscale, m0, r0, rows, n, lane);
   }
 }
 
@@ -459,7 +477,8 @@ __global__ void __launch_bounds__(GV_WARPS * 32, 2) rows_gemv_kernel(const RowsG
 // (mode 1). Row E of the router, if there is one, is the shared expert's gate.
 // Mode 2: scores s = softmax(z) over all E; the choice goes by c = s + bias, which is then not part
 // of z; the experts form `groups` equal groups of neighbours, of which only the `keep` with the
-// largest c in them can be chosen from; a chosen expert's weight is s / (sum of the chosen s + 1e-20) * scale.
+// largest c in them can be chosen from; a chosen expert's weight is s / (sum of the chosen s + 1e-20) * scale, or
+// s * scale without `normalise`.
 constexpr int ROUTE_WARPS = 8;
 
 template <typename TH>
@@ -467,7 +486,7 @@ __global__ void __launch_bounds__(ROUTE_WARPS * 32)
 moe_route_kernel(const TH* __restrict__ h, const float* __restrict__ router, int W, int E,
                  int has_gate, int top, int* __restrict__ idx, float* __restrict__ wts,
                  float* __restrict__ gate, const float* __restrict__ bias, int mode, int groups, int keep,
-                 float scale) {
+                 float scale, int normalise) {
   pdl_trigger();
   pdl_wait();  // everything below reads what kernels before this one wrote
   extern __shared__ float s[];  // [E + 1] scores, then [E + 1][ROUTE_WARPS] partial sums
@@ -563,7 +582,7 @@ moe_route_kernel(const TH* __restrict__ h, const float* __restrict__ router, int
   if (mode == 1)
     for (int k = lane; k < top; k += 32) wts[t * top + k] /= total;
   if (mode == 2)
-    for (int k = lane; k < top; k += 32) wts[t * top + k] = wts[t * top + k] / (total + 1e-20f) * scale;
+    for (int k = lane; k < top; k += 32) wts[t * top + k] = (normalise ? wts[t * top + k] / (total + 1e-20f) : wts[t * top + k]) * scale;
 }
 
 // One block. A choice idx[i] >= E is an identity expert: it has no row in the sorted order
@@ -637,7 +656,7 @@ moe_gather_rows_kernel(const bf16* __restrict__ a, const int* __restrict__ perm,
 
 // x[t] (or out[t]) (+)= sum_k wts[t * top + k] * y[pos_of[t * top + k]] + gate[t] * shared[t] (a
 // null wts or gate counts as ones; a choice without a row, pos_of < 0, is an identity expert and adds
-// wts times the token's row of h); a block per token and
+// wts times the token's row of h), the sum times `scale`; a block per token and
 // slice of 512 columns, four columns per thread (the experts' rows are added in the order k = 0, 1, ...)
 constexpr int COMBINE_SLICE = 512;
 
@@ -646,7 +665,7 @@ __global__ void __launch_bounds__(128)
 moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ pos_of, int top,
                    const float* __restrict__ shared_out, const float* __restrict__ gate,
                    float* __restrict__ out, int accumulate, int W, const float* __restrict__ wts,
-                   const TH* __restrict__ h) {
+                   const TH* __restrict__ h, float scale) {
   pdl_trigger();
   pdl_wait();  // everything below reads what kernels before this one wrote
   const int t = blockIdx.x;
@@ -681,6 +700,7 @@ moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ pos_of, 
     float r = v[j];
     if (shared_out) r += g * shared_out[(size_t)t * W + i];
     float* o = out + (size_t)t * W + i;
+    r *= scale;
     *o = accumulate ? *o + r : r;
   }
 }
@@ -734,7 +754,7 @@ extern "C" int lse_latent_write(const void* proj, int in_dtype, long long stride
 }
 
 // kind: 0 = CUDA cores (any operands), 1 = mma.sync tiles, 2 = few rows per tile (1 and 2: bfloat16
-// operands of whole 16-byte vectors; they multiply the result by a_scale instead of the input)
+// operands of whole 16-byte vectors, 2 also float32 rows; they multiply the result by a_scale instead of the input)
 static bool vectors_ok(const RowsGemm& g) {
   return g.K % 8 == 0 && g.a_stride % 8 == 0 && g.a_col0 % 8 == 0 && g.a_batch_cols % 8 == 0 &&
          reinterpret_cast<uintptr_t>(g.a) % 16 == 0 && reinterpret_cast<uintptr_t>(g.w) % 16 == 0;
@@ -750,9 +770,14 @@ static int launch_rows_gemm(const RowsGemm& g, int a_dtype, int w_dtype, int out
       else launch(rows_gemm_mma_kernel<bf16>, grid, MM_THREADS, 0, stream, g);
     } else {
       grid.x = (g.N + GV_COLS - 1) / GV_COLS;
-      if (out_dtype == LSE_F32) launch(rows_gemv_kernel<float>, grid, GV_WARPS * 32, 0, stream, g);
-      else launch(rows_gemv_kernel<bf16>, grid, GV_WARPS * 32, 0, stream, g);
+      if (out_dtype == LSE_F32) launch(rows_gemv_kernel<float, bf16>, grid, GV_WARPS * 32, 0, stream, g);
+      else launch(rows_gemv_kernel<bf16, bf16>, grid, GV_WARPS * 32, 0, stream, g);
     }
+    return LSE_CHECK_LAUNCH();
+  }
+  if (kind == 2 && a_dtype == LSE_F32 && w_dtype == LSE_BF16 && out_dtype == LSE_F32 && vectors_ok(g)) {
+    grid.x = (g.N + GV_COLS - 1) / GV_COLS;  // unrounded rows beside bfloat16 weights
+    launch(rows_gemv_kernel<float, float>, grid, GV_WARPS * 32, 0, stream, g);
     return LSE_CHECK_LAUNCH();
   }
 #define LSE_RG(TA, TW, TO) launch(rows_gemm_kernel<TA, TW, TO>, grid, 256, 0, stream, g)
@@ -806,7 +831,7 @@ extern "C" int lse_expert_linear(const void* a, int a_dtype, long long a_stride,
 extern "C" int lse_moe_route(const void* h, int h_dtype, const float* router, int T, int W, int E,
                              int has_gate, int top, int* idx, float* wts, float* gate,
                              cudaStream_t stream, const float* bias, int mode, int groups, int keep,
-                             float scale) {
+                             float scale, int normalise) {
   if (T <= 0) return LSE_OK;
   if (E <= 0 || top <= 0 || top > E || E > 1024 || (has_gate && !gate) || mode < 0 || mode > 2) return LSE_BAD_ARGUMENT;
   if (mode == 2 && (groups < 1 || E % groups || keep < 1 || keep > groups || top > keep * (E / groups)))
@@ -814,10 +839,10 @@ extern "C" int lse_moe_route(const void* h, int h_dtype, const float* router, in
   const size_t smem = (size_t)(E + 1) * (1 + ROUTE_WARPS) * sizeof(float);
   if (h_dtype == LSE_F32)
     launch(moe_route_kernel<float>, T, ROUTE_WARPS * 32, smem, stream, (const float*)h, router, W, E, has_gate, top,
-                                                                   idx, wts, gate, bias, mode, groups, keep, scale);
+                                                                   idx, wts, gate, bias, mode, groups, keep, scale, normalise);
   else if (h_dtype == LSE_BF16)
     launch(moe_route_kernel<bf16>, T, ROUTE_WARPS * 32, smem, stream, (const bf16*)h, router, W, E, has_gate, top,
-                                                                  idx, wts, gate, bias, mode, groups, keep, scale);
+                                                                  idx, wts, gate, bias, mode, groups, keep, scale, normalise);
   else
     return LSE_BAD_ARGUMENT;
   return LSE_CHECK_LAUNCH();
@@ -845,15 +870,15 @@ extern "C" int lse_moe_gather_rows(const void* a, const int* perm, int top, void
 
 extern "C" int lse_moe_combine(const float* y, const int* pos_of, int top, const float* shared_out,
                                const float* gate, float* out, int accumulate, int T, int W,
-                               cudaStream_t stream, const float* wts, const void* h, int h_dtype) {
+                               cudaStream_t stream, const float* wts, const void* h, int h_dtype, float scale) {
   if (T <= 0) return LSE_OK;
   const dim3 grid(T, (W + COMBINE_SLICE - 1) / COMBINE_SLICE);
   if (h && h_dtype == LSE_BF16)
     launch(moe_combine_kernel<bf16>, grid, 128, 0, stream, y, pos_of, top, shared_out, gate, out, accumulate, W, wts,
-           (const bf16*)h);
+           (const bf16*)h, scale);
   else if (!h || h_dtype == LSE_F32)
     launch(moe_combine_kernel<float>, grid, 128, 0, stream, y, pos_of, top, shared_out, gate, out, accumulate, W, wts,
-           (const float*)h);
+           (const float*)h, scale);
   else
     return LSE_BAD_ARGUMENT;
   return LSE_CHECK_LAUNCH();

@@ -14,7 +14,7 @@ namespace lse {
 // ------------------------------------------------------------------------------------ embedding
 template <typename T>
 __global__ void embedding_kernel(const int* __restrict__ ids, const T* __restrict__ table,
-                                 float* __restrict__ out, int H) {
+                                 float* __restrict__ out, int H, float scale) {
   pdl_trigger();
   pdl_wait();
   const int t = blockIdx.x;
@@ -27,11 +27,11 @@ __global__ void embedding_kernel(const int* __restrict__ ids, const T* __restric
 #pragma unroll
       for (int j = 0; j < V; j += 4)  // H % V == 0 and 16-byte aligned rows: whole float4 stores
         *reinterpret_cast<float4*>(dst + i + j) =
-            make_float4(Num<T>::to_float(v.v[j]), Num<T>::to_float(v.v[j + 1]),
-                        Num<T>::to_float(v.v[j + 2]), Num<T>::to_float(v.v[j + 3]));
+            make_float4(Num<T>::to_float(v.v[j]) * scale, Num<T>::to_float(v.v[j + 1]) * scale,
+                        Num<T>::to_float(v.v[j + 2]) * scale, Num<T>::to_float(v.v[j + 3]) * scale);
     }
   } else {
-    for (int i = threadIdx.x; i < H; i += blockDim.x) dst[i] = Num<T>::to_float(src[i]);
+    for (int i = threadIdx.x; i < H; i += blockDim.x) dst[i] = Num<T>::to_float(src[i]) * scale;
   }
 }
 
@@ -194,6 +194,113 @@ __global__ void add_rmsnorm_regs_kernel(float* __restrict__ x, const TR* __restr
 #pragma unroll
       for (int j = 0; j < 4; ++j) v[k][j] = v[k][j] * inv * w[k][j];
       store4<TO>(o + i, v[k]);
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------ scaled sum, norm
+// x += sum_i c_i y_i (+ row, the same for every token), in place, and out = x / rms(x) * weight where a
+// weight is given: what several sublayers of one layer leave for the next layer's norm. A y_i is a
+// float32 tensor or fixed-point sums, which are cleared as they are read. One block per token, V
+// elements per thread and visit; at most NV visits, whose values stay in registers (NV = 0: any row
+// length, x read back).
+constexpr int SUM_MAX = 4;
+struct SumItems {
+  const void* y[SUM_MAX];
+  float c[SUM_MAX];
+  int fixed[SUM_MAX];
+  int n;
+};
+
+template <typename TO, int V, int NV>
+__global__ void sum_add_rmsnorm_kernel(float* __restrict__ x, const SumItems items, const float* __restrict__ row,
+                                       const float* __restrict__ weight, float eps, TO* __restrict__ out, int H) {
+  __shared__ float scratch[32];
+  pdl_trigger();
+  constexpr int KEEP = NV > 0 ? NV : 1;
+  float w[KEEP][V], v[KEEP][V];
+  if constexpr (NV > 0) {
+    if (weight) {
+#pragma unroll
+      for (int k = 0; k < NV; ++k) {  // the weights are no result of the kernel before this one
+        const int i = (k * blockDim.x + threadIdx.x) * V;
+        if (i < H) {
+          if constexpr (V == 4) load4<float>(weight + i, w[k]);
+          else w[k][0] = weight[i];
+        }
+      }
+    }
+  }
+  pdl_wait();
+  const size_t at = (size_t)blockIdx.x * H;
+  auto sum_at = [&](int i, float (&o)[V]) {
+    if constexpr (V == 4) load4<float>(x + at + i, o);
+    else o[0] = x[at + i];
+#pragma unroll
+    for (int m = 0; m < SUM_MAX; ++m) {
+      if (m >= items.n) break;
+      float y[V];
+      if (items.fixed[m]) {
+        fixed64* p = reinterpret_cast<fixed64*>(const_cast<void*>(items.y[m])) + at + i;
+        if constexpr (V == 4) {
+          load4<fixed64>(p, y);
+        } else {
+          y[0] = fixed_to_float(p[0]);
+          p[0] = 0;
+        }
+      } else {
+        const float* p = reinterpret_cast<const float*>(items.y[m]) + at + i;
+        if constexpr (V == 4) load4<float>(p, y);
+        else y[0] = p[0];
+      }
+#pragma unroll
+      for (int j = 0; j < V; ++j) o[j] = fmaf(items.c[m], y[j], o[j]);
+    }
+    if (row) {
+#pragma unroll
+      for (int j = 0; j < V; ++j) o[j] += row[i + j];
+    }
+    if constexpr (V == 4) store4<float>(x + at + i, o);
+    else x[at + i] = o[0];
+  };
+  auto put = [&](int i, const float (&o)[V]) {
+    if constexpr (V == 4) store4<TO>(out + at + i, o);
+    else out[at + i] = Num<TO>::from_float(o[0]);
+  };
+  float ss = 0.f;
+  if constexpr (NV > 0) {
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int i = (k * blockDim.x + threadIdx.x) * V;
+      if (i >= H) continue;
+      sum_at(i, v[k]);
+#pragma unroll
+      for (int j = 0; j < V; ++j) ss += v[k][j] * v[k][j];
+    }
+  } else {
+    for (int i = threadIdx.x * V; i < H; i += blockDim.x * V) {
+      sum_at(i, v[0]);
+#pragma unroll
+      for (int j = 0; j < V; ++j) ss += v[0][j] * v[0][j];
+    }
+  }
+  if (!weight) return;
+  ss = block_sum(ss, scratch);
+  const float inv = rsqrtf(ss / (float)H + eps);
+  if constexpr (NV > 0) {
+#pragma unroll
+    for (int k = 0; k < NV; ++k) {
+      const int i = (k * blockDim.x + threadIdx.x) * V;
+      if (i >= H) continue;
+#pragma unroll
+      for (int j = 0; j < V; ++j) v[k][j] *= inv * w[k][j];
+      put(i, v[k]);
+    }
+  } else {
+    for (int i = threadIdx.x * V; i < H; i += blockDim.x * V) {  // this thread's own writes
+#pragma unroll
+      for (int j = 0; j < V; ++j) v[0][j] = x[at + i + j] * inv * weight[i + j];
+      put(i, v[0]);
     }
   }
 }
@@ -499,13 +606,13 @@ using namespace lse;
 #define LSE_CHECK_LAUNCH() (cudaPeekAtLastError() == cudaSuccess ? LSE_OK : LSE_LAUNCH_FAILED)
 
 extern "C" int lse_embedding(const int* ids, const void* table, int table_dtype, float* out, int T,
-                             int H, cudaStream_t stream) {
+                             int H, cudaStream_t stream, float scale) {
   if (T <= 0) return LSE_OK;
   const int threads = H >= 2048 ? 256 : 128;
   if (table_dtype == LSE_F32)
-    launch(embedding_kernel<float>, T, threads, 0, stream, ids, (const float*)table, out, H);
+    launch(embedding_kernel<float>, T, threads, 0, stream, ids, (const float*)table, out, H, scale);
   else if (table_dtype == LSE_BF16)
-    launch(embedding_kernel<bf16>, T, threads, 0, stream, ids, (const bf16*)table, out, H);
+    launch(embedding_kernel<bf16>, T, threads, 0, stream, ids, (const bf16*)table, out, H, scale);
   else
     return LSE_BAD_ARGUMENT;
   return LSE_CHECK_LAUNCH();
@@ -551,6 +658,40 @@ extern "C" int lse_add_rmsnorm(float* x, const void* residual, int residual_dtyp
   }
   else return LSE_BAD_ARGUMENT;
 #undef LSE_NORM
+  return LSE_CHECK_LAUNCH();
+}
+
+extern "C" int lse_sum_add_rmsnorm(float* x, const void* const* y, const float* c, const int* dtypes, int n,
+                                   const float* row, const float* weight, float eps, void* out, int out_dtype, int T,
+                                   int H, cudaStream_t stream) {
+  if (T <= 0) return LSE_OK;
+  if (!x || n < 0 || n > SUM_MAX || H <= 0 || (weight && !out)) return LSE_BAD_ARGUMENT;
+  SumItems items = {};
+  items.n = n;
+  for (int i = 0; i < n; ++i) {
+    if (!y[i] || (dtypes[i] != LSE_F32 && dtypes[i] != LSE_FIXED64)) return LSE_BAD_ARGUMENT;
+    items.y[i] = y[i];
+    items.c[i] = c[i];
+    items.fixed[i] = dtypes[i] == LSE_FIXED64;
+  }
+  const bool vec = H % 4 == 0;
+  const int per = vec ? 16 : 4, kept = H <= 1024 * per;  // elements per thread whose visits stay in registers
+  const int threads = kept ? ((H + per - 1) / per + 31) / 32 * 32 : 1024;
+#define LSE_SUM(TO)                                                                                              \
+  do {                                                                                                           \
+    if (vec && kept)                                                                                             \
+      launch(sum_add_rmsnorm_kernel<TO, 4, 4>, T, threads, 0, stream, x, items, row, weight, eps, (TO*)out, H);  \
+    else if (vec)                                                                                                \
+      launch(sum_add_rmsnorm_kernel<TO, 4, 0>, T, threads, 0, stream, x, items, row, weight, eps, (TO*)out, H);  \
+    else if (kept)                                                                                               \
+      launch(sum_add_rmsnorm_kernel<TO, 1, 4>, T, threads, 0, stream, x, items, row, weight, eps, (TO*)out, H);  \
+    else                                                                                                         \
+      launch(sum_add_rmsnorm_kernel<TO, 1, 0>, T, threads, 0, stream, x, items, row, weight, eps, (TO*)out, H);  \
+  } while (0)
+  if (!weight || out_dtype == LSE_F32) LSE_SUM(float);
+  else if (out_dtype == LSE_BF16) LSE_SUM(bf16);
+  else return LSE_BAD_ARGUMENT;
+#undef LSE_SUM
   return LSE_CHECK_LAUNCH();
 }
 

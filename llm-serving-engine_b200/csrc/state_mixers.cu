@@ -24,6 +24,17 @@ __global__ void cast_kernel(const float* __restrict__ x, TO* __restrict__ out, l
   if (i < n) out[i] = Num<TO>::from_float(x[i]);
 }
 
+template <typename TO>
+__global__ void cast_columns_kernel(const float* __restrict__ x, long long stride, TO* __restrict__ out, int cols,
+                                    long long n) {
+  pdl_trigger();
+  pdl_wait();
+  const long long i = (long long)blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= n) return;
+  const long long t = i / cols;
+  out[i] = Num<TO>::from_float(x[t * stride + (i - t * cols)]);
+}
+
 // ------------------------------------------------------------------------------------ token shift
 // One block per row. The block of a sequence's first row is the only one that touches the
 // sequence's state: each of its threads reads the old value of its elements and then stores the
@@ -829,6 +840,18 @@ extern "C" int lse_cast(const float* x, void* out, int out_dtype, long long n, c
   const unsigned blocks = (unsigned)((n + 255) / 256);
   if (out_dtype == LSE_BF16) launch(cast_kernel<bf16>, blocks, 256, 0, stream, x, (bf16*)out, n);
   else if (out_dtype == LSE_F32) launch(cast_kernel<float>, blocks, 256, 0, stream, x, (float*)out, n);
+  else return LSE_BAD_ARGUMENT;
+  return LSE_CHECK_LAUNCH();
+}
+
+extern "C" int lse_cast_columns(const float* x, long long stride, void* out, int out_dtype, int T, int cols,
+                                cudaStream_t stream) {
+  const long long n = (long long)T * cols;
+  if (n <= 0) return LSE_OK;
+  if (stride < cols) return LSE_BAD_ARGUMENT;
+  const unsigned blocks = (unsigned)((n + 255) / 256);
+  if (out_dtype == LSE_BF16) launch(cast_columns_kernel<bf16>, blocks, 256, 0, stream, x, stride, (bf16*)out, cols, n);
+  else if (out_dtype == LSE_F32) launch(cast_columns_kernel<float>, blocks, 256, 0, stream, x, stride, (float*)out, cols, n);
   else return LSE_BAD_ARGUMENT;
   return LSE_CHECK_LAUNCH();
 }

@@ -11,7 +11,7 @@ from __future__ import annotations
 import torch
 
 from ..parts.base import BLOCKS, EMBED_TERMS, NORMS, POSITION_ENCODINGS, BuildEnv, ParamDecl, role_dtype, settle
-from ..parts.base import count_states, flatten_needs
+from ..parts.base import count_states, flatten_needs, with_row
 from .plan import ModelPlan
 
 
@@ -31,6 +31,7 @@ class DecoderModel:
         self.embed_cache = 1 + max(e.cache for e in plan.run_order)
         self.embed_weight: torch.Tensor | None = None
         self.head_weight: torch.Tensor | None = None
+        self.run_vectors: torch.Tensor | None = None
         # which run of the order fills each cache layer
         self.writer_of: dict[int, int] = {}
         for k, e in enumerate(plan.run_order):
@@ -50,6 +51,8 @@ class DecoderModel:
             decls[f"final_norm.{name}"] = decl
         if not p.tie_head:
             decls["head.weight"] = ParamDecl((p.vocab_size, p.hidden_size), "matrix")
+        if p.run_vectors:
+            decls["run_vectors"] = ParamDecl((p.run_vectors, p.hidden_size), "offset")
         return decls
 
     def param_dtype(self, name: str) -> torch.dtype:
@@ -70,6 +73,7 @@ class DecoderModel:
                 )
         self.embed_weight = params["embed.weight"]
         self.head_weight = params["embed.weight"] if self.plan.tie_head else params["head.weight"]
+        self.run_vectors = params.get("run_vectors")
         for i, block in enumerate(self.blocks):
             prefix = f"layers.{i}."
             block.bind({k[len(prefix):]: v for k, v in params.items() if k.startswith(prefix)})
@@ -132,11 +136,11 @@ class DecoderModel:
     # ------------------------------------------------------------------ forward
     def forward(self, step, pools) -> torch.Tensor:
         """Run this step's tokens; return float32 logits ``[len(step.logit_rows), vocab]``."""
-        x = self.ops.embedding(step.token_ids, self.embed_weight)
         if self.plan.residual_streams > 1:  # every stream starts as the (scaled) embedded token
+            x = self.ops.embedding(step.token_ids, self.embed_weight)
             x = self.ops.streams_spread(x, self.plan.residual_streams, self.plan.embed_scale)
-        elif self.plan.embed_scale != 1.0:
-            x *= self.plan.embed_scale
+        else:
+            x = self.ops.embedding(step.token_ids, self.embed_weight, self.plan.embed_scale)
         if self.embed_terms:
             view, at = pools.view(self.embed_cache, writes=True), 0
             for term in self.embed_terms:
@@ -148,6 +152,8 @@ class DecoderModel:
         pending = None
         for k, e in enumerate(self.plan.run_order):
             view = pools.view(e.cache, writes=self.writer_of[e.cache] == k)
+            if e.vector is not None:
+                pending = with_row(self.ops, x, pending, self.run_vectors[e.vector])
             x, pending = self.blocks[e.layer].forward(x, pending, step, view)
         if step.num_logit_rows == 0:
             if hasattr(pending, "resolve"):

@@ -18,6 +18,7 @@ class RunEntry:
 
     layer: int
     cache: int
+    vector: int | None = None  # row of ``ModelPlan.run_vectors`` that is added to every token before this run
 
 
 @dataclass(frozen=True)
@@ -39,6 +40,9 @@ class ModelPlan:
     # copies of the embedded token that the blocks carry side by side (``streams`` blocks); the
     # residual state is then [T, residual_streams * hidden_size] and the final norm reads all of it
     residual_streams: int = 1
+    # learned vectors of the width that runs may add to the residual stream before they start (a layer that
+    # runs several times can tell its passes apart by them); runs name them by their row
+    run_vectors: int = 0
 
     def validate(self) -> None:
         if not self.run_order:
@@ -46,6 +50,10 @@ class ModelPlan:
         for e in self.run_order:
             if not 0 <= e.layer < len(self.layers):
                 raise ValueError(f"run_order names layer {e.layer}; the plan has {len(self.layers)}")
+            if e.vector is not None and not 0 <= e.vector < self.run_vectors:
+                raise ValueError(f"run_order names vector {e.vector}; the plan has {self.run_vectors}")
+        if self.run_vectors and self.residual_streams > 1:
+            raise ValueError("vectors before a run and several residual streams do not go together")
         ids = sorted({e.cache for e in self.run_order})
         if ids != list(range(len(ids))):
             raise ValueError(f"cache ids must be 0..n-1 without gaps, got {ids}")

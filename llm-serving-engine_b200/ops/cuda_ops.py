@@ -192,9 +192,9 @@ class CudaOps:
             raise RuntimeError(f"a CUDA kernel of llmserve_b200 gave up waiting (code {code})")
 
     # ------------------------------------------------------------------ pointwise
-    def embedding(self, token_ids, table):
+    def embedding(self, token_ids, table, scale=1.0):
         out = torch.empty(token_ids.shape[0], table.shape[1], dtype=torch.float32, device=table.device)
-        self.ext.embedding(token_ids, table, out)
+        self.ext.embedding(token_ids, table, out, float(scale))
         self.launches += 1
         return out
 
@@ -221,6 +221,26 @@ class CudaOps:
         if sums is not None:
             self._sums_taken(sums)
         return out
+
+    def sum_add_rmsnorm(self, x, items, row, weight, eps, out_dtype):
+        """``x += sum_i c_i y_i (+ row)`` in place (``items``: pairs ``(c_i, y_i)`` of a factor and a float32 tensor
+        or a :class:`DeferredProduct`; ``row``: a vector added to every token), and the norm of the new ``x``
+        (``weight`` None: nothing is normed), in one launch."""
+        while len(items) > 4:  # more than the kernel takes at once
+            self.sum_add(x, items[:4], None)
+            items = items[4:]
+        out = None if weight is None else torch.empty(x.shape, dtype=out_dtype, device=x.device)
+        taken = [y for _, y in items if isinstance(y, DeferredProduct)]
+        tensors = [y.sums if isinstance(y, DeferredProduct) else y if y.dtype == torch.float32 else y.float() for _, y in items]
+        self.ext.sum_add_rmsnorm(x, tensors, [float(c) for c, _ in items], row, weight, float(eps), out)
+        self.launches += 1
+        for y in taken:
+            self._sums_taken(y.sums)
+            y.sums = None
+        return out
+
+    def sum_add(self, x, items, row) -> None:
+        self.sum_add_rmsnorm(x, items, row, None, 0.0, None)
 
     # ------------------------------------------------------------------ fixed-point sums
     def _product_sums(self, a, w, bias) -> torch.Tensor:
@@ -259,13 +279,17 @@ class CudaOps:
         return (self.use_skinny_gemm and a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16
                 and a.shape[0] <= self.skinny_max_rows and a.shape[1] % 8 == 0)
 
-    def linear(self, a, w, bias=None, out_dtype=None, accumulate_into=None, may_defer=False):
+    def linear(self, a, w, bias=None, out_dtype=None, accumulate_into=None, may_defer=False, coefficient=None):
         """``a @ w.T (+ bias)`` as a new tensor of ``out_dtype`` (None: the compute dtype).
 
         With ``accumulate_into`` (a float32 tensor of the result's shape) the product may be
         added into that tensor instead; the return value is then None. A caller that passes
         ``may_defer=True`` may get a :class:`PendingSums` instead, which it has to hand on to
         whoever reads ``accumulate_into`` next.
+
+        ``coefficient``: what may be added into ``accumulate_into`` is ``coefficient`` times the product;
+        whatever is returned instead is the product as it is (with ``may_defer`` perhaps a
+        :class:`DeferredProduct`).
         """
         if a.dtype == torch.float32:
             if w.dtype != torch.float32:
@@ -282,7 +306,7 @@ class CudaOps:
             # few rows: the weights are streamed once through the tcgen05 kernel, work balanced
             # over all SMs, partial sums added as fixed-point numbers
             sums = self._product_sums(a, w, bias)
-            if accumulate_into is not None:
+            if accumulate_into is not None and coefficient is None:
                 pending = PendingSums(self, sums, accumulate_into)
                 return pending if may_defer else pending.resolve()
             if may_defer and out_dtype == torch.float32:
@@ -295,7 +319,8 @@ class CudaOps:
         if accumulate_into is not None and bias is None and self._addmm_in_place is not False:
             # many rows: the library adds the product into the residual stream (beta = 1)
             try:
-                torch.addmm(accumulate_into, a, w.t(), out_dtype=torch.float32, out=accumulate_into)
+                torch.addmm(accumulate_into, a, w.t(), out_dtype=torch.float32, out=accumulate_into,
+                            alpha=1.0 if coefficient is None else float(coefficient))
                 self._addmm_in_place = True
                 return None
             except (RuntimeError, TypeError):
@@ -420,12 +445,13 @@ class CudaOps:
 
     def paged_attention(self, q, *, num_heads, num_kv_heads, head_dim, scale, window, k_pages,
                         v_pages, block_tables, page_tokens, step, plan, head_scale=None, slopes=None,
-                        chunk=0, sinks=None, keep_first=0, out_dtype=None):
+                        chunk=0, sinks=None, keep_first=0, out_dtype=None, softcap=0.0):
         """``head_scale`` / ``slopes`` (float32 ``[heads]``) and ``chunk``: a factor per head on the
         score, ``slope_h * (i - j)`` taken off it, and keys limited to the query's chunk. ``sinks``
         (float32 ``[heads]``): ``exp(sink_h)`` joins the softmax's denominator. ``keep_first``: with
         a window, the sequence's first ``keep_first`` keys stay visible beside the window's.
-        ``out_dtype=torch.float32`` beside bfloat16 queries: the results are handed on unrounded."""
+        ``out_dtype=torch.float32`` beside bfloat16 queries: the results are handed on unrounded.
+        ``softcap``: the scaled score ``s`` becomes ``softcap * tanh(s / softcap)``."""
         out = torch.empty(q.shape[0], num_heads * head_dim, dtype=out_dtype or q.dtype, device=q.device)
         n_tiles = int(plan["tiles"].shape[0])
         n_dec = int(plan["decode_seqs"].shape[0])
@@ -441,6 +467,7 @@ class CudaOps:
             plan["tiles"] if n_tiles else None, n_tiles,
             plan["decode_seqs"] if n_dec else None, n_dec, splits, scratch,
             self.attention_kernel, head_scale, slopes, int(chunk), sinks, int(keep_first) if window else 0,
+            float(softcap),
         )
         self.launches += (1 if n_tiles else 0) + (1 if n_dec else 0)
         return out
@@ -575,20 +602,20 @@ class CudaOps:
     _ROUTER_WEIGHTS = {"sigmoid": 0, "softmax_of_chosen": 1, "softmax_of_all": 2}
 
     def moe_route(self, h, router, num_experts, top, has_gate, bias=None, weights="sigmoid", groups=1, keep=1,
-                  scale=1.0):
+                  scale=1.0, normalise=True):
         """Router logits (+ ``bias``) in float32; returns (the ``top`` experts with the largest
         logits ``[T, top]`` int32, their weights ``[T, top]``, the shared expert's gate ``[T]`` or
         None). ``weights``: ``sigmoid`` of each chosen logit, or ``softmax_of_chosen``: the softmax
         over the chosen logits alone, or ``softmax_of_all``: scores ``s`` are the softmax over all
         logits, ``bias`` is added to the scores for the choice only, which is limited to the
         ``keep`` best of ``groups`` equal groups of neighbours, and a chosen expert's weight is
-        ``s / (sum of the chosen s + 1e-20) * scale``."""
+        ``s / (sum of the chosen s + 1e-20) * scale``, or ``s * scale`` without ``normalise``."""
         T = h.shape[0]
         idx = torch.empty(T, top, dtype=torch.int32, device=h.device)
         wts = torch.empty(T, top, dtype=torch.float32, device=h.device)
         gate = torch.empty(T, dtype=torch.float32, device=h.device) if has_gate else None
         self.ext.moe_route(h, router, int(num_experts), int(top), idx, wts, gate, bias, self._ROUTER_WEIGHTS[weights],
-                           int(groups), int(keep), float(scale))
+                           int(groups), int(keep), float(scale), bool(normalise))
         self.launches += 1
         return idx, wts, gate
 
@@ -629,15 +656,16 @@ class CudaOps:
         self.launches += 1
         return out
 
-    def moe_combine(self, y, plan, top, shared, gate, residual, wts=None, identity=None):
+    def moe_combine(self, y, plan, top, shared, gate, residual, wts=None, identity=None, scale=1.0):
         """Per token the sum of its experts' rows of ``y``, each times its weight if ``wts``
         ``[T, top]`` is given, (+ gate * shared; no gate: + shared): added into ``residual``
-        (returns None) or returned. ``identity`` ``[T, W]``: what an identity expert hands on."""
+        (returns None) or returned. ``identity`` ``[T, W]``: what an identity expert hands on. The sum is
+        multiplied by ``scale``."""
         work, num_experts = plan.work, plan.num_experts
         T = y.shape[0] // top
         out = residual if residual is not None else torch.empty(T, y.shape[1], dtype=torch.float32, device=y.device)
         self.ext.moe_combine(y, work, int(num_experts), int(top), shared, gate if shared is not None else None,
-                             out, residual is not None, wts, identity)
+                             out, residual is not None, wts, identity, float(scale))
         self.launches += 1
         return None if residual is not None else out
 
@@ -756,25 +784,43 @@ class CudaOps:
         return out
 
     # ------------------------------------------------------------------ gated delta rule
+    def inner_linear(self, proj, col0, w, dtype):
+        """Products of neighbouring runs of columns of the float32 ``proj`` with a matrix each: ``w`` ``[H, N, K]``, run
+        h at ``col0 + h * K``; float32 ``[T, H * N]``. bfloat16 weights: few rows meet them unrounded,
+        many rows as bfloat16."""
+        T, (H, N, K) = proj.shape[0], w.shape
+        if dtype == torch.bfloat16 and T > self.skinny_max_rows:
+            low = torch.empty(T, H * K, dtype=dtype, device=proj.device)
+            self.ext.cast_columns(proj, int(col0), low)
+            self.launches += 1
+            return self.head_linear(low, 0, w, torch.float32)
+        return self.head_linear(proj, col0, w, torch.float32, kind=2 if dtype == torch.bfloat16 else 0)
+
     def delta_inputs(self, proj, col0, *, num_heads, num_kv_heads, key_dim, value_dim, conv, conv_state, A_log,
-                     dt_bias, query_scale, step):
+                     dt_bias, query_scale, step, decay_logits=None):
         """From the columns ``q | k | v | gate | b | a`` of the float32 ``proj`` (from ``col0`` on): short
         convolution over time (``conv [taps, channels]``; ``conv_state`` keeps each request's last
         inputs) and silu of q, k and v, unit norms of q (times ``query_scale``) and k, the decay and
-        step size. Returns ``(qkv [T, channels], scal [T, heads, 4])`` for :meth:`delta_rule`."""
+        step size. Returns ``(qkv [T, channels], scal [T, heads, 4])`` for :meth:`delta_rule`. With
+        ``decay_logits`` (float32 ``[T, >= heads * key_dim]``) the columns are ``q | k | v | b``, ``dt_bias`` is as long,
+        and the decays per channel ``[T, heads * key_dim]`` are returned as a third tensor."""
         T, C = proj.shape[0], conv.shape[1]
         qkv = torch.empty(T, C, dtype=torch.float32, device=proj.device)
         scal = torch.empty(T, num_heads, 4, dtype=torch.float32, device=proj.device)
+        decay = None
+        if decay_logits is not None:
+            decay = torch.empty(T, num_heads * key_dim, dtype=torch.float32, device=proj.device)
         self.ext.delta_inputs(proj, int(col0), conv, conv_state, A_log, dt_bias, step.token_seq, step.cu_q, step.ctx_lens,
                               step.state_slots, qkv, scal, int(num_heads), int(num_kv_heads), int(key_dim),
-                              int(value_dim), float(query_scale))
+                              int(value_dim), float(query_scale), decay_logits, decay)
         self.launches += 1
-        return qkv, scal
+        return (qkv, scal) if decay is None else (qkv, scal, decay)
 
-    def delta_rule(self, qkv, scal, *, num_heads, num_kv_heads, key_dim, value_dim, state, step):
+    def delta_rule(self, qkv, scal, *, num_heads, num_kv_heads, key_dim, value_dim, state, step, decay=None):
         """``S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q`` per head and token, from each
         request's ``state [slots, heads, value_dim, key_dim]``; returns ``o [T, heads * value_dim]``.
-        Portions longer than the kernel's chunk run as chunks (three launches and a scratch)."""
+        Portions longer than the kernel's chunk run as chunks (three launches and a scratch). ``decay``
+        ``[T, heads * key_dim]``: row d of S is multiplied by its channel's decay instead of ``scal``'s number."""
         T = qkv.shape[0]
         out = torch.empty(T, num_heads * value_dim, dtype=torch.float32, device=qkv.device)
         L = self._delta_chunk = getattr(self, "_delta_chunk", None) or int(self.ext.delta_rule_chunk())
@@ -784,10 +830,11 @@ class CudaOps:
         max_chunks, scratch = max(1, -(-longest // L)), None
         short_too = host is None or int(host.q_lens.min()) <= L
         if max_chunks > 1:
-            need = (T // L + seqs) * int(self.ext.delta_rule_chunk_floats(int(num_heads), int(key_dim), int(value_dim)))
+            need = (T // L + seqs) * int(self.ext.delta_rule_chunk_floats(
+                int(num_heads), int(key_dim), int(value_dim), decay is not None))
             scratch = self._kept_scratch("delta_rule", need)
         self.ext.delta_rule(qkv, scal, state, out, step.cu_q, step.ctx_lens, step.state_slots, int(num_heads),
-                            int(num_kv_heads), int(key_dim), int(value_dim), max_chunks, scratch, short_too)
+                            int(num_kv_heads), int(key_dim), int(value_dim), max_chunks, scratch, short_too, decay)
         self.launches += (3 if max_chunks > 1 else 0) + (1 if short_too else 0)
         return out
 

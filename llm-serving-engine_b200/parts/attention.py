@@ -35,7 +35,8 @@ Further options of the spec, all off by default:
 * ``qk_norm_scope="row"``: the q/k norm runs over all of a token's query rows at once (and over
   all of its key rows), with weights of that size, instead of head by head;
 * ``sinks``: a learned number per query head whose exponential joins the softmax's denominator
-  without a key or a value.
+  without a key or a value;
+* ``softcap``: the scaled score ``s`` becomes ``softcap * tanh(s / softcap)``.
 
 A rotation that pairs neighbouring dims (``RotarySpec.pairing``) becomes one of halves by an order of
 each query and key head's rows that is applied when the weights are bound.
@@ -53,7 +54,7 @@ from typing import Any
 
 import torch
 
-from .base import MIXERS, POSITION_ENCODINGS, Mixer, PagedKVNeed, ParamDecl, project_into
+from .base import MIXERS, POSITION_ENCODINGS, Mixer, PagedKVNeed, ParamDecl, add_projected, project_into
 from .positions import neighbours_to_halves
 
 
@@ -89,6 +90,7 @@ class AttentionSpec:
     o_bias: bool | None = None  # None: as bias
     qk_norm_scope: str = "head"  # "row": one norm over all query rows of a token, one over all key rows
     sinks: bool = False
+    softcap: float = 0.0  # 0: none
     kind: str = "attention"
 
 
@@ -120,7 +122,8 @@ class PagedAttention(Mixer):
         # whole-row norms, partly rotated heads, and any heads without a norm per head that the plain path does not
         # serve, go through the kernel that prepares a token's rows at once
         options = (spec.values_are_keys or spec.head_temperature or spec.distance_slopes is not None or spec.chunk > 0
-                   or self.value_dim != spec.head_dim or spec.gate == "head" or spec.sinks or spec.head_dim % 16 != 0)
+                   or self.value_dim != spec.head_dim or spec.gate == "head" or spec.sinks or spec.softcap > 0
+                   or spec.head_dim % 16 != 0)
         self.by_rows = ((spec.qk_norm_scope == "row" and spec.qk_norm_eps is not None)
                         or (self.rotary is not None and self.rot_dims != spec.head_dim)
                         or (spec.qk_norm_eps is None and options and not spec.bias and not spec.keep_first
@@ -131,7 +134,7 @@ class PagedAttention(Mixer):
         self.extended = (spec.qk_norm_eps is not None or spec.values_are_keys or spec.head_temperature
                          or spec.distance_slopes is not None or spec.chunk > 0
                          or self.value_dim != spec.head_dim or spec.keep_first > 0 or spec.gate != "none"
-                         or spec.sinks or spec.head_dim % 16 != 0 or self.by_rows)
+                         or spec.sinks or spec.softcap > 0 or spec.head_dim % 16 != 0 or self.by_rows)
         # The attention kernels take head sizes that are multiples of 16. With the score options on,
         # any other head size is padded with zeros up to the next one when the weights are bound:
         # zero dims change no dot product, the norm divides by the true size, and the padded dims
@@ -141,6 +144,7 @@ class PagedAttention(Mixer):
         self.pad = self.kernel_dim - spec.head_dim  # of a query or key head; a value head's may differ
         if self.pad and self.rotary is not None and not self.by_rows:
             raise NotImplementedError("a padded head size with rotary positions")
+        self._cap = {"softcap": spec.softcap} if spec.softcap > 0 else {}
         self.slopes = None
         if spec.distance_slopes is not None:
             if len(spec.distance_slopes) != spec.num_heads:
@@ -284,21 +288,31 @@ class PagedAttention(Mixer):
     def input_weight(self, w):
         self.qkv_weight = w
 
-    def forward_projected(self, proj, col0, step, cache, may_defer=False):
-        """As ``forward`` from the float32 product with the input, whose columns for this mixer start at ``col0``."""
+    def forward_projected(self, proj, col0, step, cache, may_defer=False, add_to=None):
+        """As ``forward`` from the float32 product with the input, whose columns for this mixer start at ``col0``;
+        with ``add_to = (x, coefficient)`` as ``forward_into``."""
         cos, sin = self.rotary if self.rotary is not None else (None, None)
         o = self._by_rows(proj, step, cache, step.block_tables[cache.group], cos, sin, col0)
+        if add_to is not None:
+            return add_projected(self.ops, o, self.o_weight, self.o_bias, *add_to)
         return project_into(self.ops, o, self.o_weight, self.o_bias, self.env.residual_dtype, None, may_defer)
 
+    def forward_into(self, h, step, cache, x, coefficient):
+        return add_projected(self.ops, self._attend(h, step, cache), self.o_weight, self.o_bias, x, coefficient)
+
     def forward(self, h, step, cache, residual=None, may_defer=False):
+        return project_into(self.ops, self._attend(h, step, cache), self.o_weight, self.o_bias, self.env.residual_dtype,
+                            residual, may_defer)
+
+    def _attend(self, h, step, cache):
+        """The concatenated heads."""
         s = self.spec
         ops = self.ops
         tables = step.block_tables[cache.group]
         cos, sin = self.rotary if self.rotary is not None else (None, None)
         if self.extended:
-            o = self._extended(h, step, cache, tables, cos, sin)
-            return project_into(ops, o, self.o_weight, self.o_bias, self.env.residual_dtype, residual, may_defer)
-        o = ops.project_attend(
+            return self._extended(h, step, cache, tables, cos, sin)
+        return ops.project_attend(
             h, self.qkv_weight, self.qkv_bias,
             num_heads=s.num_heads,
             num_kv_heads=s.num_kv_heads,
@@ -318,7 +332,6 @@ class PagedAttention(Mixer):
             plan=step.plans[self.plan_key()],
             out_dtype=self.env.dtype,
         )
-        return project_into(ops, o, self.o_weight, self.o_bias, self.env.residual_dtype, residual, may_defer)
 
     def _extended(self, h, step, cache, tables, cos, sin):
         """Projection (its sums unrounded), norm / rotation / cache write, attention with the
@@ -340,7 +353,7 @@ class PagedAttention(Mixer):
             window=s.window, k_pages=cache.k, v_pages=cache.v, block_tables=tables,
             page_tokens=cache.page_tokens, step=step, plan=step.plans[self.plan_key()],
             head_scale=self.temperature, slopes=self.slopes, chunk=s.chunk, keep_first=s.keep_first,
-            sinks=self.sinks)
+            sinks=self.sinks, **self._cap)
         if s.gate != "none":  # the gate's columns follow v's in the projection's rows
             col0 = (s.num_heads + s.num_kv_heads * (1 if s.values_are_keys else 2)) * self.kernel_dim
             ops.sigmoid_gate_mul(o, qkv, col0, 1 if s.gate == "element" else self.kernel_dim)
@@ -363,7 +376,7 @@ class PagedAttention(Mixer):
             q, num_heads=s.num_heads, num_kv_heads=s.num_kv_heads, head_dim=self.kernel_dim, scale=s.scale,
             window=s.window, k_pages=cache.k, v_pages=cache.v, block_tables=tables,
             page_tokens=cache.page_tokens, step=step, plan=step.plans[self.plan_key()],
-            head_scale=self.temperature, slopes=self.slopes, chunk=s.chunk, sinks=self.sinks)
+            head_scale=self.temperature, slopes=self.slopes, chunk=s.chunk, sinks=self.sinks, **self._cap)
         if s.gate == "head":  # one gate column per head, behind q, k (and v)
             gate0 = col0 + self.q_size + self.kv_size + self.v_size
             ops.sigmoid_gate_mul(o, qkv, gate0, self.kernel_dim)

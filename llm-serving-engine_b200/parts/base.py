@@ -260,12 +260,20 @@ class Mixer(Part):
     def forward(self, h, step, cache):  # pragma: no cover - interface
         raise NotImplementedError
 
+    def forward_into(self, h, step, cache, x, coefficient) -> list:
+        """``x += coefficient * forward(h)``, as far as the kernels can add on the way: returns what
+        is still to be added, a list of ``(factor, result)`` for a :class:`PendingAdds`."""
+        return [(coefficient, self.forward(h, step, cache))]
+
 
 class FeedForward(Part):
-    """``forward(h, step) -> [T, H]``: works on each token alone."""
+    """``forward(h, step) -> [T, H]``: works on each token alone. ``forward_into``: see :class:`Mixer`."""
 
     def forward(self, h, step):  # pragma: no cover - interface
         raise NotImplementedError
+
+    def forward_into(self, h, step, x, coefficient) -> list:
+        return [(coefficient, self.forward(h, step))]
 
 
 class Block(Part):
@@ -319,6 +327,45 @@ def project_into(ops, a, w, bias, out_dtype, residual, may_defer: bool = False):
     if may_defer and getattr(ops, "defers_adds", False):
         return ops.linear(a, w, bias, out_dtype=out_dtype, accumulate_into=residual, may_defer=True)
     return ops.linear(a, w, bias, out_dtype=out_dtype, accumulate_into=residual)
+
+
+def add_projected(ops, a, w, bias, x, coefficient) -> list:
+    """``x += coefficient * (a @ w.T (+ bias))`` (``x`` the float32 stream): the library adds the product of
+    many rows at once; otherwise what is returned, ``[(coefficient, product)]``, is still to be added."""
+    y = ops.linear(a, w, bias, out_dtype=torch.float32, accumulate_into=x, coefficient=coefficient, may_defer=True)
+    return [] if y is None else [(coefficient, y)]
+
+
+class PendingAdds:
+    """``x += sum_i c_i y_i (+ row)``, still to be done: what several sublayers that read the same norm
+    leave for the norm that reads ``x`` next. ``items``: pairs ``(c_i, y_i)``, ``y_i`` a float32 tensor or a
+    product of the kernel set that has not been taken yet; ``row``: a vector that is added to every
+    token. Exactly one of :meth:`take` (by that norm) and :meth:`resolve` (added now) happens before
+    anything else reads ``x``."""
+
+    __slots__ = ("ops", "x", "items", "row")
+
+    def __init__(self, ops, x, items, row=None) -> None:
+        self.ops, self.x, self.items, self.row = ops, x, list(items), row
+
+    def take(self):
+        items, row, self.items, self.row = self.items, self.row, [], None
+        return items, row
+
+    def resolve(self) -> None:
+        if self.items or self.row is not None:
+            self.ops.sum_add(self.x, *self.take())
+        return None
+
+
+def with_row(ops, x, pending, row) -> PendingAdds:
+    """``pending`` and, after it, a vector added to every token's row of ``x``."""
+    if not isinstance(pending, PendingAdds) or pending.row is not None:
+        if hasattr(pending, "resolve"):
+            pending = pending.resolve()
+        pending = PendingAdds(ops, x, [] if pending is None else [(1.0, pending)])
+    pending.row = row
+    return pending
 
 
 class PendingNormedBranch:

@@ -18,6 +18,12 @@ that reads ``x`` next, so a block returns its feed-forward output as ``pending``
 
 (the second half is optional).
 
+``shared_norm``: one norm, whose rows both sublayers read, and a constant on their sum:
+
+    h = norm(x);   x <- x + coefficient * (mixer(h) + feed_forward(h))
+
+(the feed-forward is optional). What is not added on the way is left for the norm that reads ``x`` next.
+
 ``filter`` is an optional input filter of the mixer (a token shift, say); the feed-forward is
 optional too. A filter that keeps something per request shares the block's cache layer with the
 mixer: the mixer's needs come first, the filter's states after them.
@@ -28,8 +34,8 @@ from __future__ import annotations
 from dataclasses import dataclass
 from typing import Any
 
-from .base import (BLOCKS, FEED_FORWARDS, INPUT_FILTERS, MIXERS, NORMS, Block, PendingNormedBranch, count_states,
-                   flatten_needs, has_pages, settle)
+from .base import (BLOCKS, FEED_FORWARDS, INPUT_FILTERS, MIXERS, NORMS, Block, PendingAdds, PendingNormedBranch,
+                   count_states, flatten_needs, has_pages, settle)
 
 
 @dataclass(frozen=True)
@@ -175,3 +181,31 @@ class SandwichBlock(Block):
         else:
             f = self.feed_forward.forward(h, step)
         return x, PendingNormedBranch(self.norm_ff_out, x, f)
+
+
+@dataclass(frozen=True)
+class SharedNormBlockSpec:
+    norm: Any
+    mixer: Any
+    feed_forward: Any = None
+    coefficient: float = 1.0
+    kind: str = "shared_norm"
+
+
+@BLOCKS.register("shared_norm")
+class SharedNormBlock(Block):
+    def __init__(self, spec: SharedNormBlockSpec, env) -> None:
+        super().__init__(spec, env)
+        self.children = {"norm": NORMS.build(spec.norm, env), "mixer": MIXERS.build(spec.mixer, env)}
+        if spec.feed_forward is not None:
+            self.children["feed_forward"] = FEED_FORWARDS.build(spec.feed_forward, env)
+        self.norm = self.children["norm"]
+        self.mixer = self.children["mixer"]
+        self.feed_forward = self.children.get("feed_forward")
+
+    def forward(self, x, pending, step, cache):
+        h = self.norm.forward(x, settle(pending, self.norm))
+        items = self.mixer.forward_into(h, step, cache, x, self.spec.coefficient)
+        if self.feed_forward is not None:
+            items += self.feed_forward.forward_into(h, step, x, self.spec.coefficient)
+        return x, PendingAdds(self.ops, x, items) if items else None

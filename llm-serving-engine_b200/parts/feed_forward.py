@@ -19,7 +19,7 @@ from __future__ import annotations
 
 from dataclasses import dataclass
 
-from .base import FEED_FORWARDS, FeedForward, ParamDecl, project_into
+from .base import FEED_FORWARDS, FeedForward, ParamDecl, add_projected, project_into
 
 
 GATED_ACTIVATIONS = ("silu", "gelu_tanh", "clamped_glu")
@@ -55,14 +55,17 @@ class SwiGLU(FeedForward):
 
     accepts_residual = True
 
-    def forward(self, h, step, residual=None, may_defer=False):
-        ops = self.ops
+    def forward_into(self, h, step, x, coefficient):
+        return add_projected(self.ops, self._inner(h), self.down_weight, None, x, coefficient)
+
+    def _inner(self, h):
         if self.spec.activation == "silu":
-            a = ops.gated_silu(h, self.gate_up_weight, None, out_dtype=self.env.dtype)
-        else:
-            a = ops.gated_silu(h, self.gate_up_weight, None, out_dtype=self.env.dtype,
-                               activation=self.spec.activation, **self._options)
-        return project_into(ops, a, self.down_weight, None, self.env.residual_dtype, residual, may_defer)
+            return self.ops.gated_silu(h, self.gate_up_weight, None, out_dtype=self.env.dtype)
+        return self.ops.gated_silu(h, self.gate_up_weight, None, out_dtype=self.env.dtype,
+                                   activation=self.spec.activation, **self._options)
+
+    def forward(self, h, step, residual=None, may_defer=False):
+        return project_into(self.ops, self._inner(h), self.down_weight, None, self.env.residual_dtype, residual, may_defer)
 
 
 PLAIN_ACTIVATIONS = ("relu2", "relu", "gelu_tanh", "silu")
@@ -101,9 +104,13 @@ class MLP(FeedForward):
         self.down_weight = params["down.weight"]
         self.coefficients = params.get("coefficients")
 
-    def forward(self, h, step, residual=None, may_defer=False):
+    def forward_into(self, h, step, x, coefficient):
+        return add_projected(self.ops, self._inner(h), self.down_weight, None, x, coefficient)
+
+    def _inner(self, h):
         if self.spec.activation == "poly_norm":
-            a = self.ops.poly_norm_linear(h, self.up_weight, self.coefficients, self.spec.eps, self.env.dtype)
-        else:
-            a = self.ops.activated_linear(h, self.up_weight, self.spec.activation, self.env.dtype)
-        return project_into(self.ops, a, self.down_weight, None, self.env.residual_dtype, residual, may_defer)
+            return self.ops.poly_norm_linear(h, self.up_weight, self.coefficients, self.spec.eps, self.env.dtype)
+        return self.ops.activated_linear(h, self.up_weight, self.spec.activation, self.env.dtype)
+
+    def forward(self, h, step, residual=None, may_defer=False):
+        return project_into(self.ops, self._inner(h), self.down_weight, None, self.env.residual_dtype, residual, may_defer)

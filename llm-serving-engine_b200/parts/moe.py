@@ -21,7 +21,7 @@ Options of the spec:
   ``correction`` a learned number per expert is added to the scores for the choice alone; the
   experts form ``groups`` equal groups of neighbours, of which only the ``keep_groups`` with the
   largest choice scores in them can be chosen from; the weights are the chosen experts' scores
-  divided by their sum (+ 1e-20) and multiplied by ``router_scale``;
+  divided by their sum (+ 1e-20; not with ``normalise_weights=False``) and multiplied by ``router_scale``;
 * ``identity_experts``: the last rows of the router stand for experts whose output is their input;
   they have no matrices and take part in the softmax, the groups and the choice like the others;
 * ``activation="clamped_glu"`` with ``limit`` (``shared_limit``: the shared expert's).
@@ -56,6 +56,7 @@ class RoutedExpertsSpec:
     groups: int = 1
     keep_groups: int = 1
     router_scale: float = 1.0
+    normalise_weights: bool = True  # softmax_of_all: divided by the sum of the chosen
     identity_experts: int = 0
     limit: float = 0.0
     shared_limit: float = 0.0
@@ -72,8 +73,10 @@ class RoutedExperts(FeedForward):
         if not 1 <= spec.top <= self.choices:
             raise ValueError("routed_experts: top must lie between 1 and the number of experts")
         self.of_all = spec.router_weights == "softmax_of_all"
-        if (spec.correction or spec.groups != 1 or spec.router_scale != 1.0 or spec.identity_experts) and not self.of_all:
-            raise ValueError("routed_experts: correction, groups, scale and identity experts go with softmax_of_all")
+        if (spec.correction or spec.groups != 1 or spec.router_scale != 1.0 or spec.identity_experts
+                or not spec.normalise_weights) and not self.of_all:
+            raise ValueError("routed_experts: correction, groups, scale, weights as they are and identity experts go "
+                             "with softmax_of_all")
         if self.of_all and (spec.router_bias or spec.weight_on != "output" or self.choices % spec.groups
                             or not 1 <= spec.keep_groups <= spec.groups
                             or spec.top > spec.keep_groups * (self.choices // spec.groups)):
@@ -126,12 +129,17 @@ class RoutedExperts(FeedForward):
         if self.shared is not None:
             self.shared.bind({k[len("shared."):]: v for k, v in params.items() if k.startswith("shared.")})
 
-    def forward(self, h, step, residual=None, may_defer=False):
+    def forward_into(self, h, step, x, coefficient):
+        y = self.forward(h, step, residual=x, scale=coefficient)
+        return [] if y is None else [(1.0, y)]  # the sum over the experts is scaled as it is formed
+
+    def forward(self, h, step, residual=None, may_defer=False, scale=1.0):
         s, ops = self.spec, self.ops
         if self.of_all:
             idx, wts, gate = ops.moe_route(h, self.router_weight, self.choices, s.top, self.has_gate,
                                            bias=self.correction, weights=s.router_weights, groups=s.groups,
-                                           keep=s.keep_groups, scale=s.router_scale)
+                                           keep=s.keep_groups, scale=s.router_scale,
+                                           **({} if s.normalise_weights else {"normalise": False}))
         elif s.router_bias or s.router_weights != "sigmoid":
             idx, wts, gate = ops.moe_route(h, self.router_weight, s.num_experts, s.top, self.has_gate,
                                            bias=self.router_bias, weights=s.router_weights)
@@ -148,11 +156,12 @@ class RoutedExperts(FeedForward):
         shared = self.shared.forward(h, step) if self.shared is not None else None
         if hasattr(shared, "resolve"):
             shared = shared.resolve()
+        scaled = {} if scale == 1.0 else {"scale": scale}
         if on_input and self.has_gate == (shared is not None):
-            return ops.moe_combine(y, plan, s.top, shared, gate, residual)
+            return ops.moe_combine(y, plan, s.top, shared, gate, residual, **scaled)
         if s.identity_experts:
-            return ops.moe_combine(y, plan, s.top, shared, gate, residual, wts=wts, identity=h)
-        return ops.moe_combine(y, plan, s.top, shared, gate, residual, wts=None if on_input else wts)
+            return ops.moe_combine(y, plan, s.top, shared, gate, residual, wts=wts, identity=h, **scaled)
+        return ops.moe_combine(y, plan, s.top, shared, gate, residual, wts=None if on_input else wts, **scaled)
 
 
 def _gcd8(*sizes: int) -> int:

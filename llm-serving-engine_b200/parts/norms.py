@@ -15,7 +15,7 @@ from __future__ import annotations
 
 from dataclasses import dataclass
 
-from .base import NORMS, BranchMix, Norm, ParamDecl, PendingNormedBranch
+from .base import NORMS, BranchMix, Norm, ParamDecl, PendingAdds, PendingNormedBranch
 
 
 @dataclass(frozen=True)
@@ -49,6 +49,10 @@ class RMSNorm(Norm):
             if rows is None:  # the branch's norm, the sum and this norm while the rows are held once
                 return residual.norm.add_normed_then(x, residual.take(), self)
             residual = residual.resolve()  # only some rows are read here: the whole sum is formed first
+        if isinstance(residual, PendingAdds):
+            if rows is None and not self._groups:  # the sums and this norm in one launch
+                return self.ops.sum_add_rmsnorm(x, *residual.take(), self.weight, self.spec.eps, out_dtype=self.env.dtype)
+            residual = residual.resolve()
         if isinstance(residual, BranchMix):
             if rows is None:  # the branches' norms, their sum into x and this norm in one launch
                 return self.ops.mix_add_rmsnorm(x, residual, self.weight, self.spec.eps, out_dtype=self.env.dtype,

@@ -3,6 +3,8 @@ and summed with fixed coefficients.
 
     out = sum_b coefficient_b * w_b * a_b / sqrt(mean(a_b^2) + eps),      a_b = branch_b(h)
 
+``normed=False``: the branches' outputs are summed as they are, ``sum_b coefficient_b * a_b``.
+
 Branches that can start from a product made for them (``input_weight``, ``forward_projected``) share
 one: their matrices are laid one below the other when the weights are bound.
 
@@ -17,7 +19,7 @@ from typing import Any
 
 import torch
 
-from .base import MIXERS, BranchMix, Mixer, ParamDecl, count_states, flatten_needs, has_pages
+from .base import MIXERS, BranchMix, Mixer, ParamDecl, PendingAdds, count_states, flatten_needs, has_pages
 
 
 @dataclass(frozen=True)
@@ -26,7 +28,8 @@ class ParallelMixerSpec:
     names: tuple[str, ...]
     branches: tuple[Any, ...]  # mixer specs
     coefficients: tuple[float, ...]
-    eps: float
+    eps: float = 0.0
+    normed: bool = True
     kind: str = "parallel"
 
 
@@ -51,7 +54,8 @@ class ParallelMixer(Mixer):
         for name, child in self.children.items():
             for pname, decl in child.param_decls().items():
                 out[f"{name}.{pname}"] = decl
-            out[f"out.{name}.weight"] = ParamDecl((self.spec.hidden_size,), "scale")
+            if self.spec.normed:
+                out[f"out.{name}.weight"] = ParamDecl((self.spec.hidden_size,), "scale")
         return out
 
     def bind(self, params):
@@ -59,7 +63,8 @@ class ParallelMixer(Mixer):
         for name, child in self.children.items():
             prefix = name + "."
             child.bind({k[len(prefix):]: v for k, v in params.items() if k.startswith(prefix)})
-            self.out_weights.append(params[f"out.{name}.weight"])
+            if self.spec.normed:
+                self.out_weights.append(params[f"out.{name}.weight"])
         self._share_product()
 
     def _share_product(self):
@@ -85,7 +90,24 @@ class ParallelMixer(Mixer):
 
     accepts_deferral = True
 
+    def forward_into(self, h, step, cache, x, coefficient):
+        if self.spec.normed:
+            return [(coefficient, self.forward(h, step, cache).resolve())]
+        items = []
+        proj = None if self.shared_weight is None else self.ops.linear(h, self.shared_weight, None, out_dtype=torch.float32)
+        for k, (b, c, (pages, first, n)) in enumerate(zip(self.branches, self.spec.coefficients, self._parts)):
+            part = cache.part(pages, first, n)
+            if proj is None:
+                items += b.forward_into(h, step, part, x, coefficient * c)
+            else:
+                items += b.forward_projected(proj, self.columns[k], step, part, add_to=(x, coefficient * c))
+        return items
+
     def forward(self, h, step, cache, may_defer=False):
+        if not self.spec.normed:
+            x = torch.zeros(h.shape[0], self.spec.hidden_size, dtype=torch.float32, device=h.device)
+            PendingAdds(self.ops, x, self.forward_into(h, step, cache, x, 1.0)).resolve()
+            return x
         outs = []
         if self.shared_weight is not None:
             proj = self.ops.linear(h, self.shared_weight, None, out_dtype=torch.float32)

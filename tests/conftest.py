@@ -617,3 +617,137 @@ def write_miberax(folder, name):
 @pytest.fixture(scope="session")
 def miberax_dirs(tmp_path_factory):
     return {name: write_miberax(tmp_path_factory.mktemp(f"miberax-{name}"), name) for name in MIBERAX_TINY}
+
+
+# ----------------------------------------------------------------------------- Tanupel
+def _tatt(heads, kv, dim, vdim, scale, rot=None, softcap=None):
+    """rot: (base, dims) and, for scaled frequencies, (factor,) or (factor, low, high, original)."""
+    m = {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": vdim, "scale": scale}
+    if rot:
+        m["rot"] = {"base": rot[0], "dims": rot[1]}
+        if len(rot) > 2:
+            m["rot"]["scaling"] = dict(zip(("factor", "low", "high", "original"), rot[2]))
+    if softcap:
+        m["softcap"] = softcap
+    return m
+
+
+def _tdelta(heads, kv, dim, vdim, conv, ranks):
+    return {"heads": heads, "kv_heads": kv, "dim": dim, "vdim": vdim, "conv": conv, "decay_rank": ranks[0], "gate_rank": ranks[1]}
+
+
+def _tlayer(left, mlp, right=None, scales=None):
+    if right is None:
+        return {"type": "attention", "mixer": left, "mlp": mlp}
+    return {"type": "parallel", "mlp": mlp,
+            "mixer": {"left": left, "left_scale": scales[0], "right": right, "right_scale": scales[1]}}
+
+
+def _tmoe(experts, top, ff):
+    return {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": ff}}
+
+
+TANUPEL_TINY = {
+    # a loop over two layers in the middle, one of each kind; values wider and narrower than keys; grouped heads
+    # on both sides; both kinds of frequency scaling; soft caps; a layer without feed-forward
+    "T1": dict(seed=6, page_tokens=16, config={
+        "architecture": "Tanupel", "vocab": 167, "width": 96, "norm": {"eps": 1e-5}, "embedding": {"scale": 3.5},
+        "residual_mult": 0.7, "loop": {"start": 1, "stop": 3, "times": 2},
+        "layers": [_tlayer(_tatt(4, 2, 24, 40, 0.3, (10000.0, 8, (8.0, 1.0, 4.0, 64)), softcap=4.0), _dense(112)),
+                   _tlayer(_tatt(3, 1, 32, 16, 0.25, (500.0, 32, (3.0,)), softcap=6.0), _tmoe(5, 2, 24),
+                           _tdelta(4, 2, 32, 16, 4, (8, 24)), (0.8, 1.4)),
+                   _tlayer(_tatt(2, 2, 16, 16, 0.35, (50.0, 12)), None),
+                   _tlayer(_tatt(4, 4, 16, 24, 0.3, (300.0, 4, (2.0,))), _dense(64),
+                           _tdelta(2, 1, 16, 40, 2, (16, 8)), (1.3, 0.6))]}),
+    # sizes that are multiples of nothing; a convolution of one tap and one of five; ranks unlike each other; no
+    # rotation; every expert chosen; one layer that runs three times, the last; pages of 8 tokens
+    "T2": dict(seed=13, page_tokens=8, config={
+        "architecture": "Tanupel", "vocab": 131, "width": 70, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+        "residual_mult": 1.0, "loop": {"start": 2, "stop": 3, "times": 3},
+        "layers": [_tlayer(_tatt(3, 3, 18, 10, 0.3, (300.0, 6, (3.0,)), softcap=2.5), _tmoe(4, 4, 10),
+                           _tdelta(5, 1, 10, 14, 1, (5, 11)), (1.0, 1.0)),
+                   _tlayer(_tatt(2, 1, 20, 12, 0.3), _dense(50)),
+                   _tlayer(_tatt(5, 1, 12, 12, 0.4, (1000.0, 12, (4.0, 1.0, 2.0, 40))), _tmoe(3, 1, 14),
+                           _tdelta(3, 1, 7, 20, 5, (3, 2)), (0.4, 2.0))]}),
+    # the head sizes of larger models (tensor-core attention with and without a cap); a wide key of the delta
+    # rule; many experts; no loop; a fully rotated head
+    "T3": dict(seed=22, page_tokens=32, config={
+        "architecture": "Tanupel", "vocab": 300, "width": 128, "norm": {"eps": 1e-5}, "embedding": {"scale": 11.0},
+        "residual_mult": 0.35,
+        "layers": [_tlayer(_tatt(8, 2, 64, 64, 0.125, (20000.0, 64, (4.0, 1.0, 4.0, 128)), softcap=10.0), _dense(192),
+                           _tdelta(2, 2, 128, 64, 4, (32, 32)), (1.2, 0.5)),
+                   _tlayer(_tatt(4, 1, 64, 64, 0.2, (10000.0, 16)), _tmoe(14, 3, 48)),
+                   _tlayer(_tatt(4, 2, 128, 128, 0.1, (700.0, 32, (2.0,)), softcap=8.0), _dense(80),
+                           _tdelta(1, 1, 160, 32, 2, (8, 40)), (0.7, 1.1))]}),
+}
+
+
+def write_tanupel(folder, name):
+    """A random folder whose attention is sharp, whose decays, step sizes and convolutions differ clearly from head
+    to head and channel to channel, and whose norms and vectors are drawn wide, so that leaving one of them out, a
+    key too many or a lost state changes the logits clearly.
+
+    No routing decision is a close call (a model computed in bfloat16 must pick the same experts as the float64
+    one): the last dims of the residual stream carry, for every token, one of evenly spaced levels per expert, in
+    an order that depends on the token; no layer and no vector of a pass writes those dims, and each router row
+    reads its expert's dim beside small random weights on all the others."""
+    from safetensors.torch import load_file, save_file
+
+    from llmserve_b200.config.tanupel import TanupelConfig
+    from llmserve_b200.weights import write_random_model
+
+    spec = TANUPEL_TINY[name]
+    cfg = spec["config"]
+    write_random_model(folder, TanupelConfig.from_dict(cfg), spec["seed"])
+    f = folder / "model.safetensors"
+    t = load_file(str(f))
+    g = torch.Generator().manual_seed(spec["seed"] + 1)
+    for k, v in t.items():
+        r = torch.rand(v.shape, generator=g)
+        if k.endswith("A_log"):
+            t[k] = (2.5 * r - 2.0).to(v.dtype)
+        elif k.endswith("dt_bias"):
+            t[k] = (6 * r - 5.0).to(v.dtype)  # from channels that keep nearly all to some that forget in a few tokens
+        elif k.endswith(".conv"):
+            t[k] = (1.6 * r - 0.5).to(v.dtype)
+        elif k.endswith(("q.norm", "k.norm")):
+            t[k] = (1.6 * (0.5 + r)).to(v.dtype)
+        elif k.endswith("norm1") or k == "final.norm":
+            t[k] = (r - 0.5).to(v.dtype)  # stored around zero
+        elif k == "loop.step":
+            t[k] = (3 * (r - 0.5)).to(v.dtype)
+        elif v.dim() == 1:  # the delta rule's norm weight (and the correction, set below)
+            t[k] = (0.5 + r).to(v.dtype)
+        elif k == "embed":
+            t[k] = (v.float() * 40 / cfg["embedding"]["scale"]).to(v.dtype)
+        elif k.endswith(("right.a1", "right.a2", "right.b", "right.g1", "right.g2")):
+            t[k] = (v.float() * 15).to(v.dtype)
+        else:
+            t[k] = (v.float() * 8).to(v.dtype)
+    width = cfg["width"]
+    moe = [(i, l["mlp"]["router"]["experts"]) for i, l in enumerate(cfg["layers"]) if l["mlp"] and l["mlp"]["kind"] == "moe"]
+    most = max(n for _, n in moe)
+    step = next(m for m in (3, 5, 7, 11) if all(most % q or m % q for q in (2, 3, 5, 7, 11)))
+    dims = [width - most + e for e in range(most)]
+    tok = torch.arange(cfg["vocab"])[:, None]
+    levels = 1.5 * (((tok * 7 + step * torch.arange(most)[None, :]) % most).float() - (most - 1) / 2)
+    t["embed"][:, dims] = (levels / cfg["embedding"]["scale"]).to(t["embed"].dtype)
+    for k in t:
+        if k.endswith(("down", "mix.o", "left.o", "right.o")):
+            t[k][dims, :] = 0
+        elif k == "loop.step":
+            t[k][:, dims] = 0
+    for i, n in moe:
+        t[f"l{i}.norm1"][dims] = 0
+        router = torch.randn(n, width, generator=g) * 0.002
+        router[torch.arange(n), dims[:n]] = 0.8
+        t[f"l{i}.mlp.router"] = router.to(torch.bfloat16)
+        # a correction that moves a choice here and there: below the gap between two scores where it counts
+        t[f"l{i}.mlp.correction"] = (0.01 * (torch.rand(n, generator=g) - 0.5)).to(torch.bfloat16)
+    save_file(t, str(f))
+    return folder
+
+
+@pytest.fixture(scope="session")
+def tanupel_dirs(tmp_path_factory):
+    return {name: write_tanupel(tmp_path_factory.mktemp(f"tanupel-{name}"), name) for name in TANUPEL_TINY}

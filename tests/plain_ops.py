@@ -46,8 +46,18 @@ class PlainOps:
             raise ValueError("head size must be a multiple of 16")
 
     # ------------------------------------------------------------------ pointwise
-    def embedding(self, token_ids, table):
-        return table[token_ids.long()].float()
+    def embedding(self, token_ids, table, scale=1.0):
+        return table[token_ids.long()].float() * scale
+
+    def sum_add_rmsnorm(self, x, items, row, weight, eps, out_dtype):
+        for c, y in items:
+            x += c * y.float()
+        if row is not None:
+            x += row
+        return None if weight is None else self.add_rmsnorm(x, None, weight, eps, out_dtype)
+
+    def sum_add(self, x, items, row):
+        self.sum_add_rmsnorm(x, items, row, None, 0.0, None)
 
     def add_rmsnorm(self, x, residual, weight, eps, out_dtype, rows=None, groups=1):
         if rows is not None:
@@ -81,12 +91,12 @@ class PlainOps:
             act = g / (1 + torch.exp(-g))
         return (act * u).to(out_dtype or gu.dtype)
 
-    def linear(self, a, w, bias=None, out_dtype=None, accumulate_into=None):
+    def linear(self, a, w, bias=None, out_dtype=None, accumulate_into=None, may_defer=False, coefficient=None):
         y = a.float() @ w.float().T
         if bias is not None:
             y = y + bias.float()
         if accumulate_into is not None and self.accumulate:
-            accumulate_into += y
+            accumulate_into += y * (1.0 if coefficient is None else coefficient)
             return None
         return y.to(out_dtype or a.dtype)
 
@@ -149,7 +159,7 @@ class PlainOps:
 
     def paged_attention(self, q, *, num_heads, num_kv_heads, head_dim, scale, window, k_pages,
                         v_pages, block_tables, page_tokens, step, plan=None, head_scale=None,
-                        slopes=None, chunk=0, sinks=None, keep_first=0, out_dtype=None):
+                        slopes=None, chunk=0, sinks=None, keep_first=0, out_dtype=None, softcap=0.0):
         T, D = q.shape[0], head_dim
         qkv = q
         q = q[:, : num_heads * D].float().reshape(T, num_heads, D)
@@ -173,6 +183,8 @@ class PlainOps:
             sc = torch.einsum("thd,shd->hts", q[a:b], k) * scale
             if head_scale is not None:
                 sc = sc * head_scale.float()[:, None, None]
+            if softcap > 0:
+                sc = softcap * torch.tanh(sc / softcap)
             if slopes is not None:
                 sc = sc - slopes.float()[:, None, None] * (qpos - j[None, :]).float()[None]
             sc = sc.masked_fill(~visible, float("-inf"))
@@ -305,7 +317,7 @@ class PlainOps:
 
     # ------------------------------------------------------------------ routed experts
     def moe_route(self, h, router, num_experts, top, has_gate, bias=None, weights="sigmoid", groups=1, keep=1,
-                  scale=1.0):
+                  scale=1.0, normalise=True):
         z = h.float() @ router.float().T
         gate = torch.sigmoid(z[:, num_experts]) if has_gate else None
         if weights == "softmax_of_all":
@@ -317,7 +329,9 @@ class PlainOps:
             c = per.masked_fill(~kept[:, :, None], float("-inf")).view(-1, num_experts)
             idx = torch.topk(c, top, dim=-1).indices
             val = s.gather(1, idx)
-            return idx.to(torch.int32), val / (val.sum(-1, keepdim=True) + 1e-20) * scale, gate
+            if normalise:
+                val = val / (val.sum(-1, keepdim=True) + 1e-20)
+            return idx.to(torch.int32), val * scale, gate
         z = z[:, :num_experts] + (bias.float() if bias is not None else 0.0)
         val, idx = torch.topk(z, top, dim=-1)
         val = torch.sigmoid(val) if weights == "sigmoid" else torch.softmax(val, dim=-1)
@@ -334,13 +348,14 @@ class PlainOps:
             rows = rows * wts.reshape(-1, 1)
         return torch.einsum("rk,rnk->rn", rows, w.float()[idx])
 
-    def moe_combine(self, y, plan, top, shared, gate, residual, wts=None, identity=None):
+    def moe_combine(self, y, plan, top, shared, gate, residual, wts=None, identity=None, scale=1.0):
         rows = y.view(-1, top, y.shape[1])
         if identity is not None:
             rows = torch.where((plan >= self.num_real_experts)[:, :, None], identity.float()[:, None, :], rows)
         out = (rows * wts[:, :, None]).sum(1) if wts is not None else rows.sum(1)
         if shared is not None:
             out = out + (gate[:, None] * shared.float() if gate is not None else shared.float())
+        out = out * scale
         if residual is not None and self.accumulate:
             residual += out
             return None
@@ -411,8 +426,11 @@ class PlainOps:
             state[slots[s_]] = S
         return out.reshape(T, H * dv)
 
+    def inner_linear(self, proj, col0, w, dtype):
+        return self.head_linear(proj, col0, w, torch.float32)
+
     def delta_inputs(self, proj, col0, *, num_heads, num_kv_heads, key_dim, value_dim, conv, conv_state, A_log,
-                     dt_bias, query_scale, step):
+                     dt_bias, query_scale, step, decay_logits=None):
         H, G, dk, dv, C = num_heads, num_kv_heads, key_dim, value_dim, conv.shape[1]
         past = conv.shape[0] - 1
         cu, ctx, slots = step.cu_q.tolist(), step.ctx_lens.tolist(), step.state_slots.tolist()
@@ -434,14 +452,20 @@ class PlainOps:
         unit = lambda t: t / torch.sqrt(t.pow(2).sum(-1, keepdim=True) + 1e-6)
         q = unit(y[:, : G * dk].view(T, G, dk)) * query_scale
         k = unit(y[:, G * dk : 2 * G * dk].view(T, G, dk))
-        b0 = col0 + C + H * dv
-        g = torch.exp(-torch.exp(A_log) * torch.nn.functional.softplus(proj[:, b0 + H : b0 + 2 * H].float() + dt_bias))
+        b0, decay = col0 + C + (H * dv if decay_logits is None else 0), None
+        if decay_logits is None:
+            g = torch.exp(-torch.exp(A_log) * torch.nn.functional.softplus(proj[:, b0 + H : b0 + 2 * H].float() + dt_bias))
+        else:
+            g = torch.ones(T, H)
+            step_ = torch.nn.functional.softplus(decay_logits[:, : H * dk].float() + dt_bias)
+            decay = torch.exp(-torch.exp(A_log).repeat_interleave(dk) * step_)
         beta = torch.sigmoid(proj[:, b0 : b0 + H].float())
         qk = (q * k).sum(-1).repeat_interleave(H // G, 1)
-        return (torch.cat([q.reshape(T, -1), k.reshape(T, -1), y[:, 2 * G * dk :]], 1),
-                torch.stack([g, beta, qk, torch.zeros_like(g)], -1))
+        out = (torch.cat([q.reshape(T, -1), k.reshape(T, -1), y[:, 2 * G * dk :]], 1),
+               torch.stack([g, beta, qk, torch.zeros_like(g)], -1))
+        return out if decay is None else (*out, decay)
 
-    def delta_rule(self, qkv, scal, *, num_heads, num_kv_heads, key_dim, value_dim, state, step):
+    def delta_rule(self, qkv, scal, *, num_heads, num_kv_heads, key_dim, value_dim, state, step, decay=None):
         T, H, G, dk, dv = qkv.shape[0], num_heads, num_kv_heads, key_dim, value_dim
         q = qkv[:, : G * dk].view(T, G, dk).repeat_interleave(H // G, 1)
         k = qkv[:, G * dk : 2 * G * dk].view(T, G, dk).repeat_interleave(H // G, 1)
@@ -452,7 +476,7 @@ class PlainOps:
             a, b = cu[s_], cu[s_ + 1]
             S = state[slots[s_]].clone() if ctx[s_] - (b - a) > 0 else torch.zeros_like(state[0])  # [H, dv, dk]
             for t in range(a, b):
-                S = scal[t, :, 0, None, None] * S
+                S = (scal[t, :, 0, None, None] if decay is None else decay[t].view(H, 1, dk)) * S
                 u = scal[t, :, 1, None] * (v[t] - torch.einsum("hvk,hk->hv", S, k[t]))
                 S = S + u[:, :, None] * k[t][:, None, :]
                 out[t] = torch.einsum("hvk,hk->hv", S, q[t])
