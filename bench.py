@@ -19,8 +19,9 @@ and a float32 replay of one 8192-token sequence against the plain implementation
 reference's own harness (src/llmserve/bench/run.py:96,124-176): fixed output lengths, greedy, a
 warm-up run that is thrown away, one JSON line with the environment.
 
-``--workload designs`` (``--arms llama,gubotar,pazivik,rirovik,lanilorn,miberax``) puts four Miberax layers (chunked
-attention beside the gated delta rule in every layer; dense and grouped routed feed-forwards), four Lanilorn layers (four
+``--workload designs`` (``--arms llama,gubotar,pazivik,rirovik,lanilorn,miberax,tanupel``) puts four Tanupel layers
+(soft-capped attention beside the gated delta rule with decays per channel, both sublayers on one norm; dense and
+routed feed-forwards), four Miberax layers (chunked attention beside the gated delta rule in every layer; dense and grouped routed feed-forwards), four Lanilorn layers (four
 residual streams; linear attention with a decay per channel and token, windowed attention with sinks and
 a norm over whole rows, differential attention; ungated dense feed-forwards), four Pazivik layers (latent attention
 with a window; dense and routed feed-forwards), four Gubotar layers (parallel, retention, retention, parallel) and
@@ -683,6 +684,26 @@ def miberax_layers(width, heads, kv_heads, head_dim, ff, chunk=512, state_dim=12
     return [layer(dense), layer(moe), layer(dense), layer(moe)]
 
 
+def tanupel_layers(width, heads, kv_heads, head_dim, ff, state_dim=128, rank=128, experts=8, top=2):
+    """Four Tanupel layers at a Llama layer's sizes: the Llama layer's heads, half of each rotated, with a soft cap on
+    the scores and no window, beside the gated delta rule with decays per channel on heads of ``state_dim`` x
+    ``state_dim`` (as the Miberax arm's); a dense feed-forward of the Llama layer's size in layers 0 and 2; in
+    layers 1 and 3 ``experts`` gated experts of a quarter of that size, ``top`` per token."""
+    lin = max(1, width // state_dim)
+
+    def layer(mlp):
+        return {"type": "parallel", "mlp": mlp, "mixer": {
+            "left": {"heads": heads, "kv_heads": kv_heads, "dim": head_dim, "vdim": head_dim, "scale": head_dim ** -0.5,
+                     "softcap": 30.0, "rot": {"base": 500000.0, "dims": head_dim // 2, "scaling": {"factor": 4.0}}},
+            "left_scale": 0.7, "right_scale": 0.7,
+            "right": {"heads": lin, "kv_heads": lin, "dim": state_dim, "vdim": state_dim, "conv": 4, "decay_rank": rank,
+                      "gate_rank": rank}}}
+
+    dense = {"kind": "dense", "ff": ff}
+    moe = {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": ff // 4}}
+    return [layer(dense), layer(moe), layer(dense), layer(moe)]
+
+
 def kernel_profile(fn, reps=3) -> dict:
     """Device time of ``fn()`` by kernel, from the framework's profiler: microseconds per call."""
     import collections
@@ -730,6 +751,8 @@ def designs_main(args) -> int:
                                                    "layers": lanilorn_layers(w, heads, kv, hd, ff, state_dim=hd if w < 2048 else 128)}),
             "miberax": ("random:miberax-2048", {"width": w, "vocab": ll["vocab_size"],
                                                  "layers": miberax_layers(w, heads, kv, hd, ff, state_dim=hd if w < 2048 else 128)}),
+            "tanupel": ("random:tanupel-2048", {"width": w, "vocab": ll["vocab_size"], "loop": None,
+                                                 "layers": tanupel_layers(w, heads, kv, hd, ff, state_dim=hd if w < 2048 else 128)}),
         }
         arms = {k: v for k, v in arms.items() if k in args.arms.split(",")}
         row = {"sizes": f"{alias}: width {w}, ff {ff}, {heads} heads of {hd}, 4 layers"}
@@ -881,7 +904,7 @@ def main() -> int:
     ap.add_argument("--warmup", type=int, default=8)
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--workload", default="decode", choices=["decode", "continuous", "long", "designs"])
-    ap.add_argument("--arms", default="llama,gubotar,pazivik,rirovik,lanilorn,miberax",
+    ap.add_argument("--arms", default="llama,gubotar,pazivik,rirovik,lanilorn,miberax,tanupel",
                     help="--workload designs: which architectures run side by side")
     ap.add_argument("--model", default="smollm2-1.7b")
     ap.add_argument("--batch", type=int, default=8)

@@ -105,7 +105,8 @@ void sum_add_rmsnorm(Tensor& x, const std::vector<Tensor>& y, const std::vector<
   }
   const float *rp = nullptr, *wp = nullptr;
   if (row) {
-    check_f32(*row, "row");
+    // a row of a matrix of such vectors: it starts on a 16-byte boundary where the width is a multiple of 4
+    check_state(*row, "row", x.size(1));
     TORCH_CHECK(row->numel() == x.size(1), "sum_add_rmsnorm: row needs x's width");
     rp = row->data_ptr<float>();
   }
@@ -207,14 +208,18 @@ Tensor rope_kv_write(Tensor& qkv, int64_t nq, int64_t nk, int64_t D, const Tenso
   return q;
 }
 
-void silu_mul(const Tensor& gu, Tensor& out, int64_t act, double limit) {
+void silu_mul(const Tensor& gu, Tensor& out, int64_t act, double limit, int64_t col0) {
   check_cuda(gu, "gu");
   check_cuda(out, "out");
-  TORCH_CHECK(gu.dim() == 2 && out.dim() == 2 && gu.size(1) == 2 * out.size(1) &&
-                  gu.size(0) == out.size(0),
-              "silu_mul: gu must be [T, 2I] and out [T, I]");
-  done(lse_silu_mul(gu.data_ptr(), dtype_code(gu, "gu"), out.data_ptr(), dtype_code(out, "out"),
-                    (int)gu.size(0), (int)out.size(1), (int)act, stream(), (float)limit),
+  const int64_t I = out.size(1);
+  TORCH_CHECK(gu.dim() == 2 && out.dim() == 2 && gu.size(0) == out.size(0) && col0 >= 0 &&
+                  (col0 ? col0 + 2 * I <= gu.size(1) : gu.size(1) == 2 * I),
+              "silu_mul: gu must be [T, 2I] (or have 2I columns from a later one on) and out [T, I]");
+  const int code = dtype_code(gu, "gu");
+  TORCH_CHECK(col0 == 0 || code == LSE_F32, "silu_mul: columns of a wider matrix are float32");
+  const void* p = col0 ? static_cast<const void*>(gu.data_ptr<float>() + col0) : gu.data_ptr();
+  done(lse_silu_mul(p, code, out.data_ptr(), dtype_code(out, "out"), (int)gu.size(0), (int)I, (int)act, stream(),
+                    (float)limit, col0 ? (long long)gu.size(1) : 0),
        "silu_mul");
 }
 
@@ -1412,7 +1417,7 @@ PYBIND11_MODULE(TORCH_EXTENSION_NAME, m) {
         py::arg("out"), py::arg("rows"), py::arg("groups") = 1);
   m.def("rope_kv_write", &rope_kv_write);
   m.def("silu_mul", &silu_mul, py::arg("gu"), py::arg("out"), py::arg("act") = 0,
-        py::arg("limit") = 0.0);
+        py::arg("limit") = 0.0, py::arg("col0") = 0);
   m.def("poly_norm", &poly_norm);
   m.def("gemm_f32", &gemm_f32);
   m.def("gemm_bf16_skinny", &gemm_bf16_skinny);

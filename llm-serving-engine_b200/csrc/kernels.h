@@ -62,7 +62,9 @@ int lse_rope_kv_write(const void* qkv, int in_dtype, void* q_out, int dtype, int
 // or LSE_ACT_CLAMPED_GLU: g sigmoid(1.702 g) (u + 1), g = min(gate, limit), u = clamp(up, -limit, limit)
 #define LSE_ACT_CLAMPED_GLU 2
 int lse_silu_mul(const void* gu, int in_dtype, void* out, int dtype, int T, int I, int act,
-                 cudaStream_t stream, float limit = 0.f);
+                 cudaStream_t stream, float limit = 0.f,
+                 // columns of a wider float32 matrix: its row length (0: 2 I)
+                 long long stride = 0);
 
 // out[t] = coef[0] N(z[t]) + coef[1] N(z[t]^2) + coef[2] N(z[t]^3) + coef[3], powers element by element,
 // N(y) = y / sqrt(mean(y^2) + eps) over the row's N values. z float32, bfloat16 or LSE_FIXED64 (taken;

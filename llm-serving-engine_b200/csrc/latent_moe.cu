@@ -658,9 +658,10 @@ moe_gather_rows_kernel(const bf16* __restrict__ a, const int* __restrict__ perm,
 // null wts or gate counts as ones; a choice without a row, pos_of < 0, is an identity expert and adds
 // wts times the token's row of h), the sum times `scale`; a block per token and
 // slice of 512 columns, four columns per thread (the experts' rows are added in the order k = 0, 1, ...)
-constexpr int COMBINE_SLICE = 512;
+constexpr int COMBINE_SLICE = 512;  // four columns per thread
 
-template <typename TH>
+// V4 (W a multiple of 4): a thread's columns are neighbours, read and written as one vector
+template <typename TH, bool V4>
 __global__ void __launch_bounds__(128)
 moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ pos_of, int top,
                    const float* __restrict__ shared_out, const float* __restrict__ gate,
@@ -670,32 +671,57 @@ moe_combine_kernel(const float* __restrict__ y, const int* __restrict__ pos_of, 
   pdl_wait();  // everything below reads what kernels before this one wrote
   const int t = blockIdx.x;
   const float g = gate ? gate[t] : 1.f;
-  const int i0 = blockIdx.y * COMBINE_SLICE + threadIdx.x;
-  float v[COMBINE_SLICE / 128];
+  constexpr int C = COMBINE_SLICE / 128, STEP = V4 ? 1 : 128;  // a thread's columns: i0 + j * STEP
+  const int i0 = blockIdx.y * COMBINE_SLICE + threadIdx.x * (V4 ? C : 1);
+  float v[C];
 #pragma unroll
-  for (int j = 0; j < COMBINE_SLICE / 128; ++j) v[j] = 0.f;
+  for (int j = 0; j < C; ++j) v[j] = 0.f;
   for (int k = 0; k < top; ++k) {
     const int pos = pos_of[(size_t)t * top + k];
     const float wk = wts ? wts[(size_t)t * top + k] : 1.f;
     if (pos < 0) {
       if (!h) continue;
 #pragma unroll
-      for (int j = 0; j < COMBINE_SLICE / 128; ++j) {
-        const int i = i0 + j * 128;
+      for (int j = 0; j < C; ++j) {
+        const int i = i0 + j * STEP;
         if (i < W) v[j] = fmaf(wk, Num<TH>::to_float(h[(size_t)t * W + i]), v[j]);
       }
       continue;
     }
     const float* row = y + (size_t)pos * W;
+    if constexpr (V4) {
+      if (i0 < W) {
+        float r[C];
+        load4<float>(row + i0, r);
 #pragma unroll
-    for (int j = 0; j < COMBINE_SLICE / 128; ++j) {
-      const int i = i0 + j * 128;
+        for (int j = 0; j < C; ++j) v[j] = fmaf(wk, r[j], v[j]);
+      }
+      continue;
+    }
+#pragma unroll
+    for (int j = 0; j < C; ++j) {
+      const int i = i0 + j * STEP;
       if (i < W) v[j] = fmaf(wk, row[i], v[j]);
     }
   }
+  if constexpr (V4) {
+    if (i0 >= W) return;
+    float* o = out + (size_t)t * W + i0;
+    float was[C];
+    if (shared_out) {
+      load4<float>(shared_out + (size_t)t * W + i0, was);
 #pragma unroll
-  for (int j = 0; j < COMBINE_SLICE / 128; ++j) {
-    const int i = i0 + j * 128;
+      for (int j = 0; j < C; ++j) v[j] += g * was[j];
+    }
+    if (accumulate) load4<float>(o, was);
+#pragma unroll
+    for (int j = 0; j < C; ++j) v[j] = accumulate ? was[j] + v[j] * scale : v[j] * scale;
+    store4<float>(o, v);
+    return;
+  }
+#pragma unroll
+  for (int j = 0; j < C; ++j) {
+    const int i = i0 + j * STEP;
     if (i >= W) continue;
     float r = v[j];
     if (shared_out) r += g * shared_out[(size_t)t * W + i];
@@ -873,11 +899,13 @@ extern "C" int lse_moe_combine(const float* y, const int* pos_of, int top, const
                                cudaStream_t stream, const float* wts, const void* h, int h_dtype, float scale) {
   if (T <= 0) return LSE_OK;
   const dim3 grid(T, (W + COMBINE_SLICE - 1) / COMBINE_SLICE);
+  auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+  const bool v4 = W % 4 == 0 && aligned(y) && aligned(shared_out) && aligned(out);
   if (h && h_dtype == LSE_BF16)
-    launch(moe_combine_kernel<bf16>, grid, 128, 0, stream, y, pos_of, top, shared_out, gate, out, accumulate, W, wts,
+    launch(v4 ? moe_combine_kernel<bf16, true> : moe_combine_kernel<bf16, false>, grid, 128, 0, stream, y, pos_of, top, shared_out, gate, out, accumulate, W, wts,
            (const bf16*)h, scale);
   else if (!h || h_dtype == LSE_F32)
-    launch(moe_combine_kernel<float>, grid, 128, 0, stream, y, pos_of, top, shared_out, gate, out, accumulate, W, wts,
+    launch(v4 ? moe_combine_kernel<float, true> : moe_combine_kernel<float, false>, grid, 128, 0, stream, y, pos_of, top, shared_out, gate, out, accumulate, W, wts,
            (const float*)h, scale);
   else
     return LSE_BAD_ARGUMENT;

@@ -234,31 +234,48 @@ __global__ void sum_add_rmsnorm_kernel(float* __restrict__ x, const SumItems ite
   pdl_wait();
   const size_t at = (size_t)blockIdx.x * H;
   auto sum_at = [&](int i, float (&o)[V]) {
+    float y[SUM_MAX][V];
     if constexpr (V == 4) load4<float>(x + at + i, o);
     else o[0] = x[at + i];
 #pragma unroll
-    for (int m = 0; m < SUM_MAX; ++m) {
+    for (int m = 0; m < SUM_MAX; ++m) {  // every load is on its way before the first store
       if (m >= items.n) break;
-      float y[V];
       if (items.fixed[m]) {
-        fixed64* p = reinterpret_cast<fixed64*>(const_cast<void*>(items.y[m])) + at + i;
+        const fixed64* p = reinterpret_cast<const fixed64*>(items.y[m]) + at + i;
         if constexpr (V == 4) {
-          load4<fixed64>(p, y);
+          const longlong2 a = reinterpret_cast<const longlong2*>(p)[0], b = reinterpret_cast<const longlong2*>(p)[1];
+          y[m][0] = fixed_to_float(a.x); y[m][1] = fixed_to_float(a.y);
+          y[m][2] = fixed_to_float(b.x); y[m][3] = fixed_to_float(b.y);
         } else {
-          y[0] = fixed_to_float(p[0]);
-          p[0] = 0;
+          y[m][0] = fixed_to_float(p[0]);
         }
       } else {
         const float* p = reinterpret_cast<const float*>(items.y[m]) + at + i;
-        if constexpr (V == 4) load4<float>(p, y);
-        else y[0] = p[0];
+        if constexpr (V == 4) load4<float>(p, y[m]);
+        else y[m][0] = p[0];
+      }
+    }
+#pragma unroll
+    for (int m = 0; m < SUM_MAX; ++m) {
+      if (m >= items.n) break;
+      if (items.fixed[m]) {
+        fixed64* p = reinterpret_cast<fixed64*>(const_cast<void*>(items.y[m])) + at + i;
+        if constexpr (V == 4) {
+          reinterpret_cast<longlong2*>(p)[0] = make_longlong2(0, 0);
+          reinterpret_cast<longlong2*>(p)[1] = make_longlong2(0, 0);
+        } else {
+          p[0] = 0;
+        }
       }
 #pragma unroll
-      for (int j = 0; j < V; ++j) o[j] = fmaf(items.c[m], y[j], o[j]);
+      for (int j = 0; j < V; ++j) o[j] = fmaf(items.c[m], y[m][j], o[j]);
     }
     if (row) {
+      float r[V];
+      if constexpr (V == 4) load4<float>(row + i, r);
+      else r[0] = row[i];
 #pragma unroll
-      for (int j = 0; j < V; ++j) o[j] += row[i + j];
+      for (int j = 0; j < V; ++j) o[j] += r[j];
     }
     if constexpr (V == 4) store4<float>(x + at + i, o);
     else x[at + i] = o[0];
@@ -449,11 +466,12 @@ __device__ __forceinline__ float silu_times(float a, float u, int act, float lim
   else return a / (1.f + expf(-a)) * u;
 }
 template <typename TIn, typename T>
-__global__ void silu_mul_kernel(const TIn* __restrict__ gu, T* __restrict__ out, int I, int act, float limit) {
+__global__ void silu_mul_kernel(const TIn* __restrict__ gu, T* __restrict__ out, int I, int act, float limit,
+                                long long stride) {
   pdl_trigger();
   pdl_wait();
   const size_t t = blockIdx.x;
-  const TIn* g = gu + t * 2 * I;
+  const TIn* g = gu + t * stride;
   const TIn* u = g + I;
   T* o = out + t * I;
   if (I % 4 == 0) {
@@ -675,11 +693,15 @@ extern "C" int lse_sum_add_rmsnorm(float* x, const void* const* y, const float* 
     items.fixed[i] = dtypes[i] == LSE_FIXED64;
   }
   const bool vec = H % 4 == 0;
-  const int per = vec ? 16 : 4, kept = H <= 1024 * per;  // elements per thread whose visits stay in registers
+  // few rows: as many threads as a row has vectors, so that all of it is on its way at once
+  const bool wide = vec && H <= 4096 && T <= 256;
+  const int per = wide ? 4 : vec ? 16 : 4, kept = H <= 1024 * per;  // elements per thread whose visits stay in registers
   const int threads = kept ? ((H + per - 1) / per + 31) / 32 * 32 : 1024;
 #define LSE_SUM(TO)                                                                                              \
   do {                                                                                                           \
-    if (vec && kept)                                                                                             \
+    if (wide)                                                                                                    \
+      launch(sum_add_rmsnorm_kernel<TO, 4, 1>, T, threads, 0, stream, x, items, row, weight, eps, (TO*)out, H);  \
+    else if (vec && kept)                                                                                        \
       launch(sum_add_rmsnorm_kernel<TO, 4, 4>, T, threads, 0, stream, x, items, row, weight, eps, (TO*)out, H);  \
     else if (vec)                                                                                                \
       launch(sum_add_rmsnorm_kernel<TO, 4, 0>, T, threads, 0, stream, x, items, row, weight, eps, (TO*)out, H);  \
@@ -737,12 +759,15 @@ extern "C" int lse_rope_kv_write(const void* qkv, int in_dtype, void* q_out, int
 }
 
 extern "C" int lse_silu_mul(const void* gu, int in_dtype, void* out, int dtype, int T, int I,
-                            int act, cudaStream_t stream, float limit) {
+                            int act, cudaStream_t stream, float limit, long long stride) {
   if (T <= 0 || I <= 0) return LSE_OK;
+  if (stride != 0 && (stride < 2LL * I || in_dtype != LSE_F32 ||
+                      (I % 4 == 0 && (stride % 4 || reinterpret_cast<uintptr_t>(gu) % 16))))
+    return LSE_BAD_ARGUMENT;
   if (act != LSE_ACT_SILU && act != LSE_ACT_GELU_TANH && act != LSE_ACT_CLAMPED_GLU) return LSE_BAD_ARGUMENT;
   const int threads = 256;
   const int vec = in_dtype == LSE_BF16 ? 8 : 4;
-  if (in_dtype == dtype && I % vec == 0 && (size_t)T * (I / vec) < (1ull << 31) &&
+  if (stride == 0 && in_dtype == dtype && I % vec == 0 && (size_t)T * (I / vec) < (1ull << 31) &&
       (reinterpret_cast<uintptr_t>(gu) % 16) == 0 && (reinterpret_cast<uintptr_t>(out) % 16) == 0) {
     const unsigned total = (unsigned)((size_t)T * (I / vec));
     const unsigned blocks = (total + threads - 1) / threads;
@@ -754,14 +779,15 @@ extern "C" int lse_silu_mul(const void* gu, int in_dtype, void* out, int dtype, 
   }
   const int per_block = threads * 4;
   dim3 grid(T, min((I + per_block - 1) / per_block, 65535));
+  if (stride == 0) stride = 2LL * I;
   if (in_dtype == LSE_F32 && dtype == LSE_F32)
-    launch(silu_mul_kernel<float, float>, grid, threads, 0, stream, (const float*)gu, (float*)out, I, act, limit);
+    launch(silu_mul_kernel<float, float>, grid, threads, 0, stream, (const float*)gu, (float*)out, I, act, limit, stride);
   else if (in_dtype == LSE_BF16 && dtype == LSE_BF16)
-    launch(silu_mul_kernel<bf16, bf16>, grid, threads, 0, stream, (const bf16*)gu, (bf16*)out, I, act, limit);
+    launch(silu_mul_kernel<bf16, bf16>, grid, threads, 0, stream, (const bf16*)gu, (bf16*)out, I, act, limit, stride);
   else if (in_dtype == LSE_F32 && dtype == LSE_BF16)
-    launch(silu_mul_kernel<float, bf16>, grid, threads, 0, stream, (const float*)gu, (bf16*)out, I, act, limit);
+    launch(silu_mul_kernel<float, bf16>, grid, threads, 0, stream, (const float*)gu, (bf16*)out, I, act, limit, stride);
   else if (in_dtype == LSE_FIXED64 && dtype == LSE_BF16 && I % 4 == 0)
-    launch(silu_mul_kernel<fixed64, bf16>, grid, threads, 0, stream, (const fixed64*)gu, (bf16*)out, I, act, limit);
+    launch(silu_mul_kernel<fixed64, bf16>, grid, threads, 0, stream, (const fixed64*)gu, (bf16*)out, I, act, limit, stride);
   else
     return LSE_BAD_ARGUMENT;
   return LSE_CHECK_LAUNCH();

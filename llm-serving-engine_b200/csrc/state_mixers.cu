@@ -328,6 +328,45 @@ __global__ void gated_group_norm_kernel(const float* __restrict__ o, const float
   }
 }
 
+// The same for groups of whole 16-byte vectors (at most 1024 values): a warp per (row, group), four values per lane
+// and visit, held in registers between the two.
+constexpr int GGN_WARPS = 4, GGN_VISITS = 8;
+template <typename TO, int K>
+__global__ void __launch_bounds__(GGN_WARPS * 32)
+gated_group_norm_warp_kernel(const float* __restrict__ o, const float* __restrict__ gate, long long gate_stride, int N,
+                             int group, const float* __restrict__ weight, float eps, int sigmoid, TO* __restrict__ out,
+                             long long units) {
+  pdl_trigger();
+  pdl_wait();
+  const long long u = (long long)blockIdx.x * GGN_WARPS + (threadIdx.x >> 5);
+  if (u >= units) return;
+  const int per_row = N / group, lane = threadIdx.x & 31;
+  const long long t = u / per_row;
+  const int g = (int)(u - t * per_row) * group;
+  float v[K][4], z[K][4];
+  float ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < K; ++k) {
+    const int i = (lane + 32 * k) * 4;
+    if (i >= group) continue;
+    load4<float>(o + (size_t)t * N + g + i, v[k]);
+    load4<float>(gate + (size_t)t * gate_stride + g + i, z[k]);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) ss += v[k][e] * v[k][e];
+  }
+  const float inv = rsqrtf(warp_sum(ss) / (float)group + eps);
+#pragma unroll
+  for (int k = 0; k < K; ++k) {
+    const int i = (lane + 32 * k) * 4;
+    if (i >= group) continue;
+    float w[4] = {1.f, 1.f, 1.f, 1.f};
+    if (weight) load4<float>(weight + g + i, w);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) v[k][e] *= inv * w[e] * (sigmoid ? sigmoid_f(z[k][e]) : silu_f(z[k][e]));
+    store4<TO>(out + (size_t)t * N + g + i, v[k]);
+  }
+}
+
 // ------------------------------------------------------------------------------------ q/k norm, rotation, page write
 // One warp per (token, head) of the projection's heads: nq query heads, nk key heads, then nk
 // value heads unless the values are the keys as projected. D <= 256.
@@ -927,6 +966,27 @@ extern "C" int lse_gated_group_norm(const float* o, const float* gate, long long
                                     int out_dtype, cudaStream_t stream) {
   if (T <= 0) return LSE_OK;
   if (group <= 0 || N % group || N / group > 65535) return LSE_BAD_ARGUMENT;
+  auto aligned = [](const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; };
+  if (group % 4 == 0 && group <= 128 * GGN_VISITS && gate_stride % 4 == 0 && aligned(o) && aligned(gate) &&
+      aligned(weight) && aligned(out)) {
+    const long long units = (long long)T * (N / group);
+    const unsigned blocks = (unsigned)((units + GGN_WARPS - 1) / GGN_WARPS);
+#define LSE_GGN(K)                                                                                                  \
+  do {                                                                                                              \
+    if (out_dtype == LSE_BF16)                                                                                      \
+      launch(gated_group_norm_warp_kernel<bf16, K>, blocks, GGN_WARPS * 32, 0, stream, o, gate, gate_stride, N,     \
+             group, weight, eps, sigmoid, (bf16*)out, units);                                                       \
+    else if (out_dtype == LSE_F32)                                                                                  \
+      launch(gated_group_norm_warp_kernel<float, K>, blocks, GGN_WARPS * 32, 0, stream, o, gate, gate_stride, N,    \
+             group, weight, eps, sigmoid, (float*)out, units);                                                      \
+    else return LSE_BAD_ARGUMENT;                                                                                   \
+  } while (0)
+    if (group <= 128) LSE_GGN(1);
+    else if (group <= 256) LSE_GGN(2);
+    else LSE_GGN(8);
+#undef LSE_GGN
+    return LSE_CHECK_LAUNCH();
+  }
   const int threads = group >= 1024 ? 256 : (group >= 128 ? 128 : (group > 32 ? 64 : 32));
   dim3 grid(T, N / group);
   if (out_dtype == LSE_BF16)

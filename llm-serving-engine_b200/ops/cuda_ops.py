@@ -263,13 +263,15 @@ class CudaOps:
 
     _ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "clamped_glu": 2}
 
-    def silu_mul(self, gu, out_dtype=None, activation="silu", limit=0.0):
+    def silu_mul(self, gu, out_dtype=None, activation="silu", limit=0.0, columns=None):
         """``act(gate) * up`` of ``gu = [gate | up]``; ``activation``: silu or gelu_tanh, or
         ``clamped_glu``: ``g sigmoid(1.702 g) (u + 1)`` with the gate cut at ``limit`` from above
-        and ``u`` between ``-limit`` and ``limit``."""
+        and ``u`` between ``-limit`` and ``limit``. ``columns``: gate and up are these columns ``(first,
+        number)`` of a wider float32 matrix."""
         out_dtype = out_dtype or gu.dtype
-        out = torch.empty(gu.shape[0], gu.shape[1] // 2, dtype=out_dtype, device=gu.device)
-        self.ext.silu_mul(gu, out, self._ACTIVATIONS[activation], float(limit))
+        col0, n = columns or (0, gu.shape[1])
+        out = torch.empty(gu.shape[0], n // 2, dtype=out_dtype, device=gu.device)
+        self.ext.silu_mul(gu, out, self._ACTIVATIONS[activation], float(limit), int(col0))
         self.launches += 1
         return out
 
@@ -278,6 +280,11 @@ class CudaOps:
         """Does the own tcgen05 kernel serve this product?"""
         return (self.use_skinny_gemm and a.dtype == torch.bfloat16 and w.dtype == torch.bfloat16
                 and a.shape[0] <= self.skinny_max_rows and a.shape[1] % 8 == 0)
+
+    def shares_products(self, a, w) -> bool:
+        """Is one product with ``w`` better than one with each of its parts? Where few rows stream the weights
+        once, a launch is all that the parts cost more; where the library runs, the parts keep their own dtypes."""
+        return self._few_rows(a, w)
 
     def linear(self, a, w, bias=None, out_dtype=None, accumulate_into=None, may_defer=False, coefficient=None):
         """``a @ w.T (+ bias)`` as a new tensor of ``out_dtype`` (None: the compute dtype).

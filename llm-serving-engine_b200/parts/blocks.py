@@ -23,6 +23,8 @@ that reads ``x`` next, so a block returns its feed-forward output as ``pending``
     h = norm(x);   x <- x + coefficient * (mixer(h) + feed_forward(h))
 
 (the feed-forward is optional). What is not added on the way is left for the norm that reads ``x`` next.
+Where both sublayers can start from columns of a product (``input_weight``, ``forward_projected``), their matrices lie
+one below the other, and a kernel set that streams weights (few rows) makes one product of both.
 
 ``filter`` is an optional input filter of the mixer (a token shift, say); the feed-forward is
 optional too. A filter that keeps something per request shares the block's cache layer with the
@@ -33,6 +35,8 @@ from __future__ import annotations
 
 from dataclasses import dataclass
 from typing import Any
+
+import torch
 
 from .base import (BLOCKS, FEED_FORWARDS, INPUT_FILTERS, MIXERS, NORMS, Block, PendingAdds, PendingNormedBranch,
                    count_states, flatten_needs, has_pages, settle)
@@ -202,9 +206,31 @@ class SharedNormBlock(Block):
         self.norm = self.children["norm"]
         self.mixer = self.children["mixer"]
         self.feed_forward = self.children.get("feed_forward")
+        self.shared_weight = None
+
+    def bind(self, params):
+        super().bind(params)
+        weights = [getattr(p, "input_weight", None) for p in (self.mixer, self.feed_forward)]
+        if any(w is None for w in weights):
+            return
+        mix, ff = weights
+        self.ff_column = mix.shape[0] + (-mix.shape[0]) % 8
+        rows = self.ff_column + ff.shape[0] + (-ff.shape[0]) % 8
+        w = mix.new_zeros(rows, mix.shape[1])
+        w[: mix.shape[0]] = mix
+        w[self.ff_column : self.ff_column + ff.shape[0]] = ff
+        self.shared_weight = w
+        self.mixer.input_weight = w[: mix.shape[0]]  # views: each may still make its own product
+        self.feed_forward.input_weight = w[self.ff_column : self.ff_column + ff.shape[0]]
 
     def forward(self, x, pending, step, cache):
         h = self.norm.forward(x, settle(pending, self.norm))
+        if self.shared_weight is not None and self.ops.shares_products(h, self.shared_weight):
+            proj = self.ops.linear(h, self.shared_weight, None, out_dtype=torch.float32)
+            add_to = (x, self.spec.coefficient)
+            items = self.mixer.forward_projected(proj, 0, step, cache, add_to=add_to)
+            items += self.feed_forward.forward_projected(proj, self.ff_column, add_to)
+            return x, PendingAdds(self.ops, x, items) if items else None
         items = self.mixer.forward_into(h, step, cache, x, self.spec.coefficient)
         if self.feed_forward is not None:
             items += self.feed_forward.forward_into(h, step, x, self.spec.coefficient)

@@ -58,6 +58,22 @@ class SwiGLU(FeedForward):
     def forward_into(self, h, step, x, coefficient):
         return add_projected(self.ops, self._inner(h), self.down_weight, None, x, coefficient)
 
+    @property
+    def input_weight(self):
+        """The matrix of this part's product with its input, where a block may make it part of a larger one."""
+        return self.gate_up_weight
+
+    @input_weight.setter
+    def input_weight(self, w):
+        self.gate_up_weight = w
+
+    def forward_projected(self, proj, col0, add_to):
+        """``forward_into`` (``add_to = (x, coefficient)``) from the float32 product with the input, whose columns for
+        this part start at ``col0``."""
+        a = self.ops.silu_mul(proj, out_dtype=self.env.dtype, activation=self.spec.activation,
+                              columns=(col0, 2 * self.spec.intermediate_size), **self._options)
+        return add_projected(self.ops, a, self.down_weight, None, *add_to)
+
     def _inner(self, h):
         if self.spec.activation == "silu":
             return self.ops.gated_silu(h, self.gate_up_weight, None, out_dtype=self.env.dtype)

@@ -81,9 +81,18 @@ class ParallelMixer(Mixer):
             extra = (-w.shape[0]) % 8
             padded += [w] + ([w.new_zeros(extra, w.shape[1])] if extra else [])
             at += w.shape[0] + extra
-        self.shared_weight = torch.cat(padded, 0).contiguous()
-        for b, w, c in zip(self.branches, weights, self.columns):
-            b.input_weight = self.shared_weight[c : c + w.shape[0]]
+        self.input_weight = torch.cat(padded, 0).contiguous()
+
+    @property
+    def input_weight(self):
+        """The matrix of the branches' one product with the input (None: they make their own)."""
+        return self.shared_weight
+
+    @input_weight.setter
+    def input_weight(self, w):
+        self.shared_weight = w
+        for b, c in zip(self.branches, self.columns):
+            b.input_weight = w[c : c + b.input_weight.shape[0]]
 
     def cache_need(self):
         return tuple(n for b in self.branches for n in flatten_needs(b.cache_need()))
@@ -93,14 +102,21 @@ class ParallelMixer(Mixer):
     def forward_into(self, h, step, cache, x, coefficient):
         if self.spec.normed:
             return [(coefficient, self.forward(h, step, cache).resolve())]
+        if self.shared_weight is not None:
+            proj = self.ops.linear(h, self.shared_weight, None, out_dtype=torch.float32)
+            return self.forward_projected(proj, 0, step, cache, add_to=(x, coefficient))
         items = []
-        proj = None if self.shared_weight is None else self.ops.linear(h, self.shared_weight, None, out_dtype=torch.float32)
-        for k, (b, c, (pages, first, n)) in enumerate(zip(self.branches, self.spec.coefficients, self._parts)):
-            part = cache.part(pages, first, n)
-            if proj is None:
-                items += b.forward_into(h, step, part, x, coefficient * c)
-            else:
-                items += b.forward_projected(proj, self.columns[k], step, part, add_to=(x, coefficient * c))
+        for b, c, part in zip(self.branches, self.spec.coefficients, self._parts):
+            items += b.forward_into(h, step, cache.part(*part), x, coefficient * c)
+        return items
+
+    def forward_projected(self, proj, col0, step, cache, add_to):
+        """``forward_into`` (``add_to = (x, coefficient)``) from the float32 product with the input, whose columns for
+        this mixer start at ``col0``."""
+        x, coefficient = add_to
+        items = []
+        for b, c, at, part in zip(self.branches, self.spec.coefficients, self.columns, self._parts):
+            items += b.forward_projected(proj, col0 + at, step, cache.part(*part), add_to=(x, coefficient * c))
         return items
 
     def forward(self, h, step, cache, may_defer=False):

@@ -662,13 +662,13 @@ TANUPEL_TINY = {
     # sizes that are multiples of nothing; a convolution of one tap and one of five; ranks unlike each other; no
     # rotation; every expert chosen; one layer that runs three times, the last; pages of 8 tokens
     "T2": dict(seed=13, page_tokens=8, config={
-        "architecture": "Tanupel", "vocab": 131, "width": 70, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0},
+        "architecture": "Tanupel", "vocab": 131, "width": 70, "norm": {"eps": 1e-3}, "embedding": {"scale": 1.0},
         "residual_mult": 1.0, "loop": {"start": 2, "stop": 3, "times": 3},
         "layers": [_tlayer(_tatt(3, 3, 18, 10, 0.3, (300.0, 6, (3.0,)), softcap=2.5), _tmoe(4, 4, 10),
                            _tdelta(5, 1, 10, 14, 1, (5, 11)), (1.0, 1.0)),
                    _tlayer(_tatt(2, 1, 20, 12, 0.3), _dense(50)),
                    _tlayer(_tatt(5, 1, 12, 12, 0.4, (1000.0, 12, (4.0, 1.0, 2.0, 40))), _tmoe(3, 1, 14),
-                           _tdelta(3, 1, 7, 20, 5, (3, 2)), (0.4, 2.0))]}),
+                           _tdelta(3, 1, 7, 20, 5, (3, 2)), (0.4, 0.9))]}),
     # the head sizes of larger models (tensor-core attention with and without a cap); a wide key of the delta
     # rule; many experts; no loop; a fully rotated head
     "T3": dict(seed=22, page_tokens=32, config={

@@ -80,7 +80,12 @@ class PlainOps:
         n = lambda y: y * torch.rsqrt(y.pow(2).mean(-1, keepdim=True) + eps)
         return (coef[0] * n(z) + coef[1] * n(z ** 2) + coef[2] * n(z ** 3) + coef[3]).to(out_dtype)
 
-    def silu_mul(self, gu, out_dtype=None, activation="silu", limit=0.0):
+    def shares_products(self, a, w):
+        return a.shape[0] <= 3  # so that steps of few rows and of many take both ways
+
+    def silu_mul(self, gu, out_dtype=None, activation="silu", limit=0.0, columns=None):
+        if columns is not None:
+            gu = gu[:, columns[0] : columns[0] + columns[1]]
         g, u = gu.float().chunk(2, dim=-1)
         if activation == "clamped_glu":
             g, u = g.clamp(max=limit), u.clamp(-limit, limit)
